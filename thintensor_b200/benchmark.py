@@ -19,7 +19,7 @@ from .sampling.sampler import SamplingParams
 
 # Named shapes for benchmarks with random weights, each a whole config.json: the three Llama 3
 # models the reference's reports measure, two tiny ones that differ in every size and option, and
-# two Famalorn, two Neruzen and two Sogidra models of six layers at the widths of the 1B and 3B Llama shapes.
+# two Famalorn, two Neruzen, two Sogidra, two Kerepel and two Zuvepel models of six layers at the widths of the 1B and 3B Llama shapes.
 # They are data (config/shapes.json), read here and by bench.py.
 SHAPES: dict[str, dict] = json.loads((Path(__file__).resolve().parent / "config" / "shapes.json").read_text(encoding="utf-8"))
 
@@ -84,14 +84,20 @@ def kv_read_bytes_per_token(model) -> int:
 
 def kv_read_bytes(model, context: float) -> float:
     """Bytes of keys and values a decode step reads for one sequence of ``context`` cached tokens: a run with a window
-    reads only the window's tokens, a coarser cache (a mixer's summary) one entry for each of its blocks."""
+    reads only the window's tokens, one with chunks its chunk's, a coarser cache (a mixer's summary) one entry for each of
+    its blocks."""
     kv, _, _ = model.cache_needs()
     width = torch.empty((), dtype=model.dtype).element_size()
+    chunked = {}                    # a run whose mask is chunks reads fewer keys than its cache keeps
+    for index, run in enumerate(model.spec.schedule):
+        for user, mixer in zip(model.users[index], model.layers[run.layer].mixers()):
+            if getattr(mixer, "chunk", None):
+                chunked[user] = mixer.visible_keys(context)
     def entries(need) -> float:     # a coarser cache holds one entry for each ``every`` tokens; a run with a window reads the window
         held = context / need.every
         return held if need.window is None else min(held, need.window)
 
-    return sum(need.kv_heads * (need.head_dim + need.v_dim) * width * entries(need) for need in kv if need is not None)
+    return sum(need.kv_heads * (need.head_dim + need.v_dim) * width * chunked.get(user, entries(need)) for user, need in enumerate(kv) if need is not None)
 
 
 def state_bytes_per_sequence(model) -> int:
@@ -194,7 +200,8 @@ def class_fractions(model, classes: dict, pk: dict, prefill_prompts: list[list[i
     sampling) has no bound worth naming and is given as time alone.  Times are those of kernels run
     one after another (see :func:`measure_classes`)."""
     attention_kernels = ("tt_attention", "tt_latent_attention", "tt_differential_attention", "tt_pooled_window_attention")
-    recurrent = ("tt_mamba2_scan", "tt_delta_scan", "tt_causal_conv", "tt_gated_group_norm", "tt_decay_scan", "tt_linear_attention_prepare")
+    recurrent = ("tt_mamba2_scan", "tt_delta_scan", "tt_causal_conv", "tt_gated_group_norm", "tt_decay_scan", "tt_row_decay_scan",
+                 "tt_low_rank", "tt_linear_attention_prepare")
 
     def split(spans: dict) -> dict:
         out = {"products": 0.0, "attention": 0.0, "recurrence": 0.0, "rest": 0.0}

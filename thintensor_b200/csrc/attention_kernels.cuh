@@ -74,7 +74,7 @@ __device__ __forceinline__ float attn_gate(const AttnExtra& x, int t, int h, int
     return 1.0f / (1.0f + expf(-z));
 }
 
-// window <= 0: all keys 0..pos.  window > 0: keys pos - window + 1 .. pos.
+// window: which keys a position sees, see tt_first_key.
 // Keys have head_dim numbers, values value_dim (the output's width per head).
 // sinks (float32, one per query head, or null): the softmax denominator also holds exp(sink_h), a
 // term that has no key and no value, is not multiplied by scale, and is counted once (by slice 0).
@@ -103,7 +103,7 @@ __global__ void attention_rows_kernel(const T* __restrict__ q, const T* __restri
     for (int d = lane; d < head_dim; d += 32) qs[d] = tt_to_float(q[((size_t)t * heads + h) * head_dim + d]) * scale;
     __syncwarp();
 
-    const int first = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    const int first = tt_first_key(pos, window);
     const int n_keys = pos - first + 1;
     int per = (n_keys + splits - 1) / splits;
     per = (per + 31) & ~31;

@@ -470,19 +470,19 @@ attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* _
         const int token = seq_begin + tok0 + local, head = kh * group + (r - local * group);
         row_q[i] = ((size_t)token * heads + head) * HD;
         st.row_pos[i] = row_ok[i] ? before + tok0 + local : -1;
-        st.row_first[i] = (window > 0 && st.row_pos[i] - window + 1 > 0) ? st.row_pos[i] - window + 1 : 0;
+        st.row_first[i] = tt_first_key(st.row_pos[i], window);
     }
     load_queries<HD>(st, q, row_q, row_ok, t);
 
     // blocks of keys: the CTA walks from the first block any of its rows sees to the last; a warp
     // skips the arithmetic of blocks beyond its own last position
     const int cta_lo = before + cta_tok0, cta_hi = before + cta_tok0 + cta_tokens - 1;
-    const int lo_key = (window > 0 && cta_lo - window + 1 > 0) ? cta_lo - window + 1 : 0;
+    const int lo_key = tt_first_key(cta_lo, window);
     const int block0 = lo_key / TT_BLOCK_TOKENS, block1 = cta_hi / TT_BLOCK_TOKENS;
     const int n_blocks = block1 - block0 + 1;
     const int my_hi = tile_tokens > 0 ? before + tok0 + tile_tokens - 1 : -1;
     const int my_lo = before + tok0;
-    const int my_lo_key = (window > 0 && my_lo - window + 1 > 0) ? my_lo - window + 1 : 0;
+    const int my_lo_key = tt_first_key(my_lo, window);
     const int* table_row = table + (size_t)b * table_width;
     uint8_t* stages = reinterpret_cast<uint8_t*>(stage_mem);
     unsigned bad = 0;                                            // bit i % 32: block i has no usable data
@@ -671,7 +671,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, DecodeRope rope, __
     for (int i = threadIdx.x; i < min(table_width, DECODE_TABLE_CACHE); i += WARPS * 32) table_sh[i] = table_row[i];
     const int pos = len_before[b];                    // position of this step's token = keys 0 .. pos
     __syncthreads();
-    const int lo_key = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    const int lo_key = tt_first_key(pos, window);
     const int block0 = lo_key / TT_BLOCK_TOKENS, block1 = pos / TT_BLOCK_TOKENS;
     const int per = (block1 - block0 + 1 + splits - 1) / splits;
     const int my_begin = block0 + split * per, my_end = min(block1 + 1, my_begin + per);

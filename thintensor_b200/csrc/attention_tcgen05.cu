@@ -170,7 +170,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     const int tok0 = tile * args.tokens_per_tile;
     const int tile_tokens = min(args.tokens_per_tile, seq_new - tok0);
     const int lo_pos = before + tok0, hi_pos = before + tok0 + tile_tokens - 1;
-    const int lo_key = (args.window > 0 && lo_pos - args.window + 1 > 0) ? lo_pos - args.window + 1 : 0;
+    const int lo_key = tt_first_key(lo_pos, args.window);
     const int block0 = lo_key / KEYS, block1 = hi_pos / KEYS;
     const int n_blocks = block1 - block0 + 1;
     // With a distance bias the blocks are walked from the nearest keys back: a row's largest score is then met in its first
@@ -257,7 +257,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         const int local = r / args.group;
         const bool row_ok = local < tile_tokens;
         const int pos = row_ok ? before + tok0 + local : -1;
-        const int first = (args.window > 0 && pos - args.window + 1 > 0) ? pos - args.window + 1 : 0;
+        const int first = tt_first_key(pos, args.window);
         const uint32_t lane_base = tmem_base + ((uint32_t)(quarter * 32) << 16);
         constexpr int SPLIT = L::SPLIT, HALF_KEYS = KEYS / SPLIT, O_COLS = HD / SPLIT;   // what one thread of a row handles
         float m_used = -INFINITY, l = 0.0f;                       // the scale in use (log2 units) and this thread's part of the sum

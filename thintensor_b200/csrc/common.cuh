@@ -125,6 +125,14 @@ __device__ __forceinline__ int tt_find_sequence(const int* __restrict__ cu, int 
     return lo;
 }
 
+// The first key that a query at position `pos` sees (its last is its own).  window == 0: every key; window > 0: the last
+// `window` of them; window < 0: the keys of its own chunk, chunks of -window positions counted from position 0 of the
+// sequence.  Later positions never see earlier first keys, so a tile of queries starts at its first query's.
+__device__ __forceinline__ int tt_first_key(int pos, int window) {
+    if (window < 0) return pos - pos % -window;
+    return (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+}
+
 // The cache of one layer is two block pools.  Keys:   [block][kv_head][TT_BLOCK_TOKENS][head_dim]
 // (a token's head vector is contiguous).  Values: [block][kv_head][head_dim][TT_BLOCK_TOKENS]
 // (transposed: the 64 tokens of one head dimension are contiguous, which is the operand

@@ -1,5 +1,6 @@
 // Memory-bound kernels between the matrix products: embedding gather (also with a hashed
-// row for the pair of the previous token and this one), residual add fused with RMSNorm,
+// row for the pair of the previous token and this one), residual add fused with RMSNorm (also with two scaled
+// branches added and two norms taken of the sum),
 // the token shift of a mixer's input, rotary encoding fused with the cache append, SwiGLU,
 // and the length bookkeeping of a step.  All statistics, angles and sums are float32.
 //
@@ -256,6 +257,200 @@ extern "C" int tt_add_layernorm(float* residual, const float* delta, int splits,
                                 const float* weight, const float* bias, float eps, void* out, int out_dtype,
                                 const int* rows, int n_rows, int hidden, cudaStream_t stream) {
     return add_norm(residual, delta, splits, split_stride, weight, 0.0f, eps, out, out_dtype, rows, n_rows, hidden, 1, bias, stream);
+}
+
+// ------------------------------------------------------------------------------------
+// residual add of two scaled branches and an addend, and one or two norms of the sum.
+//   x = residual[r] + scale * (sum_s a[s][r] + sum_s b[s][r]) + addend[r]       (each of a, b and addend may be null)
+//   residual[r] = x                                                             (only when rows == nullptr)
+//   out1[i] = norm(x) * w1 [+ b1], out2[i] = norm(x) * w2 [+ b2]                (out2 may be null)
+// norm: divided by the root mean square, or the mean taken off and divided by the standard deviation (centered).  A layer
+// whose mixer and feed-forward read the same stream through norms of their own takes the statistics once.
+// One block per output row; rows as for the kernels above.
+// ------------------------------------------------------------------------------------
+struct NormBranches {
+    const float* a;
+    const float* b;
+    const float* addend;
+    int a_splits, b_splits;
+    size_t a_stride, b_stride;
+    float scale;
+};
+struct NormOutputs {
+    const float* w1;
+    const float* b1;
+    const float* w2;
+    const float* b2;
+    void* out1;
+    void* out2;
+    float weight_offset, eps;
+    int centered;
+};
+
+template <typename TOut, int PIECES, int BATCH>
+__global__ void __launch_bounds__(1024)
+add_norms_vec_kernel(float* __restrict__ residual, const NormBranches in, const NormOutputs to, const int* __restrict__ rows, int hidden) {
+    tt_pdl_launch_dependents();
+    __shared__ float reduce[32];
+    const int i = blockIdx.x;
+    const int quads = hidden >> 2;
+    // what no kernel writes is fetched while the previous kernel still runs
+    float4 w1[PIECES], w2[PIECES];
+#pragma unroll
+    for (int v = 0; v < PIECES; ++v) {
+        const int j = threadIdx.x + v * blockDim.x;
+        if (j < quads) {
+            w1[v] = __ldg(reinterpret_cast<const float4*>(to.w1) + j);
+            if (to.out2) w2[v] = __ldg(reinterpret_cast<const float4*>(to.w2) + j);
+        }
+    }
+    tt_pdl_wait();
+    const int r = rows ? rows[i] : i;
+    float4* res = reinterpret_cast<float4*>(residual + (size_t)r * hidden);
+    const bool changed = in.a_splits + in.b_splits > 0 || in.addend;
+    float4 x[PIECES];
+    float sumsq = 0.0f, sum = 0.0f;
+#pragma unroll
+    for (int v = 0; v < PIECES; ++v) {
+        const int j = threadIdx.x + v * blockDim.x;
+        if (j < quads) {
+            float4 y = res[j];
+            float4 d = make_float4(0.0f, 0.0f, 0.0f, 0.0f), more = d;
+            if (in.addend) more = __ldg(reinterpret_cast<const float4*>(in.addend + (size_t)r * hidden) + j);
+            auto add = [&](const float* branch, int splits, size_t stride) {      // BATCH slices' loads in flight together, added in order
+                const float4* p = reinterpret_cast<const float4*>(branch + (size_t)r * hidden) + j;
+                for (int s0 = 0; s0 < splits; s0 += BATCH) {
+                    float4 q[BATCH];
+#pragma unroll
+                    for (int e = 0; e < BATCH; ++e)
+                        if (s0 + e < splits) q[e] = __ldg(p + (size_t)(s0 + e) * (stride >> 2));
+#pragma unroll
+                    for (int e = 0; e < BATCH; ++e)
+                        if (s0 + e < splits) { d.x += q[e].x; d.y += q[e].y; d.z += q[e].z; d.w += q[e].w; }
+                }
+            };
+            if (in.a_splits > 0) add(in.a, in.a_splits, in.a_stride);
+            if (in.b_splits > 0) add(in.b, in.b_splits, in.b_stride);
+            y.x = fmaf(in.scale, d.x, y.x) + more.x;
+            y.y = fmaf(in.scale, d.y, y.y) + more.y;
+            y.z = fmaf(in.scale, d.z, y.z) + more.z;
+            y.w = fmaf(in.scale, d.w, y.w) + more.w;
+            if (!rows && changed) res[j] = y;
+            x[v] = y;
+            sumsq += y.x * y.x + y.y * y.y + y.z * y.z + y.w * y.w;
+            sum += (y.x + y.y) + (y.z + y.w);
+        }
+    }
+    float total;
+    if (to.centered) {
+        const float mean = tt_block_sum(sum, reduce) / (float)hidden;
+        float dev = 0.0f;
+#pragma unroll
+        for (int v = 0; v < PIECES; ++v) {
+            const int j = threadIdx.x + v * blockDim.x;
+            if (j < quads) {
+                x[v].x -= mean; x[v].y -= mean; x[v].z -= mean; x[v].w -= mean;
+                dev += x[v].x * x[v].x + x[v].y * x[v].y + x[v].z * x[v].z + x[v].w * x[v].w;
+            }
+        }
+        total = tt_block_sum(dev, reduce);
+    } else {
+        total = tt_block_sum(sumsq, reduce);
+    }
+    const float rstd = rsqrtf(total / (float)hidden + to.eps);
+    auto put = [&](void* out, const float4& w, const float* bias, int v, int j) {
+        const float o = to.weight_offset;
+        float4 b = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (bias) b = __ldg(reinterpret_cast<const float4*>(bias) + j);
+        tt_store4((TOut*)out + (size_t)i * hidden + 4 * j, fmaf(x[v].x * rstd, w.x + o, b.x), fmaf(x[v].y * rstd, w.y + o, b.y),
+                  fmaf(x[v].z * rstd, w.z + o, b.z), fmaf(x[v].w * rstd, w.w + o, b.w));
+    };
+#pragma unroll
+    for (int v = 0; v < PIECES; ++v) {
+        const int j = threadIdx.x + v * blockDim.x;
+        if (j < quads) {
+            put(to.out1, w1[v], to.b1, v, j);
+            if (to.out2) put(to.out2, w2[v], to.b2, v, j);
+        }
+    }
+}
+
+// any width; the row is kept in shared memory as far as row_cache floats reach
+template <typename TOut>
+__global__ void add_norms_kernel(float* __restrict__ residual, const NormBranches in, const NormOutputs to, const int* __restrict__ rows,
+                                 int hidden, int row_cache) {
+    tt_pdl_launch_dependents();
+    tt_pdl_wait();
+    extern __shared__ float row_shared[];
+    float* reduce = row_shared + row_cache;
+    const int i = blockIdx.x;
+    const int r = rows ? rows[i] : i;
+    float* res = residual + (size_t)r * hidden;
+    const bool changed = in.a_splits + in.b_splits > 0 || in.addend;
+    auto value = [&](int j) {
+        const size_t at = (size_t)r * hidden + j;
+        float d = 0.0f;
+        for (int s = 0; s < in.a_splits; ++s) d += in.a[(size_t)s * in.a_stride + at];
+        for (int s = 0; s < in.b_splits; ++s) d += in.b[(size_t)s * in.b_stride + at];
+        return fmaf(in.scale, d, res[j]) + (in.addend ? in.addend[at] : 0.0f);
+    };
+    float sumsq = 0.0f, sum = 0.0f;
+    for (int j = threadIdx.x; j < hidden; j += blockDim.x) {
+        const float x = value(j);
+        if (j < row_cache) row_shared[j] = x;
+        if (!rows && changed) res[j] = x;
+        sumsq += x * x;
+        sum += x;
+    }
+    auto again = [&](int j) { return j < row_cache ? row_shared[j] : rows ? value(j) : res[j]; };
+    float mean = 0.0f, total;
+    if (to.centered) {
+        mean = tt_block_sum(sum, reduce) / (float)hidden;
+        float dev = 0.0f;
+        for (int j = threadIdx.x; j < hidden; j += blockDim.x) { const float d = again(j) - mean; dev += d * d; }
+        total = tt_block_sum(dev, reduce);
+    } else {
+        total = tt_block_sum(sumsq, reduce);
+    }
+    const float rstd = rsqrtf(total / (float)hidden + to.eps);
+    for (int j = threadIdx.x; j < hidden; j += blockDim.x) {
+        const float y = (again(j) - mean) * rstd;
+        ((TOut*)to.out1)[(size_t)i * hidden + j] = tt_from_float<TOut>(fmaf(y, to.w1[j] + to.weight_offset, to.b1 ? to.b1[j] : 0.0f));
+        if (to.out2) ((TOut*)to.out2)[(size_t)i * hidden + j] = tt_from_float<TOut>(fmaf(y, to.w2[j] + to.weight_offset, to.b2 ? to.b2[j] : 0.0f));
+    }
+}
+
+extern "C" int tt_add_norms(float* residual, const float* a, int a_splits, long long a_stride, const float* b, int b_splits, long long b_stride,
+                            float scale, const float* addend, const float* w1, const float* b1, void* out1, const float* w2, const float* b2,
+                            void* out2, float weight_offset, float eps, int centered, int out_dtype, const int* rows, int n_rows, int hidden,
+                            cudaStream_t stream) {
+    if (n_rows <= 0) return 0;
+    if (!w1 || !out1 || (out2 && !w2)) return (int)cudaErrorInvalidValue;
+    const NormBranches in{a, b, addend, a ? a_splits : 0, b ? b_splits : 0, (size_t)a_stride, (size_t)b_stride, scale};
+    const NormOutputs to{w1, b1, w2, b2, out1, out2, weight_offset, eps, centered};
+    const uintptr_t bases = (uintptr_t)residual | (uintptr_t)a | (uintptr_t)b | (uintptr_t)addend | (uintptr_t)w1 | (uintptr_t)b1 |
+                            (uintptr_t)w2 | (uintptr_t)b2 | (uintptr_t)out1 | (uintptr_t)out2;
+    if (hidden % 4 == 0 && hidden <= 4096 * NORM_VEC_MAX && a_stride % 4 == 0 && b_stride % 4 == 0 && (bases & 15) == 0) {
+        int threads = ((hidden / 4 + 31) / 32) * 32;
+        if (threads > 1024) threads = 1024;
+        if (n_rows >= 1024) {                                     // prompts: fewer, fatter blocks, as above
+            const int fewest = (((hidden / 4 + NORM_VEC_MAX - 1) / NORM_VEC_MAX + 31) / 32) * 32;
+            threads = fewest < 128 ? 128 : fewest;
+            if (threads > 1024) threads = 1024;
+        }
+        const bool one_piece = threads * 4 >= hidden;
+#define TT_NORMS(T, P, B) tt_launch_pdl(add_norms_vec_kernel<T, P, B>, dim3(n_rows), dim3(threads), 0, stream, residual, in, to, rows, hidden)
+        if (out_dtype == TT_F32) { if (one_piece) TT_NORMS(float, 1, 8); else TT_NORMS(float, NORM_VEC_MAX, 2); }
+        else { if (one_piece) TT_NORMS(__nv_bfloat16, 1, 8); else TT_NORMS(__nv_bfloat16, NORM_VEC_MAX, 2); }
+#undef TT_NORMS
+        TT_LAUNCH_CHECK();
+    }
+    const int threads = hidden >= 2048 ? 512 : (hidden >= 512 ? 256 : 128);
+    const int row_cache = hidden <= 11264 ? hidden : 11264;
+    const size_t shared = (size_t)(row_cache + 32) * sizeof(float);
+    if (out_dtype == TT_F32) tt_launch_pdl(add_norms_kernel<float>, dim3(n_rows), dim3(threads), shared, stream, residual, in, to, rows, hidden, row_cache);
+    else tt_launch_pdl(add_norms_kernel<__nv_bfloat16>, dim3(n_rows), dim3(threads), shared, stream, residual, in, to, rows, hidden, row_cache);
+    TT_LAUNCH_CHECK();
 }
 
 // ------------------------------------------------------------------------------------

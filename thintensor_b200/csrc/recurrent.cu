@@ -1,7 +1,8 @@
 // Kernels of the recurrent token mixers: the short causal convolution with its carried inputs, the
 // Mamba-2 state-space recurrence (also run with a constant decay and step size one: the linear
 // attention S <- g S + k v^T, o = S^T q, whose q, k and v a kernel here prepares), the gated delta-rule
-// recurrence, the gated group norm behind them (gate: silu or sigmoid), and the weighted sum of two branches.  Everything here is float32: inputs are the float32 partial
+// recurrence, both also with a decay of its own for every head and state row at every token, the products of low rank
+// that such decays (and gates) come from, the gated group norm behind them (gate: silu or sigmoid), and the weighted sum of two branches.  Everything here is float32: inputs are the float32 partial
 // sums of a projection ([splits][tokens][cols], summed on the way in), states live in float32 and are
 // carried per sequence slot, and only the normalised output that feeds the next matrix product is
 // narrowed to the activation dtype.
@@ -255,20 +256,22 @@ extern "C" int tt_causal_conv(const float* proj, int splits, long long split_str
 // G column groups of REC_LANES lanes per CTA, each owning C neighbouring columns: (32, 1) gives a sequence the most
 // warps (one long prompt, decoding); (16, 4) reads a token's vectors from shared memory once for four columns, which is
 // what bounds the kernel once the grid fills the GPU (batches of prompts).
-template <int K, int G, int C>
+// ROWS: every token brings a decay for each state row of its head (row_decay, float32 [tokens][groups * N], one more
+// vector staged beside B and C) instead of one for the head; step sizes are one and there is no skip.
+template <int K, int G, int C, bool ROWS>
 __global__ void __launch_bounds__(G* REC_LANES)
 mamba2_scan_kernel(const float* __restrict__ xbc, int xbc_cols, const float* __restrict__ proj, int splits, size_t split_stride,
                    int cols, int dt_col, const float* __restrict__ dt_bias, const float* __restrict__ a_log,
                    const float* __restrict__ d_skip, float* __restrict__ state, float* __restrict__ y,
                    const int* __restrict__ cu, const int* __restrict__ slots, int heads, int P, int N, int groups, int chunk,
-                   int vec, const float* __restrict__ fixed_decay) {
+                   int vec, const float* __restrict__ fixed_decay, const float* __restrict__ row_decay) {
     tt_pdl_launch_dependents();
     tt_pdl_wait();
     extern __shared__ __align__(16) float rec_shared[];
-    // two buffers of: B [chunk][NP], C [chunk][NP], x [chunk][TILE], decay [chunk], step [chunk]; rows are padded to
-    // NP = K * REC_LANES numbers and the padding is zero, so the token loop needs no bounds
-    constexpr int NP = K * REC_LANES, TILE = G * C;
-    const int buffer_floats = 2 * chunk * NP + chunk * TILE + 2 * chunk;
+    // two buffers of: B [chunk][NP], C [chunk][NP], (ROWS) decays [chunk][NP], x [chunk][TILE], decay [chunk], step [chunk];
+    // rows are padded to NP = K * REC_LANES numbers and the padding is zero, so the token loop needs no bounds
+    constexpr int NP = K * REC_LANES, TILE = G * C, VECTORS = ROWS ? 3 : 2;
+    const int buffer_floats = VECTORS * chunk * NP + chunk * TILE + 2 * chunk;
     const int h = blockIdx.x, b = blockIdx.y, p0 = blockIdx.z * TILE;
     const int first = cu[b], n = cu[b + 1] - first;
     if (n <= 0) return;
@@ -277,9 +280,10 @@ mamba2_scan_kernel(const float* __restrict__ xbc, int xbc_cols, const float* __r
     const int lane = threadIdx.x % REC_LANES, col = (threadIdx.x / REC_LANES) * C;     // first of this group's columns in the tile
     const int width = min(TILE, P - p0);                        // columns of this tile that exist
     // fixed_decay: the head's decay is a constant and every step size is one (S = decay * S + B x^T, y = S^T C)
+    const bool plain = ROWS || fixed_decay;                      // no step sizes, no skip
     const float fixed = fixed_decay ? __ldg(fixed_decay + h) : 0.0f;
-    const float neg_a = fixed_decay ? 0.0f : -expf(__ldg(a_log + h)), bias = fixed_decay ? 0.0f : __ldg(dt_bias + h);
-    const float skip = fixed_decay ? 0.0f : __ldg(d_skip + h);
+    const float neg_a = plain ? 0.0f : -expf(__ldg(a_log + h)), bias = plain ? 0.0f : __ldg(dt_bias + h);
+    const float skip = plain ? 0.0f : __ldg(d_skip + h);
     const bool vec_x = vec && (width & 3) == 0;
 
     auto stage = [&](int c0, float* base) {                      // asynchronous: B, C and x of tokens c0 .. of this sequence
@@ -287,14 +291,16 @@ mamba2_scan_kernel(const float* __restrict__ xbc, int xbc_cols, const float* __r
         const float* row = xbc + (size_t)(first + c0) * xbc_cols;
         rec_stage(base, NP, row + inner + g * N, xbc_cols, count, N, vec);
         rec_stage(base + chunk * NP, NP, row + inner + groups * N + g * N, xbc_cols, count, N, vec);
-        rec_stage(base + 2 * chunk * NP, TILE, row + h * P + p0, xbc_cols, count, width, vec_x);
+        if (ROWS) rec_stage(base + 2 * chunk * NP, NP, row_decay + ((size_t)(first + c0) * groups + g) * N, (size_t)groups * N, count, N, vec);
+        rec_stage(base + VECTORS * chunk * NP, TILE, row + h * P + p0, xbc_cols, count, width, vec_x);
         rec_commit();
     };
     auto raw_step = [&](int c0) {                                // this thread's token of the chunk: the raw step size
-        if (fixed_decay) return 0.0f;
+        if (plain) return 0.0f;
         return rec_sum_slices(proj + (size_t)(first + c0 + threadIdx.x) * cols + dt_col + h, splits, split_stride);
     };
     auto put_scalars = [&](float* base, float raw) {
+        if (ROWS) return;
         const float dt = fixed_decay ? 1.0f : rec_softplus(raw + bias);
         base[2 * chunk * NP + chunk * TILE + threadIdx.x] = fixed_decay ? fixed : expf(neg_a * dt);
         base[2 * chunk * NP + chunk * TILE + chunk + threadIdx.x] = dt;
@@ -325,14 +331,15 @@ mamba2_scan_kernel(const float* __restrict__ xbc, int xbc_cols, const float* __r
         __syncthreads();
         const float* Bs = cur;
         const float* Cs = cur + chunk * NP;
-        const float* xs = cur + 2 * chunk * NP;
+        const float* xs = cur + VECTORS * chunk * NP;
         const float* decay = xs + chunk * TILE;
         const float* step = decay + chunk;
         for (int k = 0; k < count; ++k) {
-            const float a = decay[k], dt = step[k];
-            float bv[K], cv[K];                                  // all of the token's loads are asked for before the arithmetic
+            const float a = ROWS ? 1.0f : decay[k], dt = ROWS ? 1.0f : step[k];
+            float bv[K], cv[K], av[ROWS ? K : 1];                // all of the token's loads are asked for before the arithmetic
             rec_load_vector<K>(bv, Bs + k * NP, lane);
             rec_load_vector<K>(cv, Cs + k * NP, lane);
+            if constexpr (ROWS) rec_load_vector<K>(av, Cs + (chunk + k) * NP, lane);
             float x[C], part[C];
 #pragma unroll
             for (int c = 0; c < C; ++c) {
@@ -341,9 +348,9 @@ mamba2_scan_kernel(const float* __restrict__ xbc, int xbc_cols, const float* __r
                 float part0 = 0.0f, part1 = 0.0f;                // two chains, so that neighbouring rows do not wait for each other
 #pragma unroll
                 for (int i = 0; i < K; i += 2) {
-                    s[c][i] = fmaf(dx, bv[i], a * s[c][i]);
+                    s[c][i] = fmaf(dx, bv[i], (ROWS ? av[ROWS ? i : 0] : a) * s[c][i]);
                     part0 = fmaf(s[c][i], cv[i], part0);
-                    s[c][i + 1] = fmaf(dx, bv[i + 1], a * s[c][i + 1]);
+                    s[c][i + 1] = fmaf(dx, bv[i + 1], (ROWS ? av[ROWS ? i + 1 : 0] : a) * s[c][i + 1]);
                     part1 = fmaf(s[c][i + 1], cv[i + 1], part1);
                 }
                 part[c] = part0 + part1;
@@ -367,10 +374,14 @@ mamba2_scan_kernel(const float* __restrict__ xbc, int xbc_cols, const float* __r
         if (p0 + col + c < P) rec_store_column<K>(s[c], S + (size_t)c * N, lane, N);
 }
 
-// Tokens staged at a time: 16 where two buffers of them fit the default 48 KB of shared memory, else 8.
+// Tokens staged at a time: 16 where two buffers of them (2 or 3 vectors of a state's rows, a column tile) fit the default 48 KB of shared memory, else 8 or 4.
 static int rec_padded(int rows) { return rows <= 8 * REC_LANES ? 8 * REC_LANES : rows <= 16 * REC_LANES ? 16 * REC_LANES : 32 * REC_LANES; }
-static int rec_chunk(int rows) { return rows <= 128 ? REC_CHUNK : REC_CHUNK / 2; }
-static size_t rec_shared_bytes(int rows, int chunk, int tile) { return (size_t)2 * (2 * chunk * rec_padded(rows) + chunk * tile + 2 * chunk) * sizeof(float); }
+static size_t rec_shared_bytes(int rows, int chunk, int tile, int vectors) { return (size_t)2 * (vectors * chunk * rec_padded(rows) + chunk * tile + 2 * chunk) * sizeof(float); }
+static int rec_chunk(int rows, int tile, int vectors) {
+    int chunk = rows <= 128 ? REC_CHUNK : REC_CHUNK / 2;
+    while (rec_shared_bytes(rows, chunk, tile, vectors) > 48 * 1024) chunk /= 2;
+    return chunk;
+}
 
 constexpr int REC_WIDE_GROUPS = 16, REC_WIDE_COLS = 4;      // the form for grids that fill the GPU: 16 lane groups of 4 columns each
 
@@ -392,16 +403,17 @@ static bool rec_aligned(const void* p, int a, int b, int c, int d) { return (((u
 static int mamba2_scan_launch(const float* xbc, int xbc_cols, const float* proj, int splits, long long split_stride, int cols,
                               int dt_col, const float* dt_bias, const float* a_log, const float* d_skip, float* state, float* y,
                               const int* cu, const int* slots, int sequences, int heads, int P, int N, int groups, int mode,
-                              const float* fixed_decay, cudaStream_t stream) {
+                              const float* fixed_decay, const float* row_decay, cudaStream_t stream) {
     if (sequences <= 0) return 0;
     if (N <= 0 || N > REC_MAX_ROWS || P <= 0 || groups <= 0 || heads % groups || sequences > 65535) return (int)cudaErrorInvalidValue;
-    const int chunk = rec_chunk(N);
-    const int vec = rec_aligned(xbc, xbc_cols, N, P, 0) ? 1 : 0;          // every row piece starts on 16 bytes
+    const int vec = rec_aligned(xbc, xbc_cols, N, P, 0) && ((uintptr_t)row_decay & 15) == 0 ? 1 : 0;          // every row piece starts on 16 bytes
     const bool wide = rec_wide(mode, (long long)heads * sequences * ((P + REC_COLS - 1) / REC_COLS), N);
     const int tile = wide ? REC_WIDE_GROUPS * REC_WIDE_COLS : REC_COLS;
     const dim3 grid(heads, sequences, (P + tile - 1) / tile), block((wide ? REC_WIDE_GROUPS : REC_COLS) * REC_LANES);
-    const size_t shared = rec_shared_bytes(N, chunk, tile);
-#define TT_SCAN(K, G, C) tt_launch_pdl(mamba2_scan_kernel<K, G, C>, grid, block, shared, stream, xbc, xbc_cols, proj, splits, (size_t)split_stride, cols, dt_col, dt_bias, a_log, d_skip, state, y, cu, slots, heads, P, N, groups, chunk, vec, fixed_decay)
+    const int vectors = row_decay ? 3 : 2, chunk = rec_chunk(N, tile, vectors);
+    const size_t shared = rec_shared_bytes(N, chunk, tile, vectors);
+#define TT_SCAN_FORM(K, G, C, ROWS) tt_launch_pdl(mamba2_scan_kernel<K, G, C, ROWS>, grid, block, shared, stream, xbc, xbc_cols, proj, splits, (size_t)split_stride, cols, dt_col, dt_bias, a_log, d_skip, state, y, cu, slots, heads, P, N, groups, chunk, vec, fixed_decay, row_decay)
+#define TT_SCAN(K, G, C) do { if (row_decay) TT_SCAN_FORM(K, G, C, true); else TT_SCAN_FORM(K, G, C, false); } while (0)
     if (wide) {
         if (N <= 8 * REC_LANES) TT_SCAN(8, REC_WIDE_GROUPS, REC_WIDE_COLS);
         else TT_SCAN(16, REC_WIDE_GROUPS, REC_WIDE_COLS);
@@ -411,6 +423,7 @@ static int mamba2_scan_launch(const float* xbc, int xbc_cols, const float* proj,
         else TT_SCAN(32, REC_COLS, 1);
     }
 #undef TT_SCAN
+#undef TT_SCAN_FORM
     TT_LAUNCH_CHECK();
 }
 
@@ -419,7 +432,7 @@ extern "C" int tt_mamba2_scan(const float* xbc, int xbc_cols, const float* proj,
                               const int* cu, const int* slots, int sequences, int heads, int P, int N, int groups, int mode,
                               cudaStream_t stream) {
     return mamba2_scan_launch(xbc, xbc_cols, proj, splits, split_stride, cols, dt_col, dt_bias, a_log, d_skip, state, y, cu, slots,
-                              sequences, heads, P, N, groups, mode, nullptr, stream);
+                              sequences, heads, P, N, groups, mode, nullptr, nullptr, stream);
 }
 
 // ------------------------------------------------------------------------------------
@@ -432,16 +445,25 @@ extern "C" int tt_decay_scan(const float* vkq, int vkq_cols, const float* decay,
                              const int* slots, int sequences, int heads, int V, int D, int mode, cudaStream_t stream) {
     if (!decay) return (int)cudaErrorInvalidValue;
     return mamba2_scan_launch(vkq, vkq_cols, nullptr, 0, 0, 0, 0, nullptr, nullptr, nullptr, state, out, cu, slots, sequences, heads, V, D,
-                              heads, mode, decay, stream);
+                              heads, mode, decay, nullptr, stream);
+}
+
+// The same with decays that a token brings: S_t = diag(a_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t, a_t one number per head and
+// key channel (row_decay: float32 [tokens][heads * D]).
+extern "C" int tt_row_decay_scan(const float* vkq, int vkq_cols, const float* row_decay, float* state, float* out, const int* cu,
+                                 const int* slots, int sequences, int heads, int V, int D, int mode, cudaStream_t stream) {
+    if (!row_decay) return (int)cudaErrorInvalidValue;
+    return mamba2_scan_launch(vkq, vkq_cols, nullptr, 0, 0, 0, 0, nullptr, nullptr, nullptr, state, out, cu, slots, sequences, heads, V, D,
+                              heads, mode, nullptr, row_decay, stream);
 }
 
 // q, k and v of a linear attention from the partial sums of its input projection (columns [q | k | v | ...], q and k
 // heads x D, v heads x V), as the scan reads them: [v | k | q].  activation != 0: silu on all three.  rotary_dim > 0:
 // the first rotary_dim numbers of each head of q and k are rotated by the token's position (number i pairs with
-// i + rotary_dim / 2, angle = position * inv_freq[i], float32).  k is multiplied by k_scale after the rotation.
+// i + rotary_dim / 2, angle = position * inv_freq[i], float32).  q and k are multiplied by q_scale and k_scale after the rotation.
 __global__ void linear_attention_prepare_kernel(const float* __restrict__ proj, int splits, size_t split_stride, int cols, int heads,
                                                 int D, int V, int activation, const float* __restrict__ inv_freq, int rotary_dim,
-                                                float k_scale, float* __restrict__ vkq, const int* __restrict__ cu,
+                                                float q_scale, float k_scale, float* __restrict__ vkq, const int* __restrict__ cu,
                                                 const int* __restrict__ len_before, int sequences) {
     tt_pdl_launch_dependents();
     const int t = blockIdx.x;
@@ -473,12 +495,12 @@ __global__ void linear_attention_prepare_kernel(const float* __restrict__ proj, 
             x = i < half ? x * cs - other * sn : x * cs + other * sn;
         }
         if (is_k) out[hv + (j - qk)] = x * k_scale;
-        else out[hv + qk + j] = x;
+        else out[hv + qk + j] = x * q_scale;
     }
 }
 
 extern "C" int tt_linear_attention_prepare(const float* proj, int splits, long long split_stride, int cols, int heads, int D, int V,
-                                           int activation, const float* inv_freq, int rotary_dim, float k_scale, float* vkq,
+                                           int activation, const float* inv_freq, int rotary_dim, float q_scale, float k_scale, float* vkq,
                                            const int* cu, const int* len_before, int sequences, int n_tokens, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (rotary_dim < 0 || rotary_dim > D || (rotary_dim & 1) || 2 * heads * D + heads * V > cols) return (int)cudaErrorInvalidValue;
@@ -486,7 +508,7 @@ extern "C" int tt_linear_attention_prepare(const float* proj, int splits, long l
     const int want = n_tokens >= 1024 ? (total + 1023) / 1024 : (total + 255) / 256;                // few tokens: a token's columns over more blocks
     const int tiles = want < 32 ? want : 32;
     tt_launch_pdl(linear_attention_prepare_kernel, dim3(n_tokens, tiles), dim3(256), 0, stream, proj, splits, (size_t)split_stride, cols, heads, D,
-                  V, activation, inv_freq, rotary_dim, k_scale, vkq, cu, len_before, sequences);
+                  V, activation, inv_freq, rotary_dim, q_scale, k_scale, vkq, cu, len_before, sequences);
     TT_LAUNCH_CHECK();
 }
 
@@ -497,20 +519,22 @@ extern "C" int tt_linear_attention_prepare(const float* proj, int splits, long l
 //   S = decay * S;  u = beta * (v - S^T k);  S = S + k u^T;  o[t, h] = S^T q
 // qkv: float32 [tokens][2 * qk_heads * D + heads * V] (q, k, v: the convolutions' output); b_raw and
 // a_raw: columns b_col + h and a_col + h of the projection's partial sums; state: [slots][heads][V][D].
+// ROWS: a token's decay is a number for every state row (row_decay, float32 [tokens][heads * D], made beforehand), and the
+// state's rows are multiplied by it one by one.
 // ------------------------------------------------------------------------------------
-template <int K, int G, int C>
+template <int K, int G, int C, bool ROWS>
 __global__ void __launch_bounds__(G* REC_LANES)
 delta_scan_kernel(const float* __restrict__ qkv, int qkv_cols, const float* __restrict__ proj, int splits, size_t split_stride,
                   int cols, int b_col, int a_col, const float* __restrict__ dt_bias, const float* __restrict__ a_log,
                   float* __restrict__ state, float* __restrict__ o, const int* __restrict__ cu, const int* __restrict__ slots,
-                  int heads, int qk_heads, int D, int V, int chunk, int vec) {
+                  int heads, int qk_heads, int D, int V, int chunk, int vec, const float* __restrict__ row_decay) {
     tt_pdl_launch_dependents();
     tt_pdl_wait();
     extern __shared__ __align__(16) float rec_shared[];
-    // two buffers of: q [chunk][DP], k [chunk][DP], v [chunk][TILE], decay [chunk], beta [chunk]; rows are padded to
-    // DP = K * REC_LANES numbers and the padding is zero.  G lane groups of C neighbouring columns each, as in the kernel above.
-    constexpr int DP = K * REC_LANES, TILE = G * C;
-    const int buffer_floats = 2 * chunk * DP + chunk * TILE + 2 * chunk;
+    // two buffers of: q [chunk][DP], k [chunk][DP], (ROWS) decays [chunk][DP], v [chunk][TILE], decay [chunk], beta [chunk]; rows
+    // are padded to DP = K * REC_LANES numbers and the padding is zero.  G lane groups of C neighbouring columns each, as above.
+    constexpr int DP = K * REC_LANES, TILE = G * C, VECTORS = ROWS ? 3 : 2;
+    const int buffer_floats = VECTORS * chunk * DP + chunk * TILE + 2 * chunk;
     const int h = blockIdx.x, b = blockIdx.y, p0 = blockIdx.z * TILE;
     const int first = cu[b], n = cu[b + 1] - first;
     if (n <= 0) return;
@@ -518,7 +542,7 @@ delta_scan_kernel(const float* __restrict__ qkv, int qkv_cols, const float* __re
     const int lane = threadIdx.x % REC_LANES, col = (threadIdx.x / REC_LANES) * C;
     const int warp = threadIdx.x >> 5, wlane = threadIdx.x & 31, warps = blockDim.x >> 5;
     const int width = min(TILE, V - p0);
-    const float neg_a = -expf(__ldg(a_log + h)), bias = __ldg(dt_bias + h), q_scale = rsqrtf((float)D);
+    const float neg_a = ROWS ? 0.0f : -expf(__ldg(a_log + h)), bias = ROWS ? 0.0f : __ldg(dt_bias + h), q_scale = rsqrtf((float)D);
     const int k_off = qk_heads * D, v_off = 2 * qk_heads * D;
     const bool vec_v = vec && (width & 3) == 0;
 
@@ -527,16 +551,17 @@ delta_scan_kernel(const float* __restrict__ qkv, int qkv_cols, const float* __re
         const float* row = qkv + (size_t)(first + c0) * qkv_cols;
         rec_stage(base, DP, row + g * D, qkv_cols, count, D, vec);
         rec_stage(base + chunk * DP, DP, row + k_off + g * D, qkv_cols, count, D, vec);
-        rec_stage(base + 2 * chunk * DP, TILE, row + v_off + h * V + p0, qkv_cols, count, width, vec_v);
+        if (ROWS) rec_stage(base + 2 * chunk * DP, DP, row_decay + ((size_t)(first + c0) * heads + h) * D, (size_t)heads * D, count, D, vec);
+        rec_stage(base + VECTORS * chunk * DP, TILE, row + v_off + h * V + p0, qkv_cols, count, width, vec_v);
         rec_commit();
     };
     auto raw_pair = [&](int c0) {                                // this thread's token of the chunk: raw write strength, raw decay input
         const float* row = proj + (size_t)(first + c0 + threadIdx.x) * cols;
-        return make_float2(rec_sum_slices(row + b_col + h, splits, split_stride), rec_sum_slices(row + a_col + h, splits, split_stride));
+        return make_float2(rec_sum_slices(row + b_col + h, splits, split_stride), ROWS ? 0.0f : rec_sum_slices(row + a_col + h, splits, split_stride));
     };
     auto put_scalars = [&](float* base, float2 raw) {
-        base[2 * chunk * DP + chunk * TILE + threadIdx.x] = expf(neg_a * rec_softplus(raw.y + bias));
-        base[2 * chunk * DP + chunk * TILE + chunk + threadIdx.x] = 1.0f / (1.0f + expf(-raw.x));
+        if (!ROWS) base[2 * chunk * DP + chunk * TILE + threadIdx.x] = expf(neg_a * rec_softplus(raw.y + bias));
+        base[VECTORS * chunk * DP + chunk * TILE + chunk + threadIdx.x] = 1.0f / (1.0f + expf(-raw.x));
     };
 
     for (int e = threadIdx.x; e < 2 * buffer_floats; e += blockDim.x) rec_shared[e] = 0.0f;
@@ -573,23 +598,24 @@ delta_scan_kernel(const float* __restrict__ qkv, int qkv_cols, const float* __re
             for (int r = wlane; r < D; r += 32) vecp[r] *= scale;
         }
         __syncthreads();
-        const float* vs = cur + 2 * chunk * DP;
+        const float* vs = cur + VECTORS * chunk * DP;
         const float* decay = vs + chunk * TILE;
         const float* beta = decay + chunk;
         for (int k = 0; k < count; ++k) {
-            const float a = decay[k], write = beta[k];
-            float kv[K], qv[K];                                  // all of the token's loads are asked for before the arithmetic
+            const float a = ROWS ? 1.0f : decay[k], write = beta[k];
+            float kv[K], qv[K], av[ROWS ? K : 1];                // all of the token's loads are asked for before the arithmetic
             rec_load_vector<K>(kv, ks + k * DP, lane);
             rec_load_vector<K>(qv, qs + k * DP, lane);
+            if constexpr (ROWS) rec_load_vector<K>(av, ks + (chunk + k) * DP, lane);
             float part[C];
 #pragma unroll
             for (int c = 0; c < C; ++c) {
                 float part0 = 0.0f, part1 = 0.0f;
 #pragma unroll
                 for (int i = 0; i < K; i += 2) {
-                    s[c][i] *= a;
+                    s[c][i] *= ROWS ? av[ROWS ? i : 0] : a;
                     part0 = fmaf(s[c][i], kv[i], part0);
-                    s[c][i + 1] *= a;
+                    s[c][i + 1] *= ROWS ? av[ROWS ? i + 1 : 0] : a;
                     part1 = fmaf(s[c][i + 1], kv[i + 1], part1);
                 }
                 part[c] = part0 + part1;
@@ -631,19 +657,21 @@ delta_scan_kernel(const float* __restrict__ qkv, int qkv_cols, const float* __re
         if (p0 + col + c < V) rec_store_column<K>(s[c], S + (size_t)c * D, lane, D);
 }
 
+// row_decay: the decays of the ROWS form (a_col, dt_bias and a_log are then not read), or null
 extern "C" int tt_delta_scan(const float* qkv, int qkv_cols, const float* proj, int splits, long long split_stride, int cols,
-                             int b_col, int a_col, const float* dt_bias, const float* a_log, float* state, float* o,
+                             int b_col, int a_col, const float* dt_bias, const float* a_log, const float* row_decay, float* state, float* o,
                              const int* cu, const int* slots, int sequences, int heads, int qk_heads, int D, int V, int mode,
                              cudaStream_t stream) {
     if (sequences <= 0) return 0;
     if (D <= 0 || D > REC_MAX_ROWS || V <= 0 || qk_heads <= 0 || heads % qk_heads || sequences > 65535) return (int)cudaErrorInvalidValue;
-    const int chunk = rec_chunk(D);
-    const int vec = rec_aligned(qkv, qkv_cols, D, V, 0) ? 1 : 0;
+    const int vec = rec_aligned(qkv, qkv_cols, D, V, 0) && ((uintptr_t)row_decay & 15) == 0 ? 1 : 0;
     const bool wide = rec_wide(mode, (long long)heads * sequences * ((V + REC_COLS - 1) / REC_COLS), D);
     const int tile = wide ? REC_WIDE_GROUPS * REC_WIDE_COLS : REC_COLS;
     const dim3 grid(heads, sequences, (V + tile - 1) / tile), block((wide ? REC_WIDE_GROUPS : REC_COLS) * REC_LANES);
-    const size_t shared = rec_shared_bytes(D, chunk, tile);
-#define TT_SCAN(K, G, C) tt_launch_pdl(delta_scan_kernel<K, G, C>, grid, block, shared, stream, qkv, qkv_cols, proj, splits, (size_t)split_stride, cols, b_col, a_col, dt_bias, a_log, state, o, cu, slots, heads, qk_heads, D, V, chunk, vec)
+    const int vectors = row_decay ? 3 : 2, chunk = rec_chunk(D, tile, vectors);
+    const size_t shared = rec_shared_bytes(D, chunk, tile, vectors);
+#define TT_SCAN_FORM(K, G, C, ROWS) tt_launch_pdl(delta_scan_kernel<K, G, C, ROWS>, grid, block, shared, stream, qkv, qkv_cols, proj, splits, (size_t)split_stride, cols, b_col, a_col, dt_bias, a_log, state, o, cu, slots, heads, qk_heads, D, V, chunk, vec, row_decay)
+#define TT_SCAN(K, G, C) do { if (row_decay) TT_SCAN_FORM(K, G, C, true); else TT_SCAN_FORM(K, G, C, false); } while (0)
     if (wide) {
         if (D <= 8 * REC_LANES) TT_SCAN(8, REC_WIDE_GROUPS, REC_WIDE_COLS);
         else TT_SCAN(16, REC_WIDE_GROUPS, REC_WIDE_COLS);
@@ -653,6 +681,131 @@ extern "C" int tt_delta_scan(const float* qkv, int qkv_cols, const float* proj, 
         else TT_SCAN(32, REC_COLS, 1);
     }
 #undef TT_SCAN
+#undef TT_SCAN_FORM
+    TT_LAUNCH_CHECK();
+}
+
+// ------------------------------------------------------------------------------------
+// Products of low rank: z[t, j] = sum_r W[j, r] * x[t, r] with x the columns x_col .. x_col + rank - 1 of a projection's
+// partial sums, and what is made of z at once (kind):
+//   0: z      1: exp(-exp(a_log[h]) * softplus(z + bias[j])), h = j / per_head      2: sigmoid(z + bias[j]) ^ inv_tau
+// Up to two such products of one projection in one launch (blockIdx.z).  All float32; W is stored [rank][n] (transposed, so
+// that neighbouring threads read neighbouring numbers) in either element type.  A thread owns two neighbouring columns of TT
+// tokens; with few tokens RG thread groups share the rank among themselves and add up in shared memory.
+// ------------------------------------------------------------------------------------
+struct LowRankPart {
+    int x_col, rank, n, kind, per_head;
+    const void* w;
+    const float* bias;
+    const float* a_log;
+    float inv_tau;
+    float* out;                 // float32 [tokens][n]
+};
+struct LowRankParts { LowRankPart part[2]; };
+constexpr int LR_THREADS = 128, LR_RANKS = 128;       // ranks staged at a time
+
+__device__ __forceinline__ float low_rank_finish(const LowRankPart& p, float z, int j) {
+    if (p.kind == 1) return expf(-expf(__ldg(p.a_log + j / p.per_head)) * rec_softplus(z + __ldg(p.bias + j)));
+    if (p.kind == 2) return expf(-rec_softplus(-(z + __ldg(p.bias + j))) * p.inv_tau);
+    return z;
+}
+
+template <typename TW, int TT, int RG>
+__global__ void __launch_bounds__(LR_THREADS)
+low_rank_kernel(const float* __restrict__ proj, int splits, size_t split_stride, int cols, const LowRankParts parts, int n_tokens) {
+    constexpr int LANES = LR_THREADS / RG, STRIDE = TT + 4;          // rows padded: 16-byte reads, few bank conflicts on the writes
+    __shared__ __align__(16) float xs[LR_RANKS * STRIDE];
+    __shared__ float sums[RG > 1 ? (RG - 1) * TT * 2 * LANES : 1];
+    tt_pdl_launch_dependents();
+    const LowRankPart p = blockIdx.z ? parts.part[1] : parts.part[0];
+    const int j0 = blockIdx.y * 2 * LANES;
+    if (j0 >= p.n) return;
+    const int t0 = blockIdx.x * TT, count = min(TT, n_tokens - t0);
+    const int group = threadIdx.x / LANES, lane = threadIdx.x - group * LANES;
+    const int j = j0 + 2 * lane;
+    const TW* w = reinterpret_cast<const TW*>(p.w);
+    float acc[TT][2];
+#pragma unroll
+    for (int t = 0; t < TT; ++t) acc[t][0] = acc[t][1] = 0.0f;
+    tt_pdl_wait();
+    for (int r0 = 0; r0 < p.rank; r0 += LR_RANKS) {
+        const int ranks = min(LR_RANKS, p.rank - r0);
+        if (r0) __syncthreads();
+        for (int e = threadIdx.x; e < TT * ranks; e += LR_THREADS) {
+            const int t = e / ranks, r = e - t * ranks;
+            xs[r * STRIDE + t] = t < count ? rec_sum_slices(proj + (size_t)(t0 + t) * cols + p.x_col + r0 + r, splits, split_stride) : 0.0f;
+        }
+        __syncthreads();
+#pragma unroll 4
+        for (int r = group; r < ranks; r += RG) {
+            const size_t at = (size_t)(r0 + r) * p.n + j;
+            const float w0 = j < p.n ? tt_to_float(w[at]) : 0.0f, w1 = j + 1 < p.n ? tt_to_float(w[at + 1]) : 0.0f;
+            const float4* x4 = reinterpret_cast<const float4*>(xs + r * STRIDE);
+#pragma unroll
+            for (int q = 0; q < TT / 4; ++q) {
+                const float4 x = x4[q];
+                acc[4 * q][0] = fmaf(x.x, w0, acc[4 * q][0]);         acc[4 * q][1] = fmaf(x.x, w1, acc[4 * q][1]);
+                acc[4 * q + 1][0] = fmaf(x.y, w0, acc[4 * q + 1][0]); acc[4 * q + 1][1] = fmaf(x.y, w1, acc[4 * q + 1][1]);
+                acc[4 * q + 2][0] = fmaf(x.z, w0, acc[4 * q + 2][0]); acc[4 * q + 2][1] = fmaf(x.z, w1, acc[4 * q + 2][1]);
+                acc[4 * q + 3][0] = fmaf(x.w, w0, acc[4 * q + 3][0]); acc[4 * q + 3][1] = fmaf(x.w, w1, acc[4 * q + 3][1]);
+            }
+        }
+    }
+    if constexpr (RG > 1) {
+        if (group > 0) {
+#pragma unroll
+            for (int t = 0; t < TT; ++t)
+#pragma unroll
+                for (int c = 0; c < 2; ++c) sums[(((group - 1) * TT + t) * 2 + c) * LANES + lane] = acc[t][c];
+        }
+        __syncthreads();
+        if (group > 0) return;
+#pragma unroll
+        for (int g = 0; g < RG - 1; ++g)
+#pragma unroll
+            for (int t = 0; t < TT; ++t)
+#pragma unroll
+                for (int c = 0; c < 2; ++c) acc[t][c] += sums[((g * TT + t) * 2 + c) * LANES + lane];
+    }
+#pragma unroll
+    for (int t = 0; t < TT; ++t) {
+        if (t >= count) break;
+        float* o = p.out + (size_t)(t0 + t) * p.n + j;
+        const float a = j < p.n ? low_rank_finish(p, acc[t][0], j) : 0.0f, b = j + 1 < p.n ? low_rank_finish(p, acc[t][1], j + 1) : 0.0f;
+        if (j + 1 < p.n && !(p.n & 1)) *reinterpret_cast<float2*>(o) = make_float2(a, b);
+        else {
+            if (j < p.n) o[0] = a;
+            if (j + 1 < p.n) o[1] = b;
+        }
+    }
+}
+
+constexpr int LR_FEW_TOKENS = 256;      // up to here the rank is shared among thread groups
+
+extern "C" int tt_low_rank(const float* proj, int splits, long long split_stride, int cols, int n_parts, int w_dtype,
+                           int x_col0, int rank0, int n0, int kind0, int per_head0, const void* w0, const float* bias0, const float* a_log0, float inv_tau0, float* out0,
+                           int x_col1, int rank1, int n1, int kind1, int per_head1, const void* w1, const float* bias1, const float* a_log1, float inv_tau1, float* out1,
+                           int n_tokens, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (n_parts < 1 || n_parts > 2) return (int)cudaErrorInvalidValue;
+    LowRankParts parts;
+    parts.part[0] = LowRankPart{x_col0, rank0, n0, kind0, per_head0, w0, bias0, a_log0, inv_tau0, out0};
+    parts.part[1] = n_parts > 1 ? LowRankPart{x_col1, rank1, n1, kind1, per_head1, w1, bias1, a_log1, inv_tau1, out1} : parts.part[0];
+    int widest = 0;
+    for (int i = 0; i < n_parts; ++i) {
+        const LowRankPart& p = parts.part[i];
+        if (p.rank < 1 || p.n < 1 || p.x_col < 0 || p.x_col + p.rank > cols || p.kind < 0 || p.kind > 2) return (int)cudaErrorInvalidValue;
+        if ((p.kind && !p.bias) || (p.kind == 1 && (!p.a_log || p.per_head < 1)) || ((uintptr_t)p.out & 7)) return (int)cudaErrorInvalidValue;
+        widest = p.n > widest ? p.n : widest;
+    }
+    const bool few = n_tokens <= LR_FEW_TOKENS;
+    const int tile = few ? 8 : 32, columns = 2 * LR_THREADS / (few ? 4 : 1);
+    const dim3 grid((n_tokens + tile - 1) / tile, (widest + columns - 1) / columns, n_parts);
+    if (grid.y > 65535) return (int)cudaErrorInvalidValue;
+#define TT_LOW_RANK(T, TT, RG) tt_launch_pdl(low_rank_kernel<T, TT, RG>, grid, dim3(LR_THREADS), 0, stream, proj, splits, (size_t)split_stride, cols, parts, n_tokens)
+    if (w_dtype == TT_F32) { if (few) TT_LOW_RANK(float, 8, 4); else TT_LOW_RANK(float, 32, 1); }
+    else { if (few) TT_LOW_RANK(__nv_bfloat16, 8, 4); else TT_LOW_RANK(__nv_bfloat16, 32, 1); }
+#undef TT_LOW_RANK
     TT_LAUNCH_CHECK();
 }
 

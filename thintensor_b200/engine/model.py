@@ -9,7 +9,7 @@ execution plan.
 """
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, replace
 
 import torch
 
@@ -168,9 +168,15 @@ class DecoderModel:
             raise RuntimeError("the model has no weights yet")
         residual = ctx.scratch("model.residual", (ctx.n_tokens, self.spec.hidden_size), torch.float32)
         self.embedding.part.forward(ctx, ctx.tokens, residual, None if self.embedding_entry is None else cache.run_state(self.embedding_entry))
+        embedded = None
+        if any(run.add_embedding for run in self.spec.schedule):          # kept for the runs that start by adding it
+            embedded = ctx.scratch("model.embedded", (ctx.n_tokens, self.spec.hidden_size), torch.float32)
+            embedded.copy_(residual)
         pending: Delta | None = None
         for index, run in enumerate(self.spec.schedule):
             users = self.users[index]
+            if run.add_embedding:
+                pending = replace(pending or Delta(None), addend=embedded)
             pending = self.layers[run.layer].run(ctx, residual, pending, [self._run_cache(cache, u) for u in users], [cache.run_state(u) for u in users])
         if rows is None:
             return None

@@ -9,6 +9,7 @@ from __future__ import annotations
 
 import ctypes
 from ctypes import c_float, c_int, c_longlong, c_ulonglong, c_void_p
+from dataclasses import dataclass
 
 import torch
 
@@ -303,6 +304,42 @@ def add_layernorm(residual: torch.Tensor, delta: torch.Tensor | None, weight: to
     _check(fn(_ptr(residual), _ptr(delta), splits, stride, _ptr(weight), _ptr(bias), eps, _ptr(out), dtype_code(out.dtype), _ptr(rows), n_rows, hidden, _stream()), "add_layernorm")
 
 
+def add_norms(residual: torch.Tensor, a: torch.Tensor | None, b: torch.Tensor | None, scale: float, addend: torch.Tensor | None,
+              weight: torch.Tensor, bias: torch.Tensor | None, out: torch.Tensor, eps: float, centered: bool, weight_offset: float = 0.0,
+              second: tuple[torch.Tensor, torch.Tensor | None, torch.Tensor] | None = None, rows: torch.Tensor | None = None) -> None:
+    """residual += scale * (sum(a) + sum(b)) + addend (``a`` and ``b`` are summed over their first axis; each of the three may
+    be None); out = norm(residual) * (weight + weight_offset) (+ bias), with the root mean square norm or (``centered``) the
+    layer norm.  ``second`` = (weight, bias or None, out) of another norm of the same kind and eps over the same rows.
+    ``rows`` as for :func:`add_rmsnorm`."""
+    _need(residual, torch.float32, "residual")
+    hidden = residual.shape[-1]
+    norms = [(weight, bias, out)] + ([second] if second is not None else [])
+    for w, shift, o in norms:
+        _need(w, torch.float32, "norm weight")
+        if shift is not None:
+            _need(shift, torch.float32, "norm bias")
+        if not o.is_contiguous() or o.dtype != out.dtype or o.shape != out.shape:
+            raise KernelError("norm outputs must be contiguous and alike")
+    for branch in (a, b):
+        if branch is not None:
+            _need(branch, torch.float32, "branch")
+            if tuple(branch.shape[1:]) != tuple(residual.shape):
+                raise KernelError(f"a branch is [slices, {residual.shape[0]}, {hidden}], got {tuple(branch.shape)}")
+    if addend is not None:
+        _need(addend, torch.float32, "addend")
+        if addend.shape != residual.shape:
+            raise KernelError("the addend must have the stream's shape")
+    if rows is not None:
+        _need(rows, torch.int32, "rows")
+    n_rows = rows.numel() if rows is not None else residual.shape[0]
+    size = lambda t: (_ptr(t), 0 if t is None else t.shape[0], 0 if t is None else t.stride(0))
+    w2, b2, o2 = second if second is not None else (None, None, None)
+    fn = _fn("elementwise", "tt_add_norms", [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_int, c_longlong, c_float, c_void_p, c_void_p, c_void_p,
+                                             c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float, c_int, c_int, c_void_p, c_int, c_int, c_void_p])
+    _check(fn(_ptr(residual), *size(a), *size(b), scale, _ptr(addend), _ptr(weight), _ptr(bias), _ptr(out), _ptr(w2), _ptr(b2), _ptr(o2),
+              weight_offset, eps, 1 if centered else 0, dtype_code(out.dtype), _ptr(rows), n_rows, hidden, _stream()), "add_norms")
+
+
 def qk_norm_rope_append(proj: torch.Tensor, q_norm: torch.Tensor | None, k_norm: torch.Tensor | None, norm_eps: float,
                         inv_freq: torch.Tensor, rotary_dim: int, interleaved: bool, attention_scaling: float, q_out: torch.Tensor,
                         k_pool: torch.Tensor | None, v_pool: torch.Tensor | None, table: torch.Tensor, cu: torch.Tensor,
@@ -462,7 +499,8 @@ def attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, table
     ``softcap * tanh(s / softcap)``.  ``slopes`` (float32, one per query head): ``slope_h * (i - j)`` is taken off the score of
     query position i and key position j.  ``gate``: float32 partial sums ``[slices, tokens, heads * value_dim]`` (with
     ``gate_per_head``: ``[slices, tokens, heads]``), possibly a range of a wider projection's columns; the output is
-    multiplied by their sigmoid."""
+    multiplied by their sigmoid.  ``window``, here and in the other attention entry points: 0: a position sees every key up to
+    its own; n > 0: the last n of them; -n: those of its own chunk, chunks of n positions counted from the sequence's start."""
     check_head_dim(head_dim)
     value_dim = head_dim if value_dim is None else int(value_dim)
     check_head_dim(value_dim)
@@ -778,23 +816,29 @@ def mamba2_scan(xbc: torch.Tensor, proj: torch.Tensor, dt_col: int, dt_bias: tor
               _ptr(cu), _ptr(slots), sequences, heads, head_dim, state_size, groups, SCAN_FORMS[form], _stream()), "mamba2_scan")
 
 
-def delta_scan(qkv: torch.Tensor, proj: torch.Tensor, b_col: int, a_col: int, dt_bias: torch.Tensor, a_log: torch.Tensor,
+def delta_scan(qkv: torch.Tensor, proj: torch.Tensor, b_col: int, a_col: int, dt_bias: torch.Tensor | None, a_log: torch.Tensor | None,
                state: torch.Tensor, out: torch.Tensor, cu: torch.Tensor, slots: torch.Tensor, sequences: int, heads: int, qk_heads: int,
-               key_dim: int, value_dim: int, form: str = "auto") -> None:
+               key_dim: int, value_dim: int, form: str = "auto", row_decay: torch.Tensor | None = None) -> None:
     """The gated delta rule over each sequence's tokens.  ``qkv`` float32 [tokens, 2 * qk_heads * key_dim + heads *
     value_dim] holds q, k, v (q and k are made unit vectors here, q also times key_dim^-1/2); columns ``b_col + h`` and
     ``a_col + h`` of ``proj`` the raw write strength and decay input of head h; ``state`` float32
     [slots, heads, value_dim, key_dim]; ``out`` float32 [tokens, heads * value_dim] receives S^T q.  ``form``: as for
-    :func:`mamba2_scan`."""
-    for t, name in ((qkv, "q/k/v"), (dt_bias, "dt_bias"), (a_log, "A_log"), (state, "recurrent state"), (out, "recurrence output")):
-        _need(t, torch.float32, name)
+    :func:`mamba2_scan`.  ``row_decay`` (float32 [tokens, heads * key_dim]): a decay for every key channel instead of the head's
+    own; ``a_col``, ``dt_bias`` and ``a_log`` are then not used."""
+    for t, name in ((qkv, "q/k/v"), (dt_bias, "dt_bias"), (a_log, "A_log"), (row_decay, "decays"), (state, "recurrent state"), (out, "recurrence output")):
+        if t is not None:
+            _need(t, torch.float32, name)
+    if row_decay is None and (dt_bias is None or a_log is None):
+        raise KernelError("delta_scan: a decay per head needs dt_bias and A_log")
+    if row_decay is not None and tuple(row_decay.shape) != (qkv.shape[0], heads * key_dim):
+        raise KernelError("delta_scan: the decays do not fit the sizes")
     if (qkv.shape[1] != 2 * qk_heads * key_dim + heads * value_dim or tuple(state.shape[1:]) != (heads, value_dim, key_dim)
             or out.shape[1] != heads * value_dim):
         raise KernelError("delta_scan: shapes do not fit the sizes")
     p, splits, stride, cols = _projection(proj)
-    fn = _fn("recurrent", "tt_delta_scan", [c_void_p, c_int, c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
+    fn = _fn("recurrent", "tt_delta_scan", [c_void_p, c_int, c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                                             c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
-    _check(fn(_ptr(qkv), qkv.shape[1], p, splits, stride, cols, b_col, a_col, _ptr(dt_bias), _ptr(a_log), _ptr(state), _ptr(out),
+    _check(fn(_ptr(qkv), qkv.shape[1], p, splits, stride, cols, b_col, a_col, _ptr(dt_bias), _ptr(a_log), _ptr(row_decay), _ptr(state), _ptr(out),
               _ptr(cu), _ptr(slots), sequences, heads, qk_heads, key_dim, value_dim, SCAN_FORMS[form], _stream()), "delta_scan")
 
 
@@ -825,11 +869,11 @@ def gated_group_norm(y: torch.Tensor, group: int, proj: torch.Tensor, gate_col: 
 
 def linear_attention_prepare(proj: torch.Tensor, heads: int, key_dim: int, value_dim: int, activation: bool, inv_freq: torch.Tensor | None,
                              rotary_dim: int, k_scale: float, vkq: torch.Tensor, cu: torch.Tensor, len_before: torch.Tensor,
-                             sequences: int, n_tokens: int) -> None:
+                             sequences: int, n_tokens: int, q_scale: float = 1.0) -> None:
     """q, k and v of a linear attention from the partial sums of its input projection (columns ``[q | k | v | ...]``) as
     :func:`decay_scan` reads them, ``vkq`` float32 ``[tokens, heads * value_dim + 2 * heads * key_dim]``: silu on all three
-    (``activation``), the first ``rotary_dim`` numbers of each head of q and k rotated by the position (halves paired), k times
-    ``k_scale``."""
+    (``activation``), the first ``rotary_dim`` numbers of each head of q and k rotated by the position (halves paired), q times
+    ``q_scale`` and k times ``k_scale``."""
     _need(vkq, torch.float32, "v/k/q")
     if tuple(vkq.shape) != (n_tokens, heads * value_dim + 2 * heads * key_dim):
         raise KernelError("linear_attention_prepare: the output does not fit the sizes")
@@ -839,9 +883,9 @@ def linear_attention_prepare(proj: torch.Tensor, heads: int, key_dim: int, value
             raise KernelError("linear_attention_prepare: too few inverse frequencies")
     p, splits, stride, cols = _projection(proj)
     fn = _fn("recurrent", "tt_linear_attention_prepare", [c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
-                                                          c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p])
+                                                          c_float, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p])
     _check(fn(p, splits, stride, cols, heads, key_dim, value_dim, 1 if activation else 0, _ptr(inv_freq) if rotary_dim else c_void_p(0),
-              rotary_dim, k_scale, _ptr(vkq), _ptr(cu), _ptr(len_before), sequences, n_tokens, _stream()), "linear_attention_prepare")
+              rotary_dim, q_scale, k_scale, _ptr(vkq), _ptr(cu), _ptr(len_before), sequences, n_tokens, _stream()), "linear_attention_prepare")
 
 
 def decay_scan(vkq: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, out: torch.Tensor, cu: torch.Tensor, slots: torch.Tensor,
@@ -859,6 +903,64 @@ def decay_scan(vkq: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, out:
                                             c_int, c_void_p])
     _check(fn(_ptr(vkq), vkq.shape[1], _ptr(decay), _ptr(state), _ptr(out), _ptr(cu), _ptr(slots), sequences, heads, value_dim, key_dim,
               SCAN_FORMS[form], _stream()), "decay_scan")
+
+
+def row_decay_scan(vkq: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, out: torch.Tensor, cu: torch.Tensor, slots: torch.Tensor,
+                   sequences: int, heads: int, key_dim: int, value_dim: int, form: str = "auto") -> None:
+    """:func:`decay_scan` with decays that every token brings for every head and key channel: ``S = diag(a_t) S + k v^T``,
+    ``o = S^T q``, ``decay`` float32 ``[tokens, heads * key_dim]``."""
+    for t, name in ((vkq, "v/k/q"), (decay, "decays"), (state, "recurrent state"), (out, "recurrence output")):
+        _need(t, torch.float32, name)
+    if (vkq.shape[1] != heads * value_dim + 2 * heads * key_dim or tuple(state.shape[1:]) != (heads, value_dim, key_dim)
+            or out.shape[1] != heads * value_dim or tuple(decay.shape) != (vkq.shape[0], heads * key_dim)):
+        raise KernelError("row_decay_scan: shapes do not fit the sizes")
+    fn = _fn("recurrent", "tt_row_decay_scan", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                                                c_int, c_void_p])
+    _check(fn(_ptr(vkq), vkq.shape[1], _ptr(decay), _ptr(state), _ptr(out), _ptr(cu), _ptr(slots), sequences, heads, value_dim, key_dim,
+              SCAN_FORMS[form], _stream()), "row_decay_scan")
+
+
+@dataclass(frozen=True)
+class LowRank:
+    """One product of :func:`low_rank`: ``z = W x`` with x the ``rank`` columns of a projection from ``col`` on and ``weight`` the
+    transposed matrix, ``[rank, n]``.  ``kind``: ``plain`` (z), ``delta_decay`` (``exp(-exp(a_log_h) * softplus(z + bias))``, h the
+    head of ``per_head`` neighbouring columns) or ``sigmoid_root`` (``sigmoid(z + bias) ** (1 / tau)``)."""
+
+    col: int
+    weight: torch.Tensor
+    out: torch.Tensor               # float32 [tokens, n]
+    kind: str = "plain"
+    bias: torch.Tensor | None = None
+    a_log: torch.Tensor | None = None
+    per_head: int = 1
+    tau: float = 1.0
+
+
+LOW_RANK_KINDS = {"plain": 0, "delta_decay": 1, "sigmoid_root": 2}
+
+
+def low_rank(proj: torch.Tensor, products: list[LowRank]) -> None:
+    """One or two products of low rank on columns of the same projection (float32 partial sums), in float32."""
+    if not 1 <= len(products) <= 2 or len({p.weight.dtype for p in products}) != 1:
+        raise KernelError("low_rank takes one or two products with weights of one dtype")
+    ptr, splits, stride, cols = _projection(proj)
+    tokens, args = proj.shape[1], []
+    for p in products:
+        rank, n = p.weight.shape
+        _need(p.out, torch.float32, "low-rank product")
+        if not p.weight.is_contiguous() or tuple(p.out.shape) != (tokens, n) or p.col < 0 or p.col + rank > cols:
+            raise KernelError("low_rank: shapes do not fit")
+        for t, count, name in ((p.bias, n, "bias"), (p.a_log, -(-n // p.per_head), "A_log")):
+            if t is not None:
+                _need(t, torch.float32, name)
+                if t.numel() != count:
+                    raise KernelError(f"low_rank: {name} has {t.numel()} numbers, needs {count}")
+        args += [p.col, rank, n, LOW_RANK_KINDS[p.kind], p.per_head, _ptr(p.weight), _ptr(p.bias), _ptr(p.a_log), 1.0 / p.tau, _ptr(p.out)]
+    types = [c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_float, c_void_p]
+    if len(products) == 1:
+        args += [0, 0, 0, 0, 1, c_void_p(0), c_void_p(0), c_void_p(0), 0.0, c_void_p(0)]
+    fn = _fn("recurrent", "tt_low_rank", [c_void_p, c_int, c_longlong, c_int, c_int, c_int, *types, *types, c_int, c_void_p])
+    _check(fn(ptr, splits, stride, cols, len(products), dtype_code(products[0].weight.dtype), *args, tokens, _stream()), "low_rank")
 
 
 def weighted_pair(a: torch.Tensor, wa: float, b: torch.Tensor, wb: float, out: torch.Tensor) -> None:

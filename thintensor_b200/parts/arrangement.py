@@ -98,12 +98,19 @@ class PreNormPair(Arrangement):
 
 @ARRANGEMENTS.register("parallel")
 class Parallel(Arrangement):
-    """One norm whose output both sublayers read: ``h = norm(x); x += mixer(shift(h)) + ffn(h)``.  ``shift`` (an input
-    shift, optional) stands between the norm and the mixer only; the feed-forward (optional) reads ``h`` as it is.  The
+    """Both sublayers read the same stream: ``h = norm(x); x += scale * (mixer(shift(h)) + ffn(h))``.  ``shift`` (an input
+    shift, optional) stands between the norm and the mixer only; the feed-forward (optional) reads ``h`` as it is, or, with
+    an ``ffn_norm``, the stream through a norm of its own (the two norms are then one kernel where their kinds allow).  The
     shift's per-sequence state is the arrangement's own."""
 
-    roles = {"norm": "norm", "shift": "shift", "mixer": "mixer", "ffn": "ffn"}
-    optional = ("shift", "ffn")
+    roles = {"norm": "norm", "shift": "shift", "mixer": "mixer", "ffn_norm": "norm", "ffn": "ffn"}
+    optional = ("shift", "ffn_norm", "ffn")
+
+    def __init__(self, parts, scale: float = 1.0):
+        super().__init__(parts)
+        if "ffn_norm" in parts and "ffn" not in parts:
+            raise ValueError("a parallel layer's second norm belongs to its feed-forward")
+        self.scale = float(scale)
 
     def mixers(self):
         return [self.parts["mixer"]]
@@ -117,21 +124,23 @@ class Parallel(Arrangement):
     def run(self, ctx, residual, pending: Delta | None, caches, states) -> Delta:
         hidden = residual.shape[-1]
         normed = ctx.scratch("block.normed", (ctx.n_tokens, hidden))
-        self.parts["norm"].forward(ctx, residual, pending, normed)
-        # both sublayers read `normed` and nothing reads the stream before the next norm, so either may add into it
-        ctx.residual = residual
+        ffn_in = normed
+        if "ffn_norm" in self.parts:
+            ffn_in = ctx.scratch("block.ffn_normed", (ctx.n_tokens, hidden))
+            self.parts["norm"].forward_pair(ctx, residual, pending, normed, self.parts["ffn_norm"], ffn_in)
+        else:
+            self.parts["norm"].forward(ctx, residual, pending, normed)
+        # both sublayers read normed rows and nothing reads the stream before the next norm, so either may add into it
+        # (not where the sum has a factor)
+        ctx.residual = residual if self.scale == 1.0 else None
         mixer_in = self.parts["shift"].forward(ctx, normed, states[1]) if "shift" in self.parts else normed
         mixed = self.parts["mixer"].forward(ctx, mixer_in, caches[0], states[0])
         if "ffn" not in self.parts:
-            return mixed
-        fed = self.parts["ffn"].forward(ctx, normed)
+            return Delta(mixed.tensor, scale=self.scale)
+        fed = self.parts["ffn"].forward(ctx, ffn_in)
         if mixed.tensor is None:
-            return fed
-        if fed.tensor is None:
-            return mixed
-        both = ctx.scratch("block.pair", (1, ctx.n_tokens, hidden), torch.float32)
-        api.weighted_pair(mixed.tensor, 1.0, fed.tensor, 1.0, both)
-        return Delta(both)
+            return Delta(fed.tensor, scale=self.scale)
+        return Delta(mixed.tensor, second=fed.tensor, scale=self.scale)       # the next norm's kernel adds the two
 
 
 @ARRANGEMENTS.register("sandwich")

@@ -11,7 +11,8 @@ Options beyond that form, each a parameter: value heads of another size than key
 (``value_dim``); queries and keys divided by their root mean square per head and multiplied
 by a weight of ``head_dim`` numbers that all heads share, before the rotation
 (``qk_norm_eps``); a learned number per query head whose exponential joins the softmax
-denominator without a key or a value (``sink``); a rotation that pairs neighbouring numbers
+denominator without a key or a value (``sink``), or a constant score that joins it for every head (``null_score``: 0 adds one
+to the denominator); keys of the query's own chunk only, chunks of ``chunk`` positions counted from the start of the sequence; a rotation that pairs neighbouring numbers
 (the position encoding's ``interleaved``); a short causal convolution over time on every channel
 of q, k and v right after their projections, ``y_t = sum_j w[:, j] u_(t - taps + 1 + j)`` with zeros before the
 sequence (``conv`` taps; the last ``taps - 1`` projected rows are a per-sequence state); scores capped by
@@ -48,13 +49,14 @@ def kv_splits(ctx, parallel_units: int, keys_per_slice: int, target_units: int) 
 class CausalAttention(Mixer):
     NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
              "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "sink": "sinks", "g": "g_proj.weight",
+             "q_bias": "q_proj.bias", "k_bias": "k_proj.bias", "v_bias": "v_proj.bias", "o_bias": "o_proj.bias",
              "q_conv": "q_conv.weight", "k_conv": "k_conv.weight", "v_conv": "v_conv.weight"}
 
     def __init__(self, hidden: int, heads: int, kv_heads: int, head_dim: int, position: PartSpec | None = None,
-                 bias: bool = False, window: int | None = None, scale: float | None = None, value_dim: int | None = None,
+                 bias: bool | str = False, window: int | None = None, scale: float | None = None, value_dim: int | None = None,
                  qk_norm_eps: float | None = None, sink: bool = False, names: dict | None = None, conv: int | None = None,
                  softcap: float | None = None, slope_exponent: float | None = None, gate: str | None = None, own_keys: bool = True,
-                 cache_window: int | None = None):
+                 cache_window: int | None = None, chunk: int | None = None, null_score: float | None = None):
         self.hidden, self.heads, self.kv_heads, self.head_dim = int(hidden), int(heads), int(kv_heads), int(head_dim)
         if self.heads % self.kv_heads:
             raise ValueError(f"{heads} query heads are not a multiple of {kv_heads} key/value heads")
@@ -67,7 +69,12 @@ class CausalAttention(Mixer):
         self.q_norm: torch.Tensor | None = None
         self.k_norm: torch.Tensor | None = None
         self.sinks: torch.Tensor | None = None
-        self.bias = bool(bias)
+        if bias not in (False, True, "qkv"):
+            raise ValueError(f"attention has no biases, biases on all projections, or on 'qkv', not {bias!r}")
+        self.bias = bias                        # True: q, k, v and the output projection; "qkv": the first three
+        self.null_score = None if null_score is None else float(null_score)
+        if self.sink and self.null_score is not None:
+            raise ValueError("an attention layer has learned sinks or a constant null score, not both")
         self.conv = int(conv) if conv else 0
         if self.conv and not 1 <= self.conv <= 8:
             raise ValueError("the convolution kernel takes 1 to 8 taps")
@@ -81,6 +88,9 @@ class CausalAttention(Mixer):
         self.slopes: torch.Tensor | None = None
         self.conv_weight: torch.Tensor | None = None
         self.window = None if not window else int(window)
+        self.chunk = None if not chunk else int(chunk)
+        if self.window and self.chunk:
+            raise ValueError("an attention layer has a window or chunks, not both")
         self.scale = float(scale) if scale is not None else self.head_dim ** -0.5
         position = position or PartSpec("none", {"head_dim": self.head_dim})
         self.position = POSITION_ENCODINGS.build(position.kind, dict(position.params))
@@ -114,10 +124,12 @@ class CausalAttention(Mixer):
         if self.sink:
             out[n["sink"]] = WeightDecl((self.heads,))
         if self.bias:
-            out.update({
-                "q_proj.bias": WeightDecl((q,)), "k_proj.bias": WeightDecl((kv,)), "v_proj.bias": WeightDecl((kv,)),
-                "o_proj.bias": WeightDecl((self.hidden,)),
-            })
+            out[n["q_bias"]] = WeightDecl((q,))
+            if self.own_keys:
+                out[n["k_bias"]] = WeightDecl((kv,))
+                out[n["v_bias"]] = WeightDecl((self.kv_heads * self.value_dim,))
+            if self.bias is True:
+                out[n["o_bias"]] = WeightDecl((self.hidden,))
         return out
 
     @property
@@ -130,10 +142,29 @@ class CausalAttention(Mixer):
         return self.heads * self.head_dim + (self.kv_heads * (self.head_dim + self.value_dim) if self.own_keys else 0)
 
     def cache_need(self) -> KVNeed:
-        window = self.window
+        window = self.window or self.chunk             # a chunk's keys are among its size's last ones
         if window is not None and self.cache_window:
             window = None if self.cache_window < 0 else max(window, self.cache_window)
         return KVNeed(self.kv_heads, self.head_dim, window, None if self.value_dim == self.head_dim else self.value_dim)
+
+    @property
+    def reach(self) -> int:
+        """Which keys a position sees, as the kernels take it: 0 all, n > 0 the last n, -n its own chunk's."""
+        return self.window or (-self.chunk if self.chunk else 0)
+
+    def visible_keys(self, position: float) -> float:
+        """Keys that the token at ``position`` (counted from 0) sees."""
+        seen = position + 1
+        return min(seen, self.window) if self.window else position % self.chunk + 1 if self.chunk else seen
+
+    def visible_pairs(self, tokens: int) -> float:
+        """(query, key) pairs of a sequence of ``tokens`` tokens."""
+        triangle = lambda n: n * (n + 1) / 2
+        if self.chunk:
+            return tokens // self.chunk * triangle(self.chunk) + triangle(tokens % self.chunk)
+        if self.window and self.window < tokens:
+            return triangle(self.window) + (tokens - self.window) * self.window
+        return triangle(tokens)
 
     def state_needs(self) -> list[StateNeed]:
         return [StateNeed((self.conv - 1, self.conv_channels), torch.float32)] if self.conv > 1 else []
@@ -141,7 +172,8 @@ class CausalAttention(Mixer):
     @property
     def general(self) -> bool:
         """Whether the layer needs the general kernels (see the module's text)."""
-        return (self.value_dim != self.head_dim or self.qk_norm_eps is not None or self.sink or bool(self.conv) or self.softcap > 0.0
+        return (self.value_dim != self.head_dim or self.qk_norm_eps is not None or self.sink or self.null_score is not None or bool(self.conv)
+                or self.softcap > 0.0
                 or self.slope_exponent is not None or self.gate is not None or not self.own_keys
                 or (self.rot is not None and self.rot.interleaved and self.rot.rotary_dim > 0))
 
@@ -154,13 +186,13 @@ class CausalAttention(Mixer):
         else:
             self.rot = RotaryTable(torch.zeros(1, dtype=torch.float32, device=device), 0, 1.0)
         n = self.names
-        if self.general and self.bias:
-            raise ValueError("attention with a value size of its own, a query/key norm, a sink or an interleaved rotation takes no biases")
         if self.qk_norm_eps is not None:
             self.q_norm = tensors[n["q_norm"]].to(torch.float32).contiguous()
             self.k_norm = tensors[n["k_norm"]].to(torch.float32).contiguous() if self.own_keys else None
         if self.sink:
             self.sinks = tensors[n["sink"]].to(torch.float32).contiguous()
+        elif self.null_score is not None:       # the kernels take it as a sink like any other
+            self.sinks = torch.full((self.heads,), self.null_score, dtype=torch.float32, device=device)
         if self.slope_exponent is not None:     # float64 powers, rounded once
             head = torch.arange(1, self.heads + 1, dtype=torch.float64)
             self.slopes = torch.pow(2.0, -self.slope_exponent * head / self.heads).to(torch.float32).to(device)
@@ -171,10 +203,13 @@ class CausalAttention(Mixer):
         weight = torch.cat(rows, dim=0) if len(rows) > 1 else rows[0]
         bias = None
         if self.bias:
-            bias = torch.cat([tensors["q_proj.bias"].float(), tensors["k_proj.bias"].float(), tensors["v_proj.bias"].float()])
+            pieces = [tensors[n[key + "_bias"]].float() for key in inputs]
+            if self.gate:                       # the gate has none
+                pieces.append(torch.zeros(self.gate_cols, dtype=torch.float32, device=pieces[0].device))
+            bias = torch.cat(pieces)
         self.qkv = Linear(weight, bias)                # [q | k | v | gate], without k and v in a layer that reads another's cache
         self.q_only = self.qkv.rows(0, self.heads * self.head_dim) if self.own_keys and not self.gate else self.qkv
-        self.out = Linear(tensors[n["o"]], tensors["o_proj.bias"] if self.bias else None)
+        self.out = Linear(tensors[n["o"]], tensors[n["o_bias"]] if self.bias is True else None)
 
     def projections(self) -> list:
         return [self.qkv, self.out]             # q_only is a view of qkv's first rows
@@ -236,7 +271,7 @@ class CausalAttention(Mixer):
             part_acc, part_ml = self.slice_scratch(ctx, splits)
             api.attention_decode_rope(projection, rot.inv_freq, rot.rotary_dim, rot.attention_scaling, cache.writes,
                                       cache.k_pool, cache.v_pool, table, ctx.len_before, ctx.sequences, self.heads, self.kv_heads,
-                                      self.head_dim, self.scale, self.window or 0, splits, mixed, part_acc, part_ml, ctx.status,
+                                      self.head_dim, self.scale, self.reach, splits, mixed, part_acc, part_ml, ctx.status,
                                       tickets=self.tickets(ctx, splits))
             return self.out.delta(ctx, mixed, "attention.out")
         q = ctx.scratch("attention.q", (ctx.n_tokens, q_cols))
@@ -266,7 +301,8 @@ class CausalAttention(Mixer):
         fastest when the slices just fill one wave of one CTA per SM and keep at least 8 blocks each; a
         second wave gains nothing."""
         splits = kv_splits(ctx, ctx.sequences * self.kv_heads, 512, api.sm_count(ctx.status.device))
-        return splits if not self.window else max(1, min(splits, self.window // 512))      # a window bounds the keys there are to slice
+        bound = self.window or self.chunk
+        return splits if not bound else max(1, min(splits, bound // 512))      # a window or a chunk bounds the keys there are to slice
 
     def slice_scratch(self, ctx, splits: int):
         """Where the slices of the keys leave their partial results (nothing for one slice)."""
@@ -301,7 +337,7 @@ class CausalAttention(Mixer):
             # be, but a softmax thread owns a row and reads its gate numbers one 32-byte sector a load (measured on a B200:
             # 2,048 tokens of 16 heads of 128 took 121 us with the gate inside against 50 + 15 us with the pass below)
             api.attention_tcgen05(q, cache.k_pool, cache.v_pool, table, ctx.cu, ctx.len_before, ctx.sequences, ctx.n_tokens, self.heads,
-                                  self.kv_heads, self.head_dim, self.scale, self.window or 0, mixed, ctx.status, sinks=self.sinks,
+                                  self.kv_heads, self.head_dim, self.scale, self.reach, mixed, ctx.status, sinks=self.sinks,
                                   softcap=self.softcap, slopes=self.slopes)
             if gate is not None:
                 api.sigmoid_gate(mixed, gate, self.value_dim if self.gate == "head" else 0)
@@ -315,16 +351,16 @@ class CausalAttention(Mixer):
         part_acc, part_ml = self.slice_scratch(ctx, splits)
         if tensor_cores:
             api.attention_mma(q, cache.k_pool, cache.v_pool, table, ctx.cu, ctx.len_before, ctx.sequences, ctx.n_tokens, self.heads,
-                              self.kv_heads, self.head_dim, self.scale, self.window or 0, splits, mixed, part_acc, part_ml, ctx.status,
+                              self.kv_heads, self.head_dim, self.scale, self.reach, splits, mixed, part_acc, part_ml, ctx.status,
                               one_token_each=ctx.decode, tickets=self.tickets(ctx, splits) if ctx.decode else None,
                               sinks=self.sinks if ctx.decode else None, softcap=self.softcap, slopes=self.slopes)
             if gate is not None:
                 api.sigmoid_gate(mixed, gate, self.value_dim if self.gate == "head" else 0)
         else:
-            if self.window:                     # a window bounds the keys a slice can hold
-                splits = max(1, min(splits, self.window // 64))
+            if self.window or self.chunk:       # they bound the keys a slice can hold
+                splits = max(1, min(splits, (self.window or self.chunk) // 64))
                 part_acc, part_ml = self.slice_scratch(ctx, splits)
             api.attention(q, cache.k_pool, cache.v_pool, table, ctx.cu, ctx.len_before, ctx.sequences, ctx.n_tokens, self.heads,
-                          self.kv_heads, self.head_dim, self.scale, self.window or 0, splits, mixed, part_acc, part_ml, ctx.status,
+                          self.kv_heads, self.head_dim, self.scale, self.reach, splits, mixed, part_acc, part_ml, ctx.status,
                           value_dim=self.value_dim, sinks=self.sinks, softcap=self.softcap, slopes=self.slopes, gate=gate,
                           gate_per_head=self.gate == "head")

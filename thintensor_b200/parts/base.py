@@ -40,7 +40,8 @@ import torch
 class WeightDecl:
     """A tensor a part needs.  ``init`` tells the random-weights mode how to draw it:
     ``normal`` is N(0, 0.02), ``norm`` is 1 + N(0, 0.1), ``small`` is N(0, 0.1), ``depth`` is N(0, 0.3) with one added to the last number,
-    ``zeros`` is zero.
+    ``zeros`` is zero.  ``free`` lists axes whose extent the checkpoint decides (the rank of a product of low rank, say); ``shape``
+    then holds what random weights are drawn with, and the part reads the real extent off the tensor it is bound to.
     ``alias_of`` names a checkpoint tensor (full name) to use instead when this one is
     absent from the checkpoint; with ``prefer_alias`` it is used even when this one is
     stored (a tied output head, whose stored copy is ignored)."""
@@ -51,6 +52,11 @@ class WeightDecl:
     alias_of: str | None = None
     prefer_alias: bool = False
     integer: bool = False
+    free: tuple[int, ...] = ()
+
+    def fits(self, shape) -> bool:
+        return len(shape) == len(self.shape) and all(have == want or (axis in self.free and have > 0)
+                                                     for axis, (have, want) in enumerate(zip(shape, self.shape)))
 
 
 @dataclass(frozen=True)
@@ -108,11 +114,26 @@ class Delta:
 
     ``post``: the sum is normalised (RMS norm with this weight) before it is added.  ``depth``: after the
     addition the stream is kept as a layer's result and replaced by a weighted sum of the results so far.
-    Both are carried out by the norm that follows, in its one pass over the row."""
+    Both are carried out by the norm that follows, in its one pass over the row.
+
+    ``second``: another sublayer's partial sums, added to the first's.  ``scale`` multiplies both.  ``addend`` (float32
+    ``[tokens, hidden]``) is added as it is.  The norm that follows does these too."""
 
     tensor: torch.Tensor | None
     post: "PostNorm | None" = None
     depth: "DepthStep | None" = None
+    second: torch.Tensor | None = None
+    scale: float = 1.0
+    addend: torch.Tensor | None = None
+
+    @property
+    def plain(self) -> bool:
+        """Whether the delta is nothing but the sum of ``tensor``."""
+        return self.post is None and self.depth is None and not self.branched
+
+    @property
+    def branched(self) -> bool:
+        return self.second is not None or self.scale != 1.0 or self.addend is not None
 
     @property
     def splits(self) -> int:
@@ -153,6 +174,12 @@ class Part:
 class Norm(Part):
     def forward(self, ctx, residual: torch.Tensor, delta: Delta | None, out: torch.Tensor, rows: torch.Tensor | None = None) -> None:
         raise NotImplementedError
+
+    def forward_pair(self, ctx, residual: torch.Tensor, delta: Delta | None, out: torch.Tensor, other: "Norm", other_out: torch.Tensor) -> None:
+        """Add ``delta`` into the stream and take two norms of it, this one and ``other``.  Norms that can share one pass
+        over a row override this."""
+        self.forward(ctx, residual, delta, out)
+        other.forward(ctx, residual, None, other_out)
 
 
 @dataclass(frozen=True)

@@ -7,7 +7,9 @@ for Llama (thinruntime/model_arch.py:231-233) and 1 for a weight that is stored 
 
 The delta that a norm adds may ask for more on the way (see :class:`~thintensor_b200.parts.base.Delta`): to be
 normalised itself before the stream takes it, and for the stream to be replaced, after the addition, by a weighted sum
-of the layers' results so far.  The RMS norm's kernel does all of it in its one pass over a row.
+of the layers' results so far.  The RMS norm's kernel does all of it in its one pass over a row.  Or it may bring two
+sublayers' outputs with a common factor and something else to add; both norms' kernels take those, and two norms of the
+same kind over the same stream (a parallel layer's) are one kernel.
 """
 from __future__ import annotations
 
@@ -46,6 +48,8 @@ class RMSNorm(Norm):
     def forward(self, ctx, residual, delta: Delta | None, out, rows=None) -> None:
         if delta is not None and (delta.post is not None or delta.depth is not None):
             post, depth = delta.post, delta.depth
+            if delta.branched:
+                raise NotImplementedError("a delta that is normalised or mixed on its way brings one sublayer's output without a factor")
             if post is not None and delta.tensor is None:
                 raise RuntimeError("a delta that is already in the stream cannot be normalised on its way there")
             api.add_rmsnorm_chain(residual, delta.tensor, None if post is None else post.weight, 0.0 if post is None else post.offset,
@@ -53,7 +57,19 @@ class RMSNorm(Norm):
                                   0 if depth is None else depth.index, None if depth is None else depth.weights, self.weight,
                                   self.weight_offset, self.eps, out, rows)
             return
+        if delta is not None and delta.branched:
+            api.add_norms(residual, delta.tensor, delta.second, delta.scale, delta.addend, self.weight, None, out, self.eps, False,
+                          self.weight_offset, rows=rows)
+            return
         api.add_rmsnorm(residual, None if delta is None else delta.tensor, self.weight, self.eps, out, rows, self.weight_offset)   # an empty delta is already in the stream
+
+    def forward_pair(self, ctx, residual, delta: Delta | None, out, other, other_out) -> None:
+        special = delta is not None and (delta.post is not None or delta.depth is not None)
+        if special or not isinstance(other, RMSNorm) or (other.eps, other.weight_offset) != (self.eps, self.weight_offset):
+            return super().forward_pair(ctx, residual, delta, out, other, other_out)
+        delta = delta or Delta(None)
+        api.add_norms(residual, delta.tensor, delta.second, delta.scale, delta.addend, self.weight, None, out, self.eps, False,
+                      self.weight_offset, (other.weight, None, other_out))
 
 
 @NORMS.register("layernorm")
@@ -86,5 +102,16 @@ class LayerNorm(Norm):
 
     def forward(self, ctx, residual, delta: Delta | None, out, rows=None) -> None:
         if delta is not None and (delta.post is not None or delta.depth is not None):
-            raise NotImplementedError("the layer norm adds plain deltas only")
+            raise NotImplementedError("the layer norm's kernel neither normalises a delta nor mixes results")
+        if delta is not None and delta.branched:
+            api.add_norms(residual, delta.tensor, delta.second, delta.scale, delta.addend, self.weight, self.shift, out, self.eps, True, rows=rows)
+            return
         api.add_layernorm(residual, None if delta is None else delta.tensor, self.weight, self.shift, self.eps, out, rows)
+
+    def forward_pair(self, ctx, residual, delta: Delta | None, out, other, other_out) -> None:
+        special = delta is not None and (delta.post is not None or delta.depth is not None)
+        if special or not isinstance(other, LayerNorm) or other.eps != self.eps:
+            return super().forward_pair(ctx, residual, delta, out, other, other_out)
+        delta = delta or Delta(None)
+        api.add_norms(residual, delta.tensor, delta.second, delta.scale, delta.addend, self.weight, self.shift, out, self.eps, True, 0.0,
+                      (other.weight, other.shift, other_out))

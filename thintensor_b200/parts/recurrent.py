@@ -22,7 +22,10 @@ convolutions of their own (no bias) and silu; q and k become unit vectors per he
 value_dim, ``S <- g S``, ``u = beta (v - S^T k)``, ``S <- S + k u^T``, ``o = S^T q`` with
 ``beta = sigmoid(W_b h)`` and ``g = exp(-exp(A_log) softplus(W_a h + dt_bias))``; each head's o is
 divided by its root mean square, multiplied by a weight of ``value_dim`` numbers that the heads
-share, and by ``silu(W_g h)``.
+share, and by ``silu(W_g h)``.  Options: a decay for every head and key channel from a product of low rank
+(``channel_decay``), ``g = exp(-exp(A_log) softplus(W_a2 (W_a1 h) + dt_bias))`` with ``dt_bias`` and g laid out heads x key_dim
+and A_log still one number per head, g multiplying the rows of S; a gate from a product of low rank (``low_rank_gate``),
+``W_g2 (W_g1 h)``, and ``sigmoid`` instead of silu on it (``gate``).  The ranks are the checkpoint's.
 
 ``decay_linear_attention``: linear attention with a fixed decay per head and neither softmax nor
 denominator: per head, with S of shape key_dim x value_dim, ``S <- decay_h S + k v^T`` and ``o = S^T q``.
@@ -30,7 +33,10 @@ Two published forms are parameter sets of it.  Lightning attention: ``activation
 the read-out of all heads RMS-normed together with a weight (``norm="all"``) and gated by
 ``sigmoid(W_g h)``.  Retention: q and k rotated by the position (``position``), k times
 ``key_dim ** -0.5`` (``key_scale``), every head's read-out divided by its own root mean square without a
-weight (``norm="head"``) and gated by ``silu(W_g h)``.  There is no convolution; the only state is S.
+weight (``norm="head"``) and gated by ``silu(W_g h)``.  With ``channel_decay`` the decay is not fixed but comes from the
+token, one number per head and key channel, ``S <- diag(a) S + k v^T`` with ``a = sigmoid(W_a2 (W_a1 h) + b) ** (1 / tau)``: gated
+linear attention (Yang, Wang, Shen, Panda and Kim, "Gated Linear Attention Transformers with Hardware-Efficient Training"),
+q times ``query_scale``.  There is no convolution; the only state is S.
 
 Decays, step sizes, gates of the recurrence, unit norms and the states are float32 whatever the
 model's dtype; only the normed read-out that feeds the output projection is narrowed.
@@ -47,6 +53,18 @@ from .spec import PartSpec
 
 def _f32(t: torch.Tensor) -> torch.Tensor:
     return t.to(torch.float32).contiguous()
+
+
+def _low_rank_decls(down: str, up: str, inputs: int, rank: int, outputs: int) -> dict[str, WeightDecl]:
+    """A product of low rank, ``W_up (W_down h)``; the rank is the checkpoint's."""
+    return {down: WeightDecl((rank, inputs), free=(0,)), up: WeightDecl((outputs, rank), free=(1,))}
+
+
+def _low_rank_up(tensors, down: str, up: str) -> torch.Tensor:
+    """The second matrix as the kernel reads it, ``[rank, outputs]``."""
+    if tensors[down].shape[0] != tensors[up].shape[1]:
+        raise ValueError(f"{down!r} makes {tensors[down].shape[0]} numbers, {up!r} takes {tensors[up].shape[1]}")
+    return tensors[up].t().contiguous()
 
 
 @MIXERS.register("mamba2")
@@ -123,10 +141,13 @@ class Mamba2(Mixer):
 class GatedDelta(Mixer):
     NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "q_conv": "q_conv1d.weight", "k_conv": "k_conv1d.weight",
              "v_conv": "v_conv1d.weight", "b": "b_proj.weight", "a": "a_proj.weight", "g": "g_proj.weight", "dt_bias": "dt_bias",
-             "A_log": "A_log", "norm": "o_norm.weight", "out": "o_proj.weight"}
+             "A_log": "A_log", "norm": "o_norm.weight", "out": "o_proj.weight", "a1": "a1_proj.weight", "a2": "a2_proj.weight",
+             "g1": "g1_proj.weight", "g2": "g2_proj.weight"}
 
     def __init__(self, hidden: int, heads: int, qk_heads: int, key_dim: int, value_dim: int, conv: int = 4, eps: float = 1e-6,
-                 names: dict | None = None):
+                 names: dict | None = None, channel_decay: int | None = None, low_rank_gate: int | None = None, gate: str = "silu"):
+        """``channel_decay`` and ``low_rank_gate``: the rank with which random weights are drawn (a checkpoint may bring
+        another), or None for the forms of full rank."""
         self.hidden, self.heads, self.qk_heads = int(hidden), int(heads), int(qk_heads)
         self.key_dim, self.value_dim, self.conv, self.eps = int(key_dim), int(value_dim), int(conv), float(eps)
         if self.heads % self.qk_heads:
@@ -135,6 +156,13 @@ class GatedDelta(Mixer):
             raise ValueError("the recurrent kernels take 1 to 8 convolution taps and key sizes of up to 256")
         self.qk, self.v = self.qk_heads * self.key_dim, self.heads * self.value_dim
         self.channels = 2 * self.qk + self.v                               # what passes the convolutions: q, k, v
+        self.channel_decay = None if channel_decay is None else int(channel_decay)
+        self.low_rank_gate = None if low_rank_gate is None else int(low_rank_gate)
+        if gate not in api.NORM_GATES:
+            raise ValueError(f"the gate is one of {sorted(api.NORM_GATES)}, not {gate!r}")
+        self.gate = gate
+        self.decay_up: torch.Tensor | None = None
+        self.gate_up: torch.Tensor | None = None
         self.names = {**self.NAMES, **(names or {})}
         self.proj: Linear | None = None
         self.out: Linear | None = None
@@ -151,9 +179,11 @@ class GatedDelta(Mixer):
             n["b"]: WeightDecl((self.heads, self.hidden)),
             n["A_log"]: WeightDecl((self.heads,)),
             n["norm"]: WeightDecl((self.value_dim,), init="norm"),
-            n["a"]: WeightDecl((self.heads, self.hidden)),
-            n["dt_bias"]: WeightDecl((self.heads,)),
-            n["g"]: WeightDecl((self.v, self.hidden)),
+            **(_low_rank_decls(n["a1"], n["a2"], self.hidden, self.channel_decay, self.heads * self.key_dim) if self.channel_decay
+               else {n["a"]: WeightDecl((self.heads, self.hidden))}),
+            n["dt_bias"]: WeightDecl((self.heads * self.key_dim if self.channel_decay else self.heads,)),
+            **(_low_rank_decls(n["g1"], n["g2"], self.hidden, self.low_rank_gate, self.v) if self.low_rank_gate
+               else {n["g"]: WeightDecl((self.v, self.hidden))}),
             n["out"]: WeightDecl((self.hidden, self.v)),
         }
 
@@ -163,9 +193,17 @@ class GatedDelta(Mixer):
 
     def bind(self, tensors, dtype, device) -> None:
         n = self.names
-        # one product for everything linear in the input: [q | k | v | gate | b | a]
-        self.proj = Linear(torch.cat([tensors[n[key]] for key in ("q", "k", "v", "g", "b", "a")], dim=0))
+        # one product for everything linear in the input: [q | k | v | gate | b | a], gate and a down to their ranks only where
+        # they are products of low rank
+        gate, decay = "g1" if self.low_rank_gate else "g", "a1" if self.channel_decay else "a"
+        self.proj = Linear(torch.cat([tensors[n[key]] for key in ("q", "k", "v", gate, "b", decay)], dim=0))
         self.out = Linear(tensors[n["out"]])
+        self.b_col = self.channels + tensors[n[gate]].shape[0]
+        self.a_col = self.b_col + self.heads
+        self.decay_up = _low_rank_up(tensors, n["a1"], n["a2"]) if self.channel_decay else None
+        self.gate_up = _low_rank_up(tensors, n["g1"], n["g2"]) if self.low_rank_gate else None
+        if self.decay_up is not None and self.gate_up is not None and self.decay_up.dtype != self.gate_up.dtype:
+            self.decay_up, self.gate_up = _f32(self.decay_up), _f32(self.gate_up)       # one launch for both
         self.conv_weight = torch.cat([_f32(tensors[n[key]]) for key in ("q_conv", "k_conv", "v_conv")], dim=0).contiguous()
         self.dt_bias, self.a_log, self.norm = _f32(tensors[n["dt_bias"]]), _f32(tensors[n["A_log"]]), _f32(tensors[n["norm"]])
 
@@ -173,7 +211,7 @@ class GatedDelta(Mixer):
         return [self.proj, self.out]
 
     def vectors(self) -> list[torch.Tensor]:
-        return [self.conv_weight, self.dt_bias, self.a_log, self.norm]
+        return [self.conv_weight, self.dt_bias, self.a_log, self.norm] + [t for t in (self.decay_up, self.gate_up) if t is not None]
 
     def device_driven(self) -> bool:
         return True
@@ -182,29 +220,48 @@ class GatedDelta(Mixer):
         recurrent, tail = states
         tokens = ctx.n_tokens
         proj = self.proj(ctx, x, "delta.in")
+        decay, gate_source, gate_col = None, proj, self.channels
+        products = []
+        if self.decay_up is not None:
+            decay = ctx.scratch("delta.decay", (tokens, self.heads * self.key_dim), torch.float32)
+            products.append(api.LowRank(self.a_col, self.decay_up, decay, "delta_decay", self.dt_bias, self.a_log, self.key_dim))
+        if self.gate_up is not None:
+            gates = ctx.scratch("delta.gates", (1, tokens, self.v), torch.float32)
+            products.append(api.LowRank(self.channels, self.gate_up, gates[0]))
+            gate_source, gate_col = gates, 0
+        if products:
+            api.low_rank(proj, products)
         qkv = ctx.scratch("delta.qkv", (tokens, self.channels), torch.float32)
         api.causal_conv(proj, 0, self.channels, self.conv_weight, None, True, tail, qkv, ctx.cu, ctx.slots, ctx.sequences, tokens, ctx.decode)
-        gate_col = self.channels
         read = ctx.scratch("delta.read", (tokens, self.v), torch.float32)
-        api.delta_scan(qkv, proj, gate_col + self.v, gate_col + self.v + self.heads, self.dt_bias, self.a_log, recurrent, read, ctx.cu,
-                       ctx.slots, ctx.sequences, self.heads, self.qk_heads, self.key_dim, self.value_dim)
+        api.delta_scan(qkv, proj, self.b_col, self.a_col, self.dt_bias, self.a_log, recurrent, read, ctx.cu,
+                       ctx.slots, ctx.sequences, self.heads, self.qk_heads, self.key_dim, self.value_dim, row_decay=decay)
         gated = ctx.scratch("delta.gated", (tokens, self.v))
-        api.gated_group_norm(read, self.value_dim, proj, gate_col, self.norm, self.eps, False, gated)
+        api.gated_group_norm(read, self.value_dim, gate_source, gate_col, self.norm, self.eps, False, gated, self.gate)
         return self.out.delta(ctx, gated, "delta.out")
 
 
 @MIXERS.register("decay_linear_attention")
 class DecayLinearAttention(Mixer):
     NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "g": "g_proj.weight", "norm": "norm.weight",
-             "out": "o_proj.weight"}
+             "out": "o_proj.weight", "a1": "a1_proj.weight", "a2": "a2_proj.weight", "a_bias": "a2_proj.bias"}
 
-    def __init__(self, hidden: int, heads: int, key_dim: int, value_dim: int, decay, activation: str | None = None,
+    def __init__(self, hidden: int, heads: int, key_dim: int, value_dim: int, decay=None, activation: str | None = None,
                  position: PartSpec | None = None, key_scale: float = 1.0, norm: str = "head", norm_weight: bool = False,
-                 gate: str = "silu", eps: float = 1e-6, names: dict | None = None):
+                 gate: str = "silu", eps: float = 1e-6, names: dict | None = None, channel_decay: dict | None = None,
+                 query_scale: float = 1.0):
+        """``channel_decay``: ``{"tau": the root, "rank": the rank with which random weights are drawn}``, instead of ``decay``."""
         self.hidden, self.heads, self.key_dim, self.value_dim = int(hidden), int(heads), int(key_dim), int(value_dim)
-        self.decay = tuple(float(d) for d in decay)
-        if len(self.decay) != self.heads:
+        if (decay is None) == (channel_decay is None):
+            raise ValueError("linear attention has a fixed decay per head or one per key channel from the token")
+        self.decay = None if decay is None else tuple(float(d) for d in decay)
+        if self.decay is not None and len(self.decay) != self.heads:
             raise ValueError(f"{len(self.decay)} decays for {self.heads} heads")
+        self.rank = None if channel_decay is None else int(channel_decay["rank"])
+        self.tau = None if channel_decay is None else float(channel_decay["tau"])
+        self.query_scale = float(query_scale)
+        self.decay_up: torch.Tensor | None = None
+        self.decay_bias: torch.Tensor | None = None
         if activation not in (None, "silu"):
             raise ValueError(f"q, k and v pass silu or nothing, not {activation!r}")
         if norm not in ("head", "all"):
@@ -234,6 +291,9 @@ class DecayLinearAttention(Mixer):
             n["g"]: WeightDecl((self.v, self.hidden)),
             n["out"]: WeightDecl((self.hidden, self.v)),
         }
+        if self.rank is not None:
+            out.update(_low_rank_decls(n["a1"], n["a2"], self.hidden, self.rank, self.qk))
+            out[n["a_bias"]] = WeightDecl((self.qk,))
         if self.norm_weight:
             out[n["norm"]] = WeightDecl((self.v if self.norm == "all" else self.value_dim,), init="norm")
         return out
@@ -249,10 +309,15 @@ class DecayLinearAttention(Mixer):
             self.rot = self.position.rotary()
             if self.rot.interleaved or self.rot.attention_scaling != 1.0 or self.rot.rotary_dim % 2 or self.rot.rotary_dim > self.key_dim:
                 raise ValueError("linear attention rotates halves of an even part of the head and does not scale the rotation")
-        # one product for everything linear in the input: [q | k | v | gate]
-        self.proj = Linear(torch.cat([tensors[n[key]] for key in ("q", "k", "v", "g")], dim=0))
+        # one product for everything linear in the input: [q | k | v | gate], then the first half of the decays' product
+        keys = ("q", "k", "v", "g") + (("a1",) if self.rank is not None else ())
+        self.proj = Linear(torch.cat([tensors[n[key]] for key in keys], dim=0))
         self.out = Linear(tensors[n["out"]])
-        self.decays = torch.tensor(self.decay, dtype=torch.float32, device=device)
+        self.decays = None
+        if self.rank is not None:
+            self.decay_up, self.decay_bias = _low_rank_up(tensors, n["a1"], n["a2"]), _f32(tensors[n["a_bias"]])
+        else:
+            self.decays = torch.tensor(self.decay, dtype=torch.float32, device=device)
         count = self.v if self.norm == "all" else self.value_dim
         self.norm_w = _f32(tensors[n["norm"]]) if self.norm_weight else torch.ones(count, dtype=torch.float32, device=device)
 
@@ -260,7 +325,7 @@ class DecayLinearAttention(Mixer):
         return [self.proj, self.out]
 
     def vectors(self) -> list[torch.Tensor]:
-        return [self.norm_w] if self.norm_weight else []
+        return ([self.norm_w] if self.norm_weight else []) + [t for t in (self.decay_up, self.decay_bias) if t is not None]
 
     def device_driven(self) -> bool:
         return True
@@ -273,9 +338,14 @@ class DecayLinearAttention(Mixer):
         rotary_dim = self.rot.rotary_dim if self.rot is not None else 0
         api.linear_attention_prepare(proj, self.heads, self.key_dim, self.value_dim, self.activation == "silu",
                                      self.rot.inv_freq if rotary_dim else None, rotary_dim, self.key_scale, vkq, ctx.cu, ctx.len_before,
-                                     ctx.sequences, tokens)
+                                     ctx.sequences, tokens, self.query_scale)
         read = ctx.scratch("linear_attention.read", (tokens, self.v), torch.float32)
-        api.decay_scan(vkq, self.decays, recurrent, read, ctx.cu, ctx.slots, ctx.sequences, self.heads, self.key_dim, self.value_dim)
+        if self.decay_up is not None:
+            decay = ctx.scratch("linear_attention.decay", (tokens, self.qk), torch.float32)
+            api.low_rank(proj, [api.LowRank(2 * self.qk + 2 * self.v, self.decay_up, decay, "sigmoid_root", self.decay_bias, tau=self.tau)])
+            api.row_decay_scan(vkq, decay, recurrent, read, ctx.cu, ctx.slots, ctx.sequences, self.heads, self.key_dim, self.value_dim)
+        else:
+            api.decay_scan(vkq, self.decays, recurrent, read, ctx.cu, ctx.slots, ctx.sequences, self.heads, self.key_dim, self.value_dim)
         gated = ctx.scratch("linear_attention.gated", (tokens, self.v))
         api.gated_group_norm(read, self.v if self.norm == "all" else self.value_dim, proj, 2 * self.qk + self.v, self.norm_w, self.eps,
                              False, gated, self.gate)

@@ -52,7 +52,7 @@ class TokenSide(SideInput):
         return True
 
     def forward(self, ctx, residual, pending: Delta | None) -> Delta:
-        if pending is not None and (pending.post is not None or pending.depth is not None):
+        if pending is not None and not pending.plain:
             raise RuntimeError("the token side input follows a plain delta")
         stream = ctx.scratch("side.stream", tuple(residual.shape))
         api.add_narrow(residual, None if pending is None else pending.tensor, stream)

@@ -42,10 +42,13 @@ class LayerSpec:
 class Run:
     """One entry of the schedule: run layer ``layer``.  Every run has a cache and a
     state of its own unless ``cache_from`` names an earlier entry of the schedule,
-    whose cache this run then reads without writing to it."""
+    whose cache this run then reads without writing to it.  ``add_embedding``: the embedding's
+    output is added to the stream before the layer (each further pass of a stretch of layers that
+    runs several times, say)."""
 
     layer: int
     cache_from: int | None = None
+    add_embedding: bool = False
 
 
 @dataclass(frozen=True)
@@ -60,6 +63,8 @@ class ModelSpec:
 
     def validate(self) -> None:
         for index, run in enumerate(self.schedule):
+            if run.add_embedding and index == 0:
+                raise ValueError("the schedule's first run already starts from the embedding's output")
             if not 0 <= run.layer < len(self.layers):
                 raise ValueError(f"schedule entry {index} names layer {run.layer}, but there are {len(self.layers)} layers")
             if run.cache_from is not None:

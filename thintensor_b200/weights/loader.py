@@ -69,7 +69,7 @@ def compare(declared: dict[str, WeightDecl], stored: dict[str, tuple[int, ...]])
                 missing.append(name)
             continue
         used.add(source)
-        if tuple(stored[source]) != tuple(decl.shape):
+        if not decl.fits(tuple(stored[source])):
             wrong.append(f"{source}: checkpoint has {list(stored[source])}, the model needs {list(decl.shape)}")
     unexpected = [
         name for name in stored
