@@ -112,6 +112,7 @@ FAMALORN_SHAPES = {"1b": "famalorn-w2048", "3b": "famalorn-w3072"}
 NERUZEN_SHAPES = {"1b": "neruzen-w2048", "3b": "neruzen-w3072"}
 SOGIDRA_SHAPES = {"1b": "sogidra-w2048", "3b": "sogidra-w3072"}
 KEREPEL_SHAPES = {"1b": "kerepel-w2048", "3b": "kerepel-w3072"}
+ZUVEPEL_SHAPES = {"1b": "zuvepel-w2048", "3b": "zuvepel-w3072"}
 
 
 def neruzen_pair(size: str) -> tuple[dict, dict]:
@@ -130,6 +131,14 @@ def kerepel_pair(size: str) -> tuple[dict, dict]:
     project their queries directly and gate their heads; its attention layers (16 or 24 heads of 128, a window of 1,024, two of
     the four reading another layer's keys) stand where Neruzen has linear attentions; every other feed-forward is dense (8,192)."""
     return json.loads(json.dumps(SHAPES[KEREPEL_SHAPES[size]])), json.loads(json.dumps(SHAPES[NERUZEN_SHAPES[size]]))
+
+
+def zuvepel_pair(size: str) -> tuple[dict, dict]:
+    """(Zuvepel config.json, Famalorn config.json) of one size from the table of named shapes: the same width, feed-forward
+    width, vocabulary and number of layers (six, each run once).  Famalorn is the closest model: its delta layers have the same
+    heads (a decay per head where Zuvepel's have one per key channel), its Mamba-2 scan is the like of the gla layers' scan (16 or
+    24 heads of 64 x 128), its attention branch has the same heads and a sink (Zuvepel's: chunks of 1,024)."""
+    return json.loads(json.dumps(SHAPES[ZUVEPEL_SHAPES[size]])), json.loads(json.dumps(SHAPES[FAMALORN_SHAPES[size]]))
 
 
 def sogidra_pair(size: str) -> tuple[dict, dict]:
@@ -157,14 +166,15 @@ def design_bench(args) -> int:
     """``--design famalorn``: prefill and decode of the Famalorn design beside the Llama decoder at equal size (random
     weights, bfloat16), with each step's time by class of kernel against that class's bound.  ``--design neruzen``: the
     same for the Neruzen design beside Famalorn, ``--design sogidra`` for the Sogidra design beside Llama, ``--design kerepel``
-    for the Kerepel design beside Neruzen.  One JSON line."""
+    for the Kerepel design beside Neruzen, ``--design zuvepel`` for the Zuvepel design beside Famalorn.  One JSON line."""
     import thintensor_b200
     from thintensor_b200.benchmark import class_fractions, measure_classes, measure_decode, measure_prefill
 
     pk = peaks()
     import torch
     names, pair = {"famalorn": (("famalorn", "llama"), famalorn_pair), "neruzen": (("neruzen", "famalorn"), neruzen_pair),
-                   "sogidra": (("sogidra", "llama"), sogidra_pair), "kerepel": (("kerepel", "neruzen"), kerepel_pair)}[args.design]
+                   "sogidra": (("sogidra", "llama"), sogidra_pair), "kerepel": (("kerepel", "neruzen"), kerepel_pair),
+                   "zuvepel": (("zuvepel", "famalorn"), zuvepel_pair)}[args.design]
     out = {"bench": f"{names[0].capitalize()} beside {names[1].capitalize()} at equal width, feed-forward, vocabulary and layers; random weights, bfloat16",
            "prompt_len": args.prompt_len, "batch": args.batch, "peaks": pk, "sizes": {}}
     for size in args.sizes.split(","):
@@ -213,8 +223,8 @@ def main() -> int:
     parser.add_argument("--batch", type=int, default=BATCH, help="with --only decode: sequences decoded together")
     parser.add_argument("--shape", choices=sorted(SHAPE_NAMES), default="1b", help="with --only: layer sizes of another model of the family")
     parser.add_argument("--prompt-len", type=int, default=PROMPT, help="with --only: tokens per prompt (the context is this plus room for the steps)")
-    parser.add_argument("--design", choices=["famalorn", "neruzen", "sogidra", "kerepel"],
-                        help="measure this design beside the closest model the library has at equal size (Famalorn beside Llama, Neruzen beside Famalorn, Sogidra beside Llama, Kerepel beside Neruzen) instead of the headline")
+    parser.add_argument("--design", choices=["famalorn", "neruzen", "sogidra", "kerepel", "zuvepel"],
+                        help="measure this design beside the closest model the library has at equal size (Famalorn beside Llama, Neruzen beside Famalorn, Sogidra beside Llama, Kerepel beside Neruzen, Zuvepel beside Famalorn) instead of the headline")
     parser.add_argument("--sizes", default="1b,3b", help="with --design: which sizes (1b: width 2,048; 3b: width 3,072)")
     args = parser.parse_args()
     if args.design:

@@ -200,7 +200,7 @@ def class_fractions(model, classes: dict, pk: dict, prefill_prompts: list[list[i
     sampling) has no bound worth naming and is given as time alone.  Times are those of kernels run
     one after another (see :func:`measure_classes`)."""
     attention_kernels = ("tt_attention", "tt_latent_attention", "tt_differential_attention", "tt_pooled_window_attention")
-    recurrent = ("tt_mamba2_scan", "tt_delta_scan", "tt_causal_conv", "tt_gated_group_norm", "tt_decay_scan", "tt_row_decay_scan",
+    recurrent = ("tt_mamba2_scan", "tt_delta_scan", "tt_causal_conv", "tt_gated_group_norm", "tt_decay_scan", "tt_row_decay_scan", "tt_row_decay_blocks",
                  "tt_low_rank", "tt_linear_attention_prepare")
 
     def split(spans: dict) -> dict:

@@ -686,6 +686,368 @@ extern "C" int tt_delta_scan(const float* qkv, int qkv_cols, const float* proj, 
 }
 
 // ------------------------------------------------------------------------------------
+// The two recurrences with a decay per state row, for prompts: four tokens at a time.
+//
+// Within a block of tokens 0 .. 3 with decays g_t (vectors over the state's rows), P_t = g_0 * .. * g_t elementwise and
+// s_(j,t) = g_(j+1) * .. * g_t, everything that reads the state reads the state before the block, S:
+//   delta rule:        u_t = beta_t (v_t - S^T (P_t k_t) - sum_(j<t) [k_t . (s_(j,t) k_j)] u_j)
+//   linear attention:  u_t = v_t
+//   both:              o_t = S^T (P_t q_t) + sum_(j<=t) [q_t . (s_(j,t) k_j)] u_j,   S <- P_3 S + sum_j (s_(j,3) k_j) u_j^T
+// so the eight (four) row products of a column are independent of one another and summed over its lanes together, where
+// token by token each waits for the one before.  Only products of decays enter, never a quotient, so nothing can overflow
+// that does not overflow in the recurrence itself, and all of it is float32.  The scaled vectors and the products in square
+// brackets are the same for every column: four warps of the CTA prepare them for the 16 tokens ahead while four others walk
+// the state through the 16 tokens before.
+//
+// A column's D state rows lie in the registers of RB_LANES neighbouring lanes, each lane holding the same rows of RB_COLS
+// neighbouring columns; a CTA takes RB_TILE columns of one (sequence, head).  Blocks that are not full are filled with
+// tokens that change nothing (k = q = 0, decay 1, beta 0).
+// ------------------------------------------------------------------------------------
+constexpr int RB_BLOCK = 4;                 // tokens of a block
+constexpr int RB_BLOCKS = 4;                // blocks prepared at a time, one by each preparing warp
+constexpr int RB_CHUNK = RB_BLOCK * RB_BLOCKS;
+constexpr int RB_LANES = 16, RB_COLS = 2;
+constexpr int RB_SCAN_WARPS = 4;
+constexpr int RB_TILE = RB_SCAN_WARPS * (32 / RB_LANES) * RB_COLS;      // 16 columns
+constexpr int RB_THREADS = 32 * (RB_SCAN_WARPS + RB_BLOCKS);
+constexpr int RB_SCALARS = 16 + 16 + 4 + RB_BLOCK * RB_TILE + 4;        // A [4][4], B [4][4], beta [4], v [4][RB_TILE], padding
+
+struct RowScan {
+    const float* q;             // float32 rows of row_stride numbers: query/key head g at + g * D, value head h at + h * V
+    const float* k;
+    const float* v;
+    size_t row_stride;
+    const float* decay;         // [tokens][heads * D]
+    const float* proj;          // delta rule: column b_col + h of the partial sums is the raw write strength
+    int splits, cols, b_col;
+    size_t split_stride;
+    float q_scale;
+    float* state;               // [slots][heads][V][D]
+    float* out;                 // [tokens][heads * V]
+    const int* cu;
+    const int* slots;
+    int heads, qk_heads, D, V, vec;
+};
+
+__device__ __forceinline__ float rb_pick(const float (&a)[4], int i) { return i < 2 ? (i ? a[1] : a[0]) : (i == 2 ? a[2] : a[3]); }
+
+// v[i], i < N, summed over N neighbouring lanes: lane l of the N ends up with the sum of v[l] (N a power of two)
+template <int N>
+__device__ __forceinline__ float rb_scatter_sum(float (&v)[N], int lane) {
+#pragma unroll
+    for (int o = N / 2; o > 0; o >>= 1) {
+        const bool hi = lane & o;
+#pragma unroll
+        for (int i = 0; i < o; ++i) {
+            const float send = hi ? v[i] : v[i + o], keep = hi ? v[i + o] : v[i];
+            v[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+        }
+    }
+    return v[0];
+}
+
+// two bits a value: the (t, j) of the pair products, first A's (1,0) (2,0) (2,1) (3,0) (3,1) (3,2), then B's (0,0) (1,0) (1,1) ... (3,3)
+constexpr uint32_t RB_T = 1u | 2u << 2 | 2u << 4 | 3u << 6 | 3u << 8 | 3u << 10 | 0u << 12 | 1u << 14 | 1u << 16 | 2u << 18 | 2u << 20 | 2u << 22 | 3u << 24 | 3u << 26 | 3u << 28 | 3u << 30;
+constexpr uint32_t RB_J = 0u | 0u << 2 | 1u << 4 | 0u << 6 | 1u << 8 | 2u << 10 | 0u << 12 | 0u << 14 | 1u << 16 | 0u << 18 | 1u << 20 | 2u << 22 | 0u << 24 | 1u << 26 | 2u << 28 | 3u << 30;
+
+template <int K, bool DELTA>
+__global__ void __launch_bounds__(RB_THREADS)
+row_decay_blocks_kernel(const RowScan a) {
+    tt_pdl_launch_dependents();
+    tt_pdl_wait();
+    extern __shared__ __align__(16) float rec_shared[];
+    constexpr int DP = K * RB_LANES, E = DP / 32;               // rows padded to DP numbers; E of them in a preparing lane
+    constexpr int VECTORS = (DELTA ? 3 : 2) * RB_BLOCK + 1;     // (P_t k_t) [4], P_t q_t [4], s_(j,3) k_j [4], P_3
+    constexpr int BLOCK_FLOATS = VECTORS * DP + RB_SCALARS, BUFFER = RB_BLOCKS * BLOCK_FLOATS;
+    constexpr int Q_AT = DELTA ? RB_BLOCK * DP : 0, KH_AT = Q_AT + RB_BLOCK * DP, P_AT = KH_AT + RB_BLOCK * DP, S_AT = VECTORS * DP;
+    const int h = blockIdx.x, b = blockIdx.y, p0 = blockIdx.z * RB_TILE;
+    const int first = a.cu[b], n = a.cu[b + 1] - first;
+    if (n <= 0) return;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int D = a.D, V = a.V;
+    const int chunks = (n + RB_CHUNK - 1) / RB_CHUNK;
+    for (int e = threadIdx.x; e < 2 * BUFFER; e += RB_THREADS) rec_shared[e] = 0.0f;
+    __syncthreads();
+
+    if (warp >= RB_SCAN_WARPS) {
+        // ------------------------------------------------------------ a block of four tokens prepared by a warp
+        const int mine = warp - RB_SCAN_WARPS, g = h / (a.heads / a.qk_heads);
+        auto row_of = [&](int e) { return E == 8 ? 4 * lane + 128 * (e >> 2) + (e & 3) : E * lane + e; };
+        float q[4][E], k[4][E], d[4][E], v[2], raw = 0.0f;
+        const int v_token = lane >> 3, v_col = 2 * (lane & 7);
+        auto load_row = [&](float (&x)[E], const float* row, float missing, bool live) {
+            constexpr int W = E < 4 ? E : 4;                    // numbers of a load
+#pragma unroll
+            for (int j = 0; j < E; j += W) {
+                const int r = row_of(j);
+                if (live && a.vec && r < D) {
+                    if constexpr (W == 4) {
+                        const float4 y = __ldg(reinterpret_cast<const float4*>(row + r));
+                        x[j] = y.x; x[j + 1] = y.y; x[j + 2] = y.z; x[j + 3] = y.w;
+                    } else {
+                        const float2 y = __ldg(reinterpret_cast<const float2*>(row + r));
+                        x[j] = y.x; x[j + 1] = y.y;
+                    }
+                } else {
+#pragma unroll
+                    for (int e = 0; e < W; ++e) x[j + e] = live && r + e < D ? __ldg(row + r + e) : missing;
+                }
+            }
+        };
+        auto fetch = [&](int c0) {
+            const int t0 = c0 + mine * RB_BLOCK;
+#pragma unroll
+            for (int t = 0; t < 4; ++t) {
+                const bool live = t0 + t < n;
+                const size_t row = (size_t)(first + (live ? t0 + t : 0));
+                load_row(q[t], a.q + row * a.row_stride + (size_t)g * D, 0.0f, live);
+                load_row(k[t], a.k + row * a.row_stride + (size_t)g * D, 0.0f, live);
+                load_row(d[t], a.decay + (row * a.heads + h) * D, 1.0f, live);
+            }
+            const bool live = t0 + v_token < n;
+            const float* vr = a.v + (size_t)(first + t0 + v_token) * a.row_stride + (size_t)h * V + p0 + v_col;
+            v[0] = live && p0 + v_col < V ? __ldg(vr) : 0.0f;
+            v[1] = live && p0 + v_col + 1 < V ? __ldg(vr + 1) : 0.0f;
+            if (DELTA && lane < 4 && t0 + lane < n)
+                raw = rec_sum_slices(a.proj + (size_t)(first + t0 + lane) * a.cols + a.b_col + h, a.splits, a.split_stride);
+        };
+        fetch(0);
+        for (int it = 0; it <= chunks; ++it) {
+            if (it < chunks) {
+                const int t0 = it * RB_CHUNK + mine * RB_BLOCK;
+                float* base = rec_shared + (it & 1) * BUFFER + mine * BLOCK_FLOATS;
+                constexpr int PAIRS = DELTA ? 32 : 16, A_AT = 8, B_AT = DELTA ? 14 : 0;
+                float sums[PAIRS];                              // delta rule: |q_t|^2 [4], |k_t|^2 [4], A's six, B's ten; else B's ten
+#pragma unroll
+                for (int i = 0; i < PAIRS; ++i) sums[i] = 0.0f;
+                float kh[4][E];
+#pragma unroll
+                for (int e = 0; e < E; ++e) {
+                    if (DELTA) {
+#pragma unroll
+                        for (int t = 0; t < 4; ++t) {
+                            sums[t] = fmaf(q[t][e], q[t][e], sums[t]);
+                            sums[4 + t] = fmaf(k[t][e], k[t][e], sums[4 + t]);
+                        }
+                    }
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {
+                        float w = k[j][e];
+                        sums[B_AT + j * (j + 1) / 2 + j] = fmaf(q[j][e], w, sums[B_AT + j * (j + 1) / 2 + j]);
+#pragma unroll
+                        for (int t = j + 1; t < 4; ++t) {
+                            w *= d[t][e];
+                            if (DELTA) sums[A_AT + t * (t - 1) / 2 + j] = fmaf(k[t][e], w, sums[A_AT + t * (t - 1) / 2 + j]);
+                            sums[B_AT + t * (t + 1) / 2 + j] = fmaf(q[t][e], w, sums[B_AT + t * (t + 1) / 2 + j]);
+                        }
+                        kh[j][e] = w;
+                    }
+                }
+                float total = rb_scatter_sum<PAIRS>(sums, lane);
+                float nq[4], nk[4], beta[4];
+#pragma unroll
+                for (int t = 0; t < 4; ++t) {
+                    if (DELTA) {
+                        nq[t] = rsqrtf(__shfl_sync(0xffffffffu, total, t) + 1e-6f) * a.q_scale;
+                        nk[t] = rsqrtf(__shfl_sync(0xffffffffu, total, 4 + t) + 1e-6f);
+                        beta[t] = t0 + t < n ? 1.0f / (1.0f + expf(-__shfl_sync(0xffffffffu, raw, t))) : 0.0f;
+                    } else {
+                        nq[t] = a.q_scale;
+                        nk[t] = beta[t] = 1.0f;
+                    }
+                }
+                if (!DELTA) total += __shfl_xor_sync(0xffffffffu, total, 16);
+                const int pair = DELTA ? lane - 8 : lane + 6;   // its place among the 16 pairs
+                if (pair >= (DELTA ? 0 : 6) && pair < 16) {
+                    const int t = (RB_T >> (2 * pair)) & 3, j = (RB_J >> (2 * pair)) & 3;
+                    const float into = pair < 6 ? rb_pick(beta, t) * rb_pick(nk, t) : rb_pick(nq, t);
+                    base[S_AT + (pair < 6 ? 0 : 16) + t * 4 + j] = total * into * rb_pick(nk, j);
+                }
+                if (DELTA && lane < 4) base[S_AT + 32 + lane] = rb_pick(beta, lane);
+                *reinterpret_cast<float2*>(base + S_AT + 36 + v_token * RB_TILE + v_col) = make_float2(v[0] * rb_pick(beta, v_token), v[1] * rb_pick(beta, v_token));
+                float p[E];
+#pragma unroll
+                for (int e = 0; e < E; ++e) p[e] = 1.0f;
+                auto put = [&](float* to, const float (&x)[E]) {
+                    constexpr int W = E < 4 ? E : 4;
+#pragma unroll
+                    for (int j = 0; j < E; j += W) {
+                        if constexpr (W == 4) *reinterpret_cast<float4*>(to + row_of(j)) = make_float4(x[j], x[j + 1], x[j + 2], x[j + 3]);
+                        else *reinterpret_cast<float2*>(to + row_of(j)) = make_float2(x[j], x[j + 1]);
+                    }
+                };
+#pragma unroll
+                for (int t = 0; t < 4; ++t) {
+                    float x[E];
+#pragma unroll
+                    for (int e = 0; e < E; ++e) { p[e] *= d[t][e]; x[e] = q[t][e] * p[e] * nq[t]; }
+                    put(base + Q_AT + t * DP, x);
+                    if (DELTA) {
+#pragma unroll
+                        for (int e = 0; e < E; ++e) x[e] = k[t][e] * p[e] * nk[t];
+                        put(base + t * DP, x);
+                    }
+#pragma unroll
+                    for (int e = 0; e < E; ++e) x[e] = kh[t][e] * nk[t];
+                    put(base + KH_AT + t * DP, x);
+                }
+                put(base + P_AT, p);
+                if (it + 1 < chunks) fetch((it + 1) * RB_CHUNK);          // lands while the others walk
+            }
+            __syncthreads();
+        }
+        return;
+    }
+
+    // ---------------------------------------------------------------- the state, walked through the prepared blocks
+    const int l = lane & (RB_LANES - 1);
+    const int col = (warp * (32 / RB_LANES) + lane / RB_LANES) * RB_COLS;          // first of this lane group's columns in the tile
+    float* S = a.state + (((size_t)a.slots[b] * a.heads + h) * V + p0 + col) * D;
+    float s[RB_COLS][K];
+    auto state_row = [&](int i) { return 4 * l + 4 * RB_LANES * (i >> 2) + (i & 3); };
+#pragma unroll
+    for (int c = 0; c < RB_COLS; ++c)
+#pragma unroll
+        for (int i = 0; i < K; i += 4) {
+            const int r = state_row(i);
+            const bool live = p0 + col + c < V;
+            if (live && !(D & 3) && r < D) {
+                const float4 y = *reinterpret_cast<const float4*>(S + (size_t)c * D + r);
+                s[c][i] = y.x; s[c][i + 1] = y.y; s[c][i + 2] = y.z; s[c][i + 3] = y.w;
+            } else {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) s[c][i + e] = live && r + e < D ? S[(size_t)c * D + r + e] : 0.0f;
+            }
+        }
+    __syncthreads();                                            // the first chunk is prepared
+    for (int it = 1; it <= chunks; ++it) {
+        const float* buffer = rec_shared + ((it - 1) & 1) * BUFFER;
+        const int left = n - (it - 1) * RB_CHUNK;
+        for (int blk = 0; blk < RB_BLOCKS && blk * RB_BLOCK < left; ++blk) {
+            const float* base = buffer + blk * BLOCK_FLOATS;
+            constexpr int DOTS = DELTA ? 16 : 8;                // [keys, queries][column][token], or [column][token]
+            float dots[DOTS];
+#pragma unroll
+            for (int i = 0; i < DOTS; ++i) dots[i] = 0.0f;
+#pragma unroll
+            for (int i = 0; i < K; i += 4) {
+#pragma unroll
+                for (int t = 0; t < 4; ++t) {
+                    const float4 y = *reinterpret_cast<const float4*>(base + Q_AT + t * DP + state_row(i));
+#pragma unroll
+                    for (int c = 0; c < RB_COLS; ++c) {
+                        float& o = dots[(DELTA ? 8 : 0) + c * 4 + t];
+                        o = fmaf(s[c][i], y.x, o); o = fmaf(s[c][i + 1], y.y, o); o = fmaf(s[c][i + 2], y.z, o); o = fmaf(s[c][i + 3], y.w, o);
+                    }
+                    if (DELTA) {
+                        const float4 z = *reinterpret_cast<const float4*>(base + t * DP + state_row(i));
+#pragma unroll
+                        for (int c = 0; c < RB_COLS; ++c) {
+                            float& o = dots[c * 4 + t];
+                            o = fmaf(s[c][i], z.x, o); o = fmaf(s[c][i + 1], z.y, o); o = fmaf(s[c][i + 2], z.z, o); o = fmaf(s[c][i + 3], z.w, o);
+                        }
+                    }
+                }
+            }
+            float dot = rb_scatter_sum<DOTS>(dots, l);
+            if (!DELTA) dot += __shfl_xor_sync(0xffffffffu, dot, 8);
+            const float* scalars = base + S_AT;
+            float u[RB_COLS][4];
+#pragma unroll
+            for (int t = 0; t < 4; ++t) {
+                const float2 y = *reinterpret_cast<const float2*>(scalars + 36 + t * RB_TILE + col);
+                u[0][t] = y.x; u[1][t] = y.y;
+            }
+            if (DELTA) {
+                const float4 beta = *reinterpret_cast<const float4*>(scalars + 32);
+                const float4 a1 = *reinterpret_cast<const float4*>(scalars + 4), a2 = *reinterpret_cast<const float4*>(scalars + 8), a3 = *reinterpret_cast<const float4*>(scalars + 12);
+#pragma unroll
+                for (int c = 0; c < RB_COLS; ++c) {
+                    float r[4];
+#pragma unroll
+                    for (int t = 0; t < 4; ++t) r[t] = __shfl_sync(0xffffffffu, dot, c * 4 + t, RB_LANES);
+                    u[c][0] = fmaf(-beta.x, r[0], u[c][0]);
+                    u[c][1] = fmaf(-a1.x, u[c][0], fmaf(-beta.y, r[1], u[c][1]));
+                    u[c][2] = fmaf(-a2.y, u[c][1], fmaf(-a2.x, u[c][0], fmaf(-beta.z, r[2], u[c][2])));
+                    u[c][3] = fmaf(-a3.z, u[c][2], fmaf(-a3.y, u[c][1], fmaf(-a3.x, u[c][0], fmaf(-beta.w, r[3], u[c][3]))));
+                }
+            }
+            {                                                   // the lane that holds a query's row product writes its token's output
+                const int t = l & 3, c = (l >> 2) & 1, token = (it - 1) * RB_CHUNK + blk * RB_BLOCK + t;
+                const float4 w = *reinterpret_cast<const float4*>(scalars + 16 + 4 * t);
+                float o = dot;
+                o = fmaf(w.x, c ? u[1][0] : u[0][0], o);
+                o = fmaf(w.y, c ? u[1][1] : u[0][1], o);
+                o = fmaf(w.z, c ? u[1][2] : u[0][2], o);
+                o = fmaf(w.w, c ? u[1][3] : u[0][3], o);
+                if ((l >= 8) == DELTA && token < n && p0 + col + c < V) a.out[(size_t)(first + token) * (a.heads * V) + (size_t)h * V + p0 + col + c] = o;
+            }
+#pragma unroll
+            for (int i = 0; i < K; i += 4) {
+                const float4 p = *reinterpret_cast<const float4*>(base + P_AT + state_row(i));
+#pragma unroll
+                for (int c = 0; c < RB_COLS; ++c) { s[c][i] *= p.x; s[c][i + 1] *= p.y; s[c][i + 2] *= p.z; s[c][i + 3] *= p.w; }
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    const float4 y = *reinterpret_cast<const float4*>(base + KH_AT + j * DP + state_row(i));
+#pragma unroll
+                    for (int c = 0; c < RB_COLS; ++c) {
+                        s[c][i] = fmaf(y.x, u[c][j], s[c][i]);
+                        s[c][i + 1] = fmaf(y.y, u[c][j], s[c][i + 1]);
+                        s[c][i + 2] = fmaf(y.z, u[c][j], s[c][i + 2]);
+                        s[c][i + 3] = fmaf(y.w, u[c][j], s[c][i + 3]);
+                    }
+                }
+            }
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int c = 0; c < RB_COLS; ++c)
+#pragma unroll
+        for (int i = 0; i < K; i += 4) {
+            const int r = state_row(i);
+            if (p0 + col + c >= V) continue;
+            if (!(D & 3) && r < D) {
+                *reinterpret_cast<float4*>(S + (size_t)c * D + r) = make_float4(s[c][i], s[c][i + 1], s[c][i + 2], s[c][i + 3]);
+            } else {
+#pragma unroll
+                for (int e = 0; e < 4; ++e)
+                    if (r + e < D) S[(size_t)c * D + r + e] = s[c][i + e];
+            }
+        }
+}
+
+template <int K, bool DELTA>
+static int row_decay_blocks_launch(const RowScan& scan, int sequences, cudaStream_t stream) {
+    constexpr size_t shared = (size_t)2 * RB_BLOCKS * (((DELTA ? 3 : 2) * RB_BLOCK + 1) * K * RB_LANES + RB_SCALARS) * sizeof(float);
+    static bool allowed = false;
+    if (!allowed) {
+        const cudaError_t code = cudaFuncSetAttribute(row_decay_blocks_kernel<K, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
+        if (code != cudaSuccess) return (int)code;
+        allowed = true;
+    }
+    tt_launch_pdl(row_decay_blocks_kernel<K, DELTA>, dim3(scan.heads, sequences, (scan.V + RB_TILE - 1) / RB_TILE), dim3(RB_THREADS), shared, stream, scan);
+    TT_LAUNCH_CHECK();
+}
+
+// delta != 0: the delta rule (q and k are made unit vectors, q also times q_scale; beta from proj); else linear attention (q times q_scale)
+extern "C" int tt_row_decay_blocks(const float* q, const float* k, const float* v, long long row_stride, const float* decay, int delta,
+                                   const float* proj, int splits, long long split_stride, int cols, int b_col, float q_scale, float* state,
+                                   float* out, const int* cu, const int* slots, int sequences, int heads, int qk_heads, int D, int V,
+                                   cudaStream_t stream) {
+    if (sequences <= 0) return 0;
+    if (!q || !k || !v || !decay || D <= 0 || D > REC_MAX_ROWS || V <= 0 || qk_heads <= 0 || heads % qk_heads || sequences > 65535) return (int)cudaErrorInvalidValue;
+    if (delta && !proj) return (int)cudaErrorInvalidValue;
+    const uintptr_t bases = (uintptr_t)q | (uintptr_t)k | (uintptr_t)decay;
+    const RowScan scan{q, k, v, (size_t)row_stride, decay, proj, splits, cols, b_col, (size_t)split_stride, q_scale, state, out, cu, slots,
+                       heads, qk_heads, D, V, (bases & 15) == 0 && !(D & 3) && !(row_stride & 3) ? 1 : 0};
+    if (D <= 4 * RB_LANES) return delta ? row_decay_blocks_launch<4, true>(scan, sequences, stream) : row_decay_blocks_launch<4, false>(scan, sequences, stream);
+    if (D <= 8 * RB_LANES) return delta ? row_decay_blocks_launch<8, true>(scan, sequences, stream) : row_decay_blocks_launch<8, false>(scan, sequences, stream);
+    return delta ? row_decay_blocks_launch<16, true>(scan, sequences, stream) : row_decay_blocks_launch<16, false>(scan, sequences, stream);
+}
+
+// ------------------------------------------------------------------------------------
 // Products of low rank: z[t, j] = sum_r W[j, r] * x[t, r] with x the columns x_col .. x_col + rank - 1 of a projection's
 // partial sums, and what is made of z at once (kind):
 //   0: z      1: exp(-exp(a_log[h]) * softplus(z + bias[j])), h = j / per_head      2: sigmoid(z + bias[j]) ^ inv_tau
@@ -702,12 +1064,22 @@ struct LowRankPart {
     float* out;                 // float32 [tokens][n]
 };
 struct LowRankParts { LowRankPart part[2]; };
-constexpr int LR_THREADS = 128, LR_RANKS = 128;       // ranks staged at a time
+constexpr int LR_THREADS = 256, LR_RANKS = 128;       // ranks staged at a time
 
 __device__ __forceinline__ float low_rank_finish(const LowRankPart& p, float z, int j) {
     if (p.kind == 1) return expf(-expf(__ldg(p.a_log + j / p.per_head)) * rec_softplus(z + __ldg(p.bias + j)));
     if (p.kind == 2) return expf(-rec_softplus(-(z + __ldg(p.bias + j))) * p.inv_tau);
     return z;
+}
+
+__device__ __forceinline__ void low_rank_pair(const float* p, float& a, float& b) {
+    const float2 v = __ldg(reinterpret_cast<const float2*>(p));
+    a = v.x; b = v.y;
+}
+__device__ __forceinline__ void low_rank_pair(const __nv_bfloat16* p, float& a, float& b) {
+    const uint32_t raw = __ldg(reinterpret_cast<const uint32_t*>(p));
+    const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw));
+    a = v.x; b = v.y;
 }
 
 template <typename TW, int TT, int RG>
@@ -724,6 +1096,7 @@ low_rank_kernel(const float* __restrict__ proj, int splits, size_t split_stride,
     const int group = threadIdx.x / LANES, lane = threadIdx.x - group * LANES;
     const int j = j0 + 2 * lane;
     const TW* w = reinterpret_cast<const TW*>(p.w);
+    const bool paired = !(p.n & 1) && j < p.n;                  // the two columns' weights lie on a pair's boundary
     float acc[TT][2];
 #pragma unroll
     for (int t = 0; t < TT; ++t) acc[t][0] = acc[t][1] = 0.0f;
@@ -731,6 +1104,7 @@ low_rank_kernel(const float* __restrict__ proj, int splits, size_t split_stride,
     for (int r0 = 0; r0 < p.rank; r0 += LR_RANKS) {
         const int ranks = min(LR_RANKS, p.rank - r0);
         if (r0) __syncthreads();
+#pragma unroll 8                                                         // loads in flight together
         for (int e = threadIdx.x; e < TT * ranks; e += LR_THREADS) {
             const int t = e / ranks, r = e - t * ranks;
             xs[r * STRIDE + t] = t < count ? rec_sum_slices(proj + (size_t)(t0 + t) * cols + p.x_col + r0 + r, splits, split_stride) : 0.0f;
@@ -738,8 +1112,13 @@ low_rank_kernel(const float* __restrict__ proj, int splits, size_t split_stride,
         __syncthreads();
 #pragma unroll 4
         for (int r = group; r < ranks; r += RG) {
-            const size_t at = (size_t)(r0 + r) * p.n + j;
-            const float w0 = j < p.n ? tt_to_float(w[at]) : 0.0f, w1 = j + 1 < p.n ? tt_to_float(w[at + 1]) : 0.0f;
+            const TW* at = w + (size_t)(r0 + r) * p.n + j;
+            float w0 = 0.0f, w1 = 0.0f;
+            if (paired) low_rank_pair(at, w0, w1);
+            else {
+                if (j < p.n) w0 = tt_to_float(at[0]);
+                if (j + 1 < p.n) w1 = tt_to_float(at[1]);
+            }
             const float4* x4 = reinterpret_cast<const float4*>(xs + r * STRIDE);
 #pragma unroll
             for (int q = 0; q < TT / 4; ++q) {
@@ -795,16 +1174,16 @@ extern "C" int tt_low_rank(const float* proj, int splits, long long split_stride
     for (int i = 0; i < n_parts; ++i) {
         const LowRankPart& p = parts.part[i];
         if (p.rank < 1 || p.n < 1 || p.x_col < 0 || p.x_col + p.rank > cols || p.kind < 0 || p.kind > 2) return (int)cudaErrorInvalidValue;
-        if ((p.kind && !p.bias) || (p.kind == 1 && (!p.a_log || p.per_head < 1)) || ((uintptr_t)p.out & 7)) return (int)cudaErrorInvalidValue;
+        if ((p.kind && !p.bias) || (p.kind == 1 && (!p.a_log || p.per_head < 1)) || ((uintptr_t)p.out & 7) || ((uintptr_t)p.w & 7)) return (int)cudaErrorInvalidValue;
         widest = p.n > widest ? p.n : widest;
     }
     const bool few = n_tokens <= LR_FEW_TOKENS;
-    const int tile = few ? 8 : 32, columns = 2 * LR_THREADS / (few ? 4 : 1);
+    const int tile = few ? 8 : 32, columns = 2 * LR_THREADS / (few ? 8 : 1);
     const dim3 grid((n_tokens + tile - 1) / tile, (widest + columns - 1) / columns, n_parts);
     if (grid.y > 65535) return (int)cudaErrorInvalidValue;
 #define TT_LOW_RANK(T, TT, RG) tt_launch_pdl(low_rank_kernel<T, TT, RG>, grid, dim3(LR_THREADS), 0, stream, proj, splits, (size_t)split_stride, cols, parts, n_tokens)
-    if (w_dtype == TT_F32) { if (few) TT_LOW_RANK(float, 8, 4); else TT_LOW_RANK(float, 32, 1); }
-    else { if (few) TT_LOW_RANK(__nv_bfloat16, 8, 4); else TT_LOW_RANK(__nv_bfloat16, 32, 1); }
+    if (w_dtype == TT_F32) { if (few) TT_LOW_RANK(float, 8, 8); else TT_LOW_RANK(float, 32, 1); }
+    else { if (few) TT_LOW_RANK(__nv_bfloat16, 8, 8); else TT_LOW_RANK(__nv_bfloat16, 32, 1); }
 #undef TT_LOW_RANK
     TT_LAUNCH_CHECK();
 }

@@ -920,6 +920,35 @@ def row_decay_scan(vkq: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, 
               SCAN_FORMS[form], _stream()), "row_decay_scan")
 
 
+def row_decay_blocks(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, out: torch.Tensor,
+                     cu: torch.Tensor, slots: torch.Tensor, sequences: int, heads: int, qk_heads: int, key_dim: int, value_dim: int,
+                     q_scale: float, write: tuple[torch.Tensor, int] | None = None) -> None:
+    """The recurrences with a decay per head and key channel, four tokens at a time (for prompts; token by token they are
+    :func:`delta_scan` with ``row_decay`` and :func:`row_decay_scan`).  ``q``, ``k``, ``v``: float32 ``[tokens, columns]`` of
+    ``qk_heads * key_dim`` and ``heads * value_dim`` columns, views of one matrix (equal row strides).  ``write`` = (projection
+    partial sums, first column of the raw write strengths): the delta rule, which makes q and k unit vectors; without it: linear
+    attention.  q is multiplied by ``q_scale``."""
+    for t, cols, name in ((q, qk_heads * key_dim, "q"), (k, qk_heads * key_dim, "k"), (v, heads * value_dim, "v")):
+        if t.dtype != torch.float32 or t.dim() != 2 or t.stride(1) != 1 or t.stride(0) != q.stride(0) or t.shape[1] != cols:
+            raise KernelError(f"row_decay_blocks: {name} must be float32 [tokens, {cols}] with the row stride of q")
+    for t, name in ((decay, "decays"), (state, "recurrent state"), (out, "recurrence output")):
+        _need(t, torch.float32, name)
+    if (tuple(decay.shape) != (q.shape[0], heads * key_dim) or tuple(state.shape[1:]) != (heads, value_dim, key_dim)
+            or tuple(out.shape) != (q.shape[0], heads * value_dim)):
+        raise KernelError("row_decay_blocks: shapes do not fit the sizes")
+    p, splits, stride, cols, b_col = c_void_p(0), 0, 0, 0, 0
+    if write is not None:
+        p, splits, stride, cols = _projection(write[0])
+        b_col = int(write[1])
+        if b_col < 0 or b_col + heads > cols:
+            raise KernelError("row_decay_blocks: the write strengths lie outside the projection")
+    fn = _fn("recurrent", "tt_row_decay_blocks", [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_int, c_longlong, c_int,
+                                                  c_int, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
+                                                  c_void_p])
+    _check(fn(_ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(decay), 0 if write is None else 1, p, splits, stride, cols, b_col, q_scale,
+              _ptr(state), _ptr(out), _ptr(cu), _ptr(slots), sequences, heads, qk_heads, key_dim, value_dim, _stream()), "row_decay_blocks")
+
+
 @dataclass(frozen=True)
 class LowRank:
     """One product of :func:`low_rank`: ``z = W x`` with x the ``rank`` columns of a projection from ``col`` on and ``weight`` the

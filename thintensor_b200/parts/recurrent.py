@@ -67,6 +67,12 @@ def _low_rank_up(tensors, down: str, up: str) -> torch.Tensor:
     return tensors[up].t().contiguous()
 
 
+def _in_blocks(ctx) -> bool:
+    """Whether a recurrence with decays per channel takes its tokens four at a time: prompts do (decided by the step's
+    shape alone, so a replayed step and the step it was captured from agree)."""
+    return not ctx.decode and ctx.n_tokens >= 4 * ctx.sequences
+
+
 @MIXERS.register("mamba2")
 class Mamba2(Mixer):
     NAMES = {"in": "in_proj.weight", "conv": "conv1d.weight", "conv_bias": "conv1d.bias", "dt_bias": "dt_bias", "A_log": "A_log",
@@ -234,8 +240,12 @@ class GatedDelta(Mixer):
         qkv = ctx.scratch("delta.qkv", (tokens, self.channels), torch.float32)
         api.causal_conv(proj, 0, self.channels, self.conv_weight, None, True, tail, qkv, ctx.cu, ctx.slots, ctx.sequences, tokens, ctx.decode)
         read = ctx.scratch("delta.read", (tokens, self.v), torch.float32)
-        api.delta_scan(qkv, proj, self.b_col, self.a_col, self.dt_bias, self.a_log, recurrent, read, ctx.cu,
-                       ctx.slots, ctx.sequences, self.heads, self.qk_heads, self.key_dim, self.value_dim, row_decay=decay)
+        if decay is not None and _in_blocks(ctx):
+            api.row_decay_blocks(qkv[:, :self.qk], qkv[:, self.qk: 2 * self.qk], qkv[:, 2 * self.qk:], decay, recurrent, read, ctx.cu, ctx.slots,
+                                 ctx.sequences, self.heads, self.qk_heads, self.key_dim, self.value_dim, self.key_dim ** -0.5, (proj, self.b_col))
+        else:
+            api.delta_scan(qkv, proj, self.b_col, self.a_col, self.dt_bias, self.a_log, recurrent, read, ctx.cu,
+                           ctx.slots, ctx.sequences, self.heads, self.qk_heads, self.key_dim, self.value_dim, row_decay=decay)
         gated = ctx.scratch("delta.gated", (tokens, self.v))
         api.gated_group_norm(read, self.value_dim, gate_source, gate_col, self.norm, self.eps, False, gated, self.gate)
         return self.out.delta(ctx, gated, "delta.out")
@@ -334,19 +344,35 @@ class DecayLinearAttention(Mixer):
         (recurrent,) = states
         tokens = ctx.n_tokens
         proj = self.proj(ctx, x, "linear_attention.in")
-        vkq = ctx.scratch("linear_attention.vkq", (tokens, self.v + 2 * self.qk), torch.float32)
         rotary_dim = self.rot.rotary_dim if self.rot is not None else 0
-        api.linear_attention_prepare(proj, self.heads, self.key_dim, self.value_dim, self.activation == "silu",
-                                     self.rot.inv_freq if rotary_dim else None, rotary_dim, self.key_scale, vkq, ctx.cu, ctx.len_before,
-                                     ctx.sequences, tokens, self.query_scale)
         read = ctx.scratch("linear_attention.read", (tokens, self.v), torch.float32)
+        decay = None
         if self.decay_up is not None:
             decay = ctx.scratch("linear_attention.decay", (tokens, self.qk), torch.float32)
             api.low_rank(proj, [api.LowRank(2 * self.qk + 2 * self.v, self.decay_up, decay, "sigmoid_root", self.decay_bias, tau=self.tau)])
+        blocks = decay is not None and _in_blocks(ctx)
+        if blocks and proj.shape[0] == 1 and not rotary_dim and self.activation is None and self.key_scale == 1.0:
+            q, k, v = proj[0].split((self.qk, self.qk, self.v, proj.shape[2] - 2 * self.qk - self.v), dim=1)[:3]     # the product as it is
+            api.row_decay_blocks(q, k, v, decay, recurrent, read, ctx.cu, ctx.slots, ctx.sequences, self.heads, self.heads, self.key_dim,
+                                 self.value_dim, self.query_scale)
+            return self.finish(ctx, proj, read)
+        vkq = ctx.scratch("linear_attention.vkq", (tokens, self.v + 2 * self.qk), torch.float32)
+        api.linear_attention_prepare(proj, self.heads, self.key_dim, self.value_dim, self.activation == "silu",
+                                     self.rot.inv_freq if rotary_dim else None, rotary_dim, self.key_scale, vkq, ctx.cu, ctx.len_before,
+                                     ctx.sequences, tokens, self.query_scale)
+        if blocks:
+            v, k, q = vkq.split((self.v, self.qk, self.qk), dim=1)
+            api.row_decay_blocks(q, k, v, decay, recurrent, read, ctx.cu, ctx.slots, ctx.sequences, self.heads, self.heads, self.key_dim,
+                                 self.value_dim, 1.0)
+        elif decay is not None:
             api.row_decay_scan(vkq, decay, recurrent, read, ctx.cu, ctx.slots, ctx.sequences, self.heads, self.key_dim, self.value_dim)
         else:
             api.decay_scan(vkq, self.decays, recurrent, read, ctx.cu, ctx.slots, ctx.sequences, self.heads, self.key_dim, self.value_dim)
-        gated = ctx.scratch("linear_attention.gated", (tokens, self.v))
+        return self.finish(ctx, proj, read)
+
+    def finish(self, ctx, proj, read) -> Delta:
+        """Norm and gate of the read-out, output projection."""
+        gated = ctx.scratch("linear_attention.gated", (ctx.n_tokens, self.v))
         api.gated_group_norm(read, self.v if self.norm == "all" else self.value_dim, proj, 2 * self.qk + self.v, self.norm_w, self.eps,
                              False, gated, self.gate)
         return self.out.delta(ctx, gated, "linear_attention.out")
