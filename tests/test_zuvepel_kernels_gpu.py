@@ -77,7 +77,7 @@ def test_branches_addend_and_two_norms(rows, hidden, out_dtype, a_splits, b_spli
 
 
 # ------------------------------------------------------------------------------- low rank
-@pytest.mark.parametrize("tokens", [1, 7, 9, 256, 300])
+@pytest.mark.parametrize("tokens", [1, 7, 9, 128, 300])
 @pytest.mark.parametrize("weights", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("splits,rank_a,heads,dim,rank_b,n_b", [(1, 16, 4, 24, 130, 66), (3, 5, 3, 7, 24, 77), (2, 129, 2, 136, 1, 600)])
 def test_low_rank_products(tokens, weights, splits, rank_a, heads, dim, rank_b, n_b):
@@ -105,6 +105,18 @@ def test_low_rank_products(tokens, weights, splits, rank_a, heads, dim, rank_b, 
     out_a.fill_(float("nan"))
     api.low_rank(proj, [api.LowRank(off, up_a, out_a, "sigmoid_root", bias.to(DEV), tau=tau)])
     assert float((out_a.double().cpu() - root).abs().max()) <= 2e-5
+    # the pieces of the form for many tokens
+    for dtype in (torch.float32, torch.bfloat16):
+        in_a, in_b = (torch.empty(tokens, n, dtype=dtype, device=DEV) for n in (rank_a, rank_b))
+        api.low_rank_inputs(proj, [(off, in_a), (off + rank_a + 2, in_b)])
+        for got, lo in ((in_a, off), (in_b, off + rank_a + 2)):
+            want = x[:, lo: lo + got.shape[1]]
+            assert float((got.double().cpu() - want).abs().max()) <= (1e-5 if dtype == torch.float32 else 5e-3) * float(want.abs().max())
+    product = slices((z - bias.double()).float(), splits, 30).to(DEV)
+    api.low_rank_finish(product, "delta_decay", bias.to(DEV), out_a, a_log.to(DEV), dim)
+    assert float((out_a.double().cpu() - delta).abs().max()) <= 2e-5
+    api.low_rank_finish(product, "sigmoid_root", bias.to(DEV), product[0], tau=tau)         # in place
+    assert float((product[0].double().cpu() - root).abs().max()) <= 2e-5
 
 
 # ---------------------------------------------------------------------------- recurrences

@@ -1052,8 +1052,7 @@ extern "C" int tt_row_decay_blocks(const float* q, const float* k, const float* 
 // partial sums, and what is made of z at once (kind):
 //   0: z      1: exp(-exp(a_log[h]) * softplus(z + bias[j])), h = j / per_head      2: sigmoid(z + bias[j]) ^ inv_tau
 // Up to two such products of one projection in one launch (blockIdx.z).  All float32; W is stored [rank][n] (transposed, so
-// that neighbouring threads read neighbouring numbers) in either element type.  A thread owns two neighbouring columns of TT
-// tokens; with few tokens RG thread groups share the rank among themselves and add up in shared memory.
+// that neighbouring threads read neighbouring numbers) in either element type.
 // ------------------------------------------------------------------------------------
 struct LowRankPart {
     int x_col, rank, n, kind, per_head;
@@ -1064,7 +1063,6 @@ struct LowRankPart {
     float* out;                 // float32 [tokens][n]
 };
 struct LowRankParts { LowRankPart part[2]; };
-constexpr int LR_THREADS = 256, LR_RANKS = 128;       // ranks staged at a time
 
 __device__ __forceinline__ float low_rank_finish(const LowRankPart& p, float z, int j) {
     if (p.kind == 1) return expf(-expf(__ldg(p.a_log + j / p.per_head)) * rec_softplus(z + __ldg(p.bias + j)));
@@ -1072,94 +1070,135 @@ __device__ __forceinline__ float low_rank_finish(const LowRankPart& p, float z, 
     return z;
 }
 
-__device__ __forceinline__ void low_rank_pair(const float* p, float& a, float& b) {
-    const float2 v = __ldg(reinterpret_cast<const float2*>(p));
-    a = v.x; b = v.y;
-}
-__device__ __forceinline__ void low_rank_pair(const __nv_bfloat16* p, float& a, float& b) {
-    const uint32_t raw = __ldg(reinterpret_cast<const uint32_t*>(p));
-    const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw));
-    a = v.x; b = v.y;
-}
+// Few tokens (decoding): a CTA takes LRF_TOKENS tokens and LRF_COLS columns, whose rank its eight warps share among
+// themselves.  The weights, which no kernel writes, are on their way to registers before the wait for the projection.
+constexpr int LRF_TOKENS = 8, LRF_COLS = 64, LRF_WARPS = 8, LRF_RANKS = 128, LRF_EACH = LRF_RANKS / LRF_WARPS, LRF_SLICES = 16;
 
-template <typename TW, int TT, int RG>
-__global__ void __launch_bounds__(LR_THREADS)
-low_rank_kernel(const float* __restrict__ proj, int splits, size_t split_stride, int cols, const LowRankParts parts, int n_tokens) {
-    constexpr int LANES = LR_THREADS / RG, STRIDE = TT + 4;          // rows padded: 16-byte reads, few bank conflicts on the writes
-    __shared__ __align__(16) float xs[LR_RANKS * STRIDE];
-    __shared__ float sums[RG > 1 ? (RG - 1) * TT * 2 * LANES : 1];
+template <typename TW>
+__global__ void __launch_bounds__(32 * LRF_WARPS)
+low_rank_few_kernel(const float* __restrict__ proj, int splits, size_t split_stride, int cols, const LowRankParts parts, int n_tokens) {
+    __shared__ __align__(16) float xs[LRF_RANKS * LRF_TOKENS];
+    __shared__ float sums[LRF_WARPS][LRF_TOKENS][LRF_COLS];
     tt_pdl_launch_dependents();
     const LowRankPart p = blockIdx.z ? parts.part[1] : parts.part[0];
-    const int j0 = blockIdx.y * 2 * LANES;
+    const int j0 = blockIdx.y * LRF_COLS;
     if (j0 >= p.n) return;
-    const int t0 = blockIdx.x * TT, count = min(TT, n_tokens - t0);
-    const int group = threadIdx.x / LANES, lane = threadIdx.x - group * LANES;
-    const int j = j0 + 2 * lane;
+    const int t0 = blockIdx.x * LRF_TOKENS, count = min(LRF_TOKENS, n_tokens - t0);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int ja = j0 + lane, jb = ja + 32;
     const TW* w = reinterpret_cast<const TW*>(p.w);
-    const bool paired = !(p.n & 1) && j < p.n;                  // the two columns' weights lie on a pair's boundary
-    float acc[TT][2];
+    TW wa[LRF_EACH], wb[LRF_EACH];
+    auto weights = [&](int r0) {
 #pragma unroll
-    for (int t = 0; t < TT; ++t) acc[t][0] = acc[t][1] = 0.0f;
+        for (int i = 0; i < LRF_EACH; ++i) {
+            const int r = r0 + warp + i * LRF_WARPS;
+            const TW* at = w + (size_t)r * p.n;
+            wa[i] = r < p.rank && ja < p.n ? at[ja] : tt_from_float<TW>(0.0f);
+            wb[i] = r < p.rank && jb < p.n ? at[jb] : tt_from_float<TW>(0.0f);
+        }
+    };
+    weights(0);
+    float acc[LRF_TOKENS][2];
+#pragma unroll
+    for (int t = 0; t < LRF_TOKENS; ++t) acc[t][0] = acc[t][1] = 0.0f;
     tt_pdl_wait();
-    for (int r0 = 0; r0 < p.rank; r0 += LR_RANKS) {
-        const int ranks = min(LR_RANKS, p.rank - r0);
-        if (r0) __syncthreads();
-#pragma unroll 8                                                         // loads in flight together
-        for (int e = threadIdx.x; e < TT * ranks; e += LR_THREADS) {
-            const int t = e / ranks, r = e - t * ranks;
-            xs[r * STRIDE + t] = t < count ? rec_sum_slices(proj + (size_t)(t0 + t) * cols + p.x_col + r0 + r, splits, split_stride) : 0.0f;
+    for (int r0 = 0; r0 < p.rank; r0 += LRF_RANKS) {
+        if (r0) { __syncthreads(); weights(r0); }
+        const int ranks = min(LRF_RANKS, p.rank - r0);
+#pragma unroll
+        for (int i = 0; i < LRF_RANKS * LRF_TOKENS / (32 * LRF_WARPS); ++i) {       // neighbouring threads: neighbouring ranks of one token
+            const int e = threadIdx.x + i * 32 * LRF_WARPS, t = e / LRF_RANKS, r = e % LRF_RANKS;
+            float total = 0.0f;
+            if (t < count && r < ranks) {
+                const float* from = proj + (size_t)(t0 + t) * cols + p.x_col + r0 + r;
+                for (int s0 = 0; s0 < splits; s0 += LRF_SLICES) {                  // the slices' loads in flight together, added in order
+                    float v[LRF_SLICES];
+#pragma unroll
+                    for (int s = 0; s < LRF_SLICES; ++s) v[s] = s0 + s < splits ? __ldg(from + (size_t)(s0 + s) * split_stride) : 0.0f;
+#pragma unroll
+                    for (int s = 0; s < LRF_SLICES; ++s) total += v[s];
+                }
+            }
+            xs[r * LRF_TOKENS + t] = total;
         }
         __syncthreads();
-#pragma unroll 4
-        for (int r = group; r < ranks; r += RG) {
-            const TW* at = w + (size_t)(r0 + r) * p.n + j;
-            float w0 = 0.0f, w1 = 0.0f;
-            if (paired) low_rank_pair(at, w0, w1);
-            else {
-                if (j < p.n) w0 = tt_to_float(at[0]);
-                if (j + 1 < p.n) w1 = tt_to_float(at[1]);
-            }
-            const float4* x4 = reinterpret_cast<const float4*>(xs + r * STRIDE);
 #pragma unroll
-            for (int q = 0; q < TT / 4; ++q) {
+        for (int i = 0; i < LRF_EACH; ++i) {
+            const float4* x4 = reinterpret_cast<const float4*>(xs + (warp + i * LRF_WARPS) * LRF_TOKENS);
+            const float a = tt_to_float(wa[i]), b = tt_to_float(wb[i]);
+#pragma unroll
+            for (int q = 0; q < LRF_TOKENS / 4; ++q) {
                 const float4 x = x4[q];
-                acc[4 * q][0] = fmaf(x.x, w0, acc[4 * q][0]);         acc[4 * q][1] = fmaf(x.x, w1, acc[4 * q][1]);
-                acc[4 * q + 1][0] = fmaf(x.y, w0, acc[4 * q + 1][0]); acc[4 * q + 1][1] = fmaf(x.y, w1, acc[4 * q + 1][1]);
-                acc[4 * q + 2][0] = fmaf(x.z, w0, acc[4 * q + 2][0]); acc[4 * q + 2][1] = fmaf(x.z, w1, acc[4 * q + 2][1]);
-                acc[4 * q + 3][0] = fmaf(x.w, w0, acc[4 * q + 3][0]); acc[4 * q + 3][1] = fmaf(x.w, w1, acc[4 * q + 3][1]);
+                acc[4 * q][0] = fmaf(x.x, a, acc[4 * q][0]);         acc[4 * q][1] = fmaf(x.x, b, acc[4 * q][1]);
+                acc[4 * q + 1][0] = fmaf(x.y, a, acc[4 * q + 1][0]); acc[4 * q + 1][1] = fmaf(x.y, b, acc[4 * q + 1][1]);
+                acc[4 * q + 2][0] = fmaf(x.z, a, acc[4 * q + 2][0]); acc[4 * q + 2][1] = fmaf(x.z, b, acc[4 * q + 2][1]);
+                acc[4 * q + 3][0] = fmaf(x.w, a, acc[4 * q + 3][0]); acc[4 * q + 3][1] = fmaf(x.w, b, acc[4 * q + 3][1]);
             }
         }
     }
-    if constexpr (RG > 1) {
-        if (group > 0) {
 #pragma unroll
-            for (int t = 0; t < TT; ++t)
+    for (int t = 0; t < LRF_TOKENS; ++t) { sums[warp][t][lane] = acc[t][0]; sums[warp][t][lane + 32] = acc[t][1]; }
+    __syncthreads();
+    for (int e = threadIdx.x; e < count * LRF_COLS; e += 32 * LRF_WARPS) {
+        const int t = e / LRF_COLS, c = e % LRF_COLS;
+        if (j0 + c >= p.n) continue;
+        float z = 0.0f;
 #pragma unroll
-                for (int c = 0; c < 2; ++c) sums[(((group - 1) * TT + t) * 2 + c) * LANES + lane] = acc[t][c];
-        }
-        __syncthreads();
-        if (group > 0) return;
-#pragma unroll
-        for (int g = 0; g < RG - 1; ++g)
-#pragma unroll
-            for (int t = 0; t < TT; ++t)
-#pragma unroll
-                for (int c = 0; c < 2; ++c) acc[t][c] += sums[((g * TT + t) * 2 + c) * LANES + lane];
-    }
-#pragma unroll
-    for (int t = 0; t < TT; ++t) {
-        if (t >= count) break;
-        float* o = p.out + (size_t)(t0 + t) * p.n + j;
-        const float a = j < p.n ? low_rank_finish(p, acc[t][0], j) : 0.0f, b = j + 1 < p.n ? low_rank_finish(p, acc[t][1], j + 1) : 0.0f;
-        if (j + 1 < p.n && !(p.n & 1)) *reinterpret_cast<float2*>(o) = make_float2(a, b);
-        else {
-            if (j < p.n) o[0] = a;
-            if (j + 1 < p.n) o[1] = b;
-        }
+        for (int g = 0; g < LRF_WARPS; ++g) z += sums[g][t][c];
+        p.out[(size_t)(t0 + t) * p.n + j0 + c] = low_rank_finish(p, z, j0 + c);
     }
 }
 
-constexpr int LR_FEW_TOKENS = 256;      // up to here the rank is shared among thread groups
+// Prompts: the products themselves are matrix products like any other (the caller's); here are their inputs, columns of a
+// projection's partial sums in the activation dtype, and what is made of their results, in place.
+template <typename TAct>
+__global__ void low_rank_inputs_kernel(const float* __restrict__ proj, int splits, size_t split_stride, int cols, int col0, int width0,
+                                       TAct* __restrict__ out0, int col1, int width1, TAct* __restrict__ out1) {
+    tt_pdl_launch_dependents();
+    tt_pdl_wait();
+    const float* row = proj + (size_t)blockIdx.x * cols;
+    for (int r = threadIdx.x; r < width0 + width1; r += blockDim.x) {
+        const bool second = r >= width0;
+        const float x = rec_sum_slices(row + (second ? col1 + r - width0 : col0 + r), splits, split_stride);
+        if (second) out1[(size_t)blockIdx.x * width1 + r - width0] = tt_from_float<TAct>(x);
+        else out0[(size_t)blockIdx.x * width0 + r] = tt_from_float<TAct>(x);
+    }
+}
+
+extern "C" int tt_low_rank_inputs(const float* proj, int splits, long long split_stride, int cols, int col0, int width0, void* out0, int col1,
+                                  int width1, void* out1, int out_dtype, int n_tokens, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (width0 < 1 || width1 < 0 || col0 < 0 || col0 + width0 > cols || (width1 && (!out1 || col1 < 0 || col1 + width1 > cols))) return (int)cudaErrorInvalidValue;
+    const int threads = width0 + width1 <= 64 ? 64 : (width0 + width1 <= 128 ? 128 : 256);
+    if (out_dtype == TT_F32) tt_launch_pdl(low_rank_inputs_kernel<float>, dim3(n_tokens), dim3(threads), 0, stream, proj, splits, (size_t)split_stride, cols, col0, width0, (float*)out0, col1, width1, (float*)out1);
+    else tt_launch_pdl(low_rank_inputs_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(threads), 0, stream, proj, splits, (size_t)split_stride, cols, col0, width0, (__nv_bfloat16*)out0, col1, width1, (__nv_bfloat16*)out1);
+    TT_LAUNCH_CHECK();
+}
+
+// out = finish(sum of z's slices), z float32 [splits][tokens][n]; out may be z's first slice
+__global__ void low_rank_finish_kernel(const float* z, int splits, size_t split_stride, const LowRankPart p) {
+    tt_pdl_launch_dependents();
+    const int j = blockIdx.y * blockDim.x + threadIdx.x;
+    if (j >= p.n) return;
+    const float bias = __ldg(p.bias + j), rate = p.kind == 1 ? -expf(__ldg(p.a_log + j / p.per_head)) : 0.0f;
+    tt_pdl_wait();
+    const size_t at = (size_t)blockIdx.x * p.n + j;
+    float x = bias;
+    for (int s = 0; s < splits; ++s) x += z[(size_t)s * split_stride + at];
+    p.out[at] = p.kind == 1 ? expf(rate * rec_softplus(x)) : expf(-rec_softplus(-x) * p.inv_tau);
+}
+
+extern "C" int tt_low_rank_finish(const float* z, int splits, long long split_stride, int n, int kind, int per_head, const float* bias,
+                                  const float* a_log, float inv_tau, float* out, int n_tokens, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (n < 1 || (kind != 1 && kind != 2) || !bias || (kind == 1 && (!a_log || per_head < 1))) return (int)cudaErrorInvalidValue;
+    const LowRankPart p{0, 0, n, kind, per_head, nullptr, bias, a_log, inv_tau, out};
+    const int threads = 256;
+    const unsigned blocks = (unsigned)((n + threads - 1) / threads);
+    if (blocks > 65535) return (int)cudaErrorInvalidValue;
+    tt_launch_pdl(low_rank_finish_kernel, dim3(n_tokens, blocks), dim3(threads), 0, stream, z, splits, (size_t)split_stride, p);
+    TT_LAUNCH_CHECK();
+}
 
 extern "C" int tt_low_rank(const float* proj, int splits, long long split_stride, int cols, int n_parts, int w_dtype,
                            int x_col0, int rank0, int n0, int kind0, int per_head0, const void* w0, const float* bias0, const float* a_log0, float inv_tau0, float* out0,
@@ -1174,16 +1213,13 @@ extern "C" int tt_low_rank(const float* proj, int splits, long long split_stride
     for (int i = 0; i < n_parts; ++i) {
         const LowRankPart& p = parts.part[i];
         if (p.rank < 1 || p.n < 1 || p.x_col < 0 || p.x_col + p.rank > cols || p.kind < 0 || p.kind > 2) return (int)cudaErrorInvalidValue;
-        if ((p.kind && !p.bias) || (p.kind == 1 && (!p.a_log || p.per_head < 1)) || ((uintptr_t)p.out & 7) || ((uintptr_t)p.w & 7)) return (int)cudaErrorInvalidValue;
+        if ((p.kind && !p.bias) || (p.kind == 1 && (!p.a_log || p.per_head < 1))) return (int)cudaErrorInvalidValue;
         widest = p.n > widest ? p.n : widest;
     }
-    const bool few = n_tokens <= LR_FEW_TOKENS;
-    const int tile = few ? 8 : 32, columns = 2 * LR_THREADS / (few ? 8 : 1);
-    const dim3 grid((n_tokens + tile - 1) / tile, (widest + columns - 1) / columns, n_parts);
+    const dim3 grid((n_tokens + LRF_TOKENS - 1) / LRF_TOKENS, (widest + LRF_COLS - 1) / LRF_COLS, n_parts);
     if (grid.y > 65535) return (int)cudaErrorInvalidValue;
-#define TT_LOW_RANK(T, TT, RG) tt_launch_pdl(low_rank_kernel<T, TT, RG>, grid, dim3(LR_THREADS), 0, stream, proj, splits, (size_t)split_stride, cols, parts, n_tokens)
-    if (w_dtype == TT_F32) { if (few) TT_LOW_RANK(float, 8, 8); else TT_LOW_RANK(float, 32, 1); }
-    else { if (few) TT_LOW_RANK(__nv_bfloat16, 8, 8); else TT_LOW_RANK(__nv_bfloat16, 32, 1); }
+#define TT_LOW_RANK(T) tt_launch_pdl(low_rank_few_kernel<T>, grid, dim3(32 * LRF_WARPS), 0, stream, proj, splits, (size_t)split_stride, cols, parts, n_tokens)
+    if (w_dtype == TT_F32) TT_LOW_RANK(float); else TT_LOW_RANK(__nv_bfloat16);
 #undef TT_LOW_RANK
     TT_LAUNCH_CHECK();
 }

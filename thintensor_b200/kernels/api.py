@@ -969,7 +969,8 @@ LOW_RANK_KINDS = {"plain": 0, "delta_decay": 1, "sigmoid_root": 2}
 
 
 def low_rank(proj: torch.Tensor, products: list[LowRank]) -> None:
-    """One or two products of low rank on columns of the same projection (float32 partial sums), in float32."""
+    """One or two products of low rank on columns of the same projection (float32 partial sums), in float32, with what is made
+    of them, in one launch: the form for few tokens.  For many, :func:`low_rank_inputs`, matrix products, :func:`low_rank_finish`."""
     if not 1 <= len(products) <= 2 or len({p.weight.dtype for p in products}) != 1:
         raise KernelError("low_rank takes one or two products with weights of one dtype")
     ptr, splits, stride, cols = _projection(proj)
@@ -990,6 +991,39 @@ def low_rank(proj: torch.Tensor, products: list[LowRank]) -> None:
         args += [0, 0, 0, 0, 1, c_void_p(0), c_void_p(0), c_void_p(0), 0.0, c_void_p(0)]
     fn = _fn("recurrent", "tt_low_rank", [c_void_p, c_int, c_longlong, c_int, c_int, c_int, *types, *types, c_int, c_void_p])
     _check(fn(ptr, splits, stride, cols, len(products), dtype_code(products[0].weight.dtype), *args, tokens, _stream()), "low_rank")
+
+
+def low_rank_inputs(proj: torch.Tensor, columns: list[tuple[int, torch.Tensor]]) -> None:
+    """One or two ranges of a projection's columns (float32 partial sums, summed) as matrices of their own: ``columns`` lists
+    (first column, out ``[tokens, width]``)."""
+    ptr, splits, stride, cols = _projection(proj)
+    if not 1 <= len(columns) <= 2 or len({out.dtype for _, out in columns}) != 1:
+        raise KernelError("low_rank_inputs takes one or two ranges into one dtype")
+    args = []
+    for col, out in columns:
+        if out.dim() != 2 or out.shape[0] != proj.shape[1] or not out.is_contiguous() or col < 0 or col + out.shape[1] > cols:
+            raise KernelError("low_rank_inputs: shapes do not fit")
+        args += [col, out.shape[1], _ptr(out)]
+    if len(columns) == 1:
+        args += [0, 0, c_void_p(0)]
+    fn = _fn("recurrent", "tt_low_rank_inputs", [c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_int,
+                                                 c_void_p])
+    _check(fn(ptr, splits, stride, cols, *args, dtype_code(columns[0][1].dtype), proj.shape[1], _stream()), "low_rank_inputs")
+
+
+def low_rank_finish(z: torch.Tensor, kind: str, bias: torch.Tensor, out: torch.Tensor, a_log: torch.Tensor | None = None, per_head: int = 1,
+                    tau: float = 1.0) -> None:
+    """What :class:`LowRank` makes of its product (``delta_decay`` or ``sigmoid_root``), from the product's partial sums; ``out``
+    (float32 ``[tokens, n]``) may be the first slice of ``z``."""
+    ptr, splits, stride, n = _projection(z)
+    for t, name in ((bias, "bias"), (a_log, "A_log"), (out, "decays")):
+        if t is not None:
+            _need(t, torch.float32, name)
+    if kind == "plain" or bias.numel() != n or tuple(out.shape) != (z.shape[1], n) or (a_log is not None and a_log.numel() != -(-n // per_head)):
+        raise KernelError("low_rank_finish: shapes do not fit")
+    fn = _fn("recurrent", "tt_low_rank_finish", [c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p, c_int, c_void_p])
+    _check(fn(ptr, splits, stride, n, LOW_RANK_KINDS[kind], per_head, _ptr(bias), _ptr(a_log), 1.0 / tau, _ptr(out), z.shape[1], _stream()),
+           "low_rank_finish")
 
 
 def weighted_pair(a: torch.Tensor, wa: float, b: torch.Tensor, wb: float, out: torch.Tensor) -> None:

@@ -60,11 +60,46 @@ def _low_rank_decls(down: str, up: str, inputs: int, rank: int, outputs: int) ->
     return {down: WeightDecl((rank, inputs), free=(0,)), up: WeightDecl((outputs, rank), free=(1,))}
 
 
-def _low_rank_up(tensors, down: str, up: str) -> torch.Tensor:
-    """The second matrix as the kernel reads it, ``[rank, outputs]``."""
-    if tensors[down].shape[0] != tensors[up].shape[1]:
-        raise ValueError(f"{down!r} makes {tensors[down].shape[0]} numbers, {up!r} takes {tensors[up].shape[1]}")
-    return tensors[up].t().contiguous()
+class LowRankProduct:
+    """The second half of a product of low rank, ``W_up`` on columns ``col ..`` of an input product (which ends with the ``W_down``
+    rows), and what is made of it: nothing (``plain``), a ``delta_decay`` or a ``sigmoid_root`` (see :class:`api.LowRank`).  Few
+    tokens run one kernel that does all of it in float32 for up to two such products of one layer; for many the columns become
+    a matrix of the activation dtype and the product one like any other."""
+
+    FEW_TOKENS = 128
+
+    def __init__(self, tensors, down: str, up: str, col: int, name: str, kind: str = "plain", bias: torch.Tensor | None = None,
+                 a_log: torch.Tensor | None = None, per_head: int = 1, tau: float = 1.0):
+        if tensors[down].shape[0] != tensors[up].shape[1]:
+            raise ValueError(f"{down!r} makes {tensors[down].shape[0]} numbers, {up!r} takes {tensors[up].shape[1]}")
+        self.up = Linear(tensors[up])
+        self.transposed = tensors[up].t().contiguous()          # as the kernel for few tokens reads it
+        self.col, self.rank, self.cols = int(col), tensors[up].shape[1], tensors[up].shape[0]
+        self.name, self.kind, self.bias, self.a_log, self.per_head, self.tau = name, kind, bias, a_log, int(per_head), float(tau)
+
+    @staticmethod
+    def run(ctx, proj: torch.Tensor, products: "list[LowRankProduct]") -> list[torch.Tensor]:
+        """One float32 tensor of partial sums ``[slices, tokens, cols]`` for each product (one slice where something is made of it)."""
+        tokens = proj.shape[1]
+        if tokens <= LowRankProduct.FEW_TOKENS:
+            out = [ctx.scratch(p.name, (1, tokens, p.cols), torch.float32) for p in products]
+            jobs = [api.LowRank(p.col, p.transposed, o[0], p.kind, p.bias, p.a_log, p.per_head, p.tau) for p, o in zip(products, out)]
+            if len({p.transposed.dtype for p in products}) == 1:
+                api.low_rank(proj, jobs)
+            else:
+                for job in jobs:
+                    api.low_rank(proj, [job])
+            return out
+        inputs = [ctx.scratch(p.name + ".in", (tokens, p.rank)) for p in products]
+        api.low_rank_inputs(proj, [(p.col, x) for p, x in zip(products, inputs)])
+        out = []
+        for p, x in zip(products, inputs):
+            z = p.up(ctx, x, p.name)
+            if p.kind != "plain":
+                api.low_rank_finish(z, p.kind, p.bias, z[0], p.a_log, p.per_head, p.tau)
+                z = z[:1]
+            out.append(z)
+        return out
 
 
 def _in_blocks(ctx) -> bool:
@@ -167,8 +202,7 @@ class GatedDelta(Mixer):
         if gate not in api.NORM_GATES:
             raise ValueError(f"the gate is one of {sorted(api.NORM_GATES)}, not {gate!r}")
         self.gate = gate
-        self.decay_up: torch.Tensor | None = None
-        self.gate_up: torch.Tensor | None = None
+        self.low_rank: list[LowRankProduct] = []       # the decay's, then the gate's
         self.names = {**self.NAMES, **(names or {})}
         self.proj: Linear | None = None
         self.out: Linear | None = None
@@ -206,18 +240,20 @@ class GatedDelta(Mixer):
         self.out = Linear(tensors[n["out"]])
         self.b_col = self.channels + tensors[n[gate]].shape[0]
         self.a_col = self.b_col + self.heads
-        self.decay_up = _low_rank_up(tensors, n["a1"], n["a2"]) if self.channel_decay else None
-        self.gate_up = _low_rank_up(tensors, n["g1"], n["g2"]) if self.low_rank_gate else None
-        if self.decay_up is not None and self.gate_up is not None and self.decay_up.dtype != self.gate_up.dtype:
-            self.decay_up, self.gate_up = _f32(self.decay_up), _f32(self.gate_up)       # one launch for both
         self.conv_weight = torch.cat([_f32(tensors[n[key]]) for key in ("q_conv", "k_conv", "v_conv")], dim=0).contiguous()
         self.dt_bias, self.a_log, self.norm = _f32(tensors[n["dt_bias"]]), _f32(tensors[n["A_log"]]), _f32(tensors[n["norm"]])
+        self.low_rank = []
+        if self.channel_decay:
+            self.low_rank.append(LowRankProduct(tensors, n["a1"], n["a2"], self.a_col, "delta.decay", "delta_decay", self.dt_bias, self.a_log,
+                                                self.key_dim))
+        if self.low_rank_gate:
+            self.low_rank.append(LowRankProduct(tensors, n["g1"], n["g2"], self.channels, "delta.gates"))
 
     def projections(self) -> list:
-        return [self.proj, self.out]
+        return [self.proj, self.out] + [p.up for p in self.low_rank]
 
     def vectors(self) -> list[torch.Tensor]:
-        return [self.conv_weight, self.dt_bias, self.a_log, self.norm] + [t for t in (self.decay_up, self.gate_up) if t is not None]
+        return [self.conv_weight, self.dt_bias, self.a_log, self.norm]
 
     def device_driven(self) -> bool:
         return True
@@ -227,16 +263,12 @@ class GatedDelta(Mixer):
         tokens = ctx.n_tokens
         proj = self.proj(ctx, x, "delta.in")
         decay, gate_source, gate_col = None, proj, self.channels
-        products = []
-        if self.decay_up is not None:
-            decay = ctx.scratch("delta.decay", (tokens, self.heads * self.key_dim), torch.float32)
-            products.append(api.LowRank(self.a_col, self.decay_up, decay, "delta_decay", self.dt_bias, self.a_log, self.key_dim))
-        if self.gate_up is not None:
-            gates = ctx.scratch("delta.gates", (1, tokens, self.v), torch.float32)
-            products.append(api.LowRank(self.channels, self.gate_up, gates[0]))
-            gate_source, gate_col = gates, 0
-        if products:
-            api.low_rank(proj, products)
+        if self.low_rank:
+            made = LowRankProduct.run(ctx, proj, self.low_rank)
+            if self.channel_decay:
+                decay = made[0][0]
+            if self.low_rank_gate:
+                gate_source, gate_col = made[-1], 0
         qkv = ctx.scratch("delta.qkv", (tokens, self.channels), torch.float32)
         api.causal_conv(proj, 0, self.channels, self.conv_weight, None, True, tail, qkv, ctx.cu, ctx.slots, ctx.sequences, tokens, ctx.decode)
         read = ctx.scratch("delta.read", (tokens, self.v), torch.float32)
@@ -270,8 +302,7 @@ class DecayLinearAttention(Mixer):
         self.rank = None if channel_decay is None else int(channel_decay["rank"])
         self.tau = None if channel_decay is None else float(channel_decay["tau"])
         self.query_scale = float(query_scale)
-        self.decay_up: torch.Tensor | None = None
-        self.decay_bias: torch.Tensor | None = None
+        self.low_rank: LowRankProduct | None = None
         if activation not in (None, "silu"):
             raise ValueError(f"q, k and v pass silu or nothing, not {activation!r}")
         if norm not in ("head", "all"):
@@ -325,17 +356,18 @@ class DecayLinearAttention(Mixer):
         self.out = Linear(tensors[n["out"]])
         self.decays = None
         if self.rank is not None:
-            self.decay_up, self.decay_bias = _low_rank_up(tensors, n["a1"], n["a2"]), _f32(tensors[n["a_bias"]])
+            self.low_rank = LowRankProduct(tensors, n["a1"], n["a2"], 2 * self.qk + 2 * self.v, "linear_attention.decay", "sigmoid_root",
+                                           _f32(tensors[n["a_bias"]]), tau=self.tau)
         else:
             self.decays = torch.tensor(self.decay, dtype=torch.float32, device=device)
         count = self.v if self.norm == "all" else self.value_dim
         self.norm_w = _f32(tensors[n["norm"]]) if self.norm_weight else torch.ones(count, dtype=torch.float32, device=device)
 
     def projections(self) -> list:
-        return [self.proj, self.out]
+        return [self.proj, self.out] + ([self.low_rank.up] if self.low_rank is not None else [])
 
     def vectors(self) -> list[torch.Tensor]:
-        return ([self.norm_w] if self.norm_weight else []) + [t for t in (self.decay_up, self.decay_bias) if t is not None]
+        return ([self.norm_w] if self.norm_weight else []) + ([self.low_rank.bias] if self.low_rank is not None else [])
 
     def device_driven(self) -> bool:
         return True
@@ -347,9 +379,8 @@ class DecayLinearAttention(Mixer):
         rotary_dim = self.rot.rotary_dim if self.rot is not None else 0
         read = ctx.scratch("linear_attention.read", (tokens, self.v), torch.float32)
         decay = None
-        if self.decay_up is not None:
-            decay = ctx.scratch("linear_attention.decay", (tokens, self.qk), torch.float32)
-            api.low_rank(proj, [api.LowRank(2 * self.qk + 2 * self.v, self.decay_up, decay, "sigmoid_root", self.decay_bias, tau=self.tau)])
+        if self.low_rank is not None:
+            decay = LowRankProduct.run(ctx, proj, [self.low_rank])[0][0]
         blocks = decay is not None and _in_blocks(ctx)
         if blocks and proj.shape[0] == 1 and not rotary_dim and self.activation is None and self.key_scale == 1.0:
             q, k, v = proj[0].split((self.qk, self.qk, self.v, proj.shape[2] - 2 * self.qk - self.v), dim=1)[:3]     # the product as it is
