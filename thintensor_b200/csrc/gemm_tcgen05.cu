@@ -103,9 +103,10 @@ struct Args {
 };
 
 // the gate's activation of the gated forms: act(gate) * up is what they store
+// (the tanh form of gelu is g times the logistic function of twice tanh's argument: (1 + tanh(z)) / 2 = 1 / (1 + exp(-2 z)))
 __device__ __forceinline__ float gate_activation(float g, int activation) {
     if (activation == 1) return fmaxf(g, 0.0f);
-    if (activation == 2) return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
+    if (activation == 2) return __fdividef(g, 1.0f + __expf(-1.5957691216057308f * fmaf(0.044715f * g * g, g, g)));
     return __fdividef(g, 1.0f + __expf(-g));
 }
 
@@ -117,6 +118,24 @@ __device__ __forceinline__ float gated_unit(float g, float u, int feature, const
         return __fdividef(g, 1.0f + __expf(-args.clamp_alpha * g)) * (u + 1.0f);
     }
     return gate_activation(g, args.activation) * u;
+}
+
+// Eight neighbouring features at a time, with the choice of the unit outside the loop over them: chosen feature by feature it
+// cost the prompt kernels' epilogues more than their tiles' products (2,048 x 8,192 x 2,048: 200 us against 95).
+__device__ __forceinline__ void gated_units(const float (&g)[8], const float (&u)[8], float (&y)[8], int feature, const Args& args) {
+    if (args.activation == 0) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) y[e] = gate_activation(g[e], 0) * u[e];
+    } else if (args.activation == 1) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) y[e] = gate_activation(g[e], 1) * u[e];
+    } else if (args.activation == 2) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) y[e] = gate_activation(g[e], 2) * u[e];
+    } else {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) y[e] = gated_unit(g[e], u[e], feature + e, args);
+    }
 }
 
 // GROUP: k-blocks that share one round of the full / empty barriers (STAGES is a multiple of it).  With few tokens
@@ -386,12 +405,10 @@ __device__ __forceinline__ void store_accumulator(uint32_t lane_addr, int token,
 #pragma unroll
                 for (int e0 = 0; e0 < 32; e0 += 8) {
                     const int f = f_base + c + e0;
-                    float y[8];
+                    float y[8], g[8], u[8];
 #pragma unroll
-                    for (int e = 0; e < 8; ++e) {
-                        const float g = tmem_loaded(gate[cur][e0 + e]), u = tmem_loaded(up[cur][e0 + e]);
-                        y[e] = gated_unit(g, u, f + e, args);
-                    }
+                    for (int e = 0; e < 8; ++e) { g[e] = tmem_loaded(gate[cur][e0 + e]); u[e] = tmem_loaded(up[cur][e0 + e]); }
+                    gated_units(g, u, y, f, args);
                     if (vec && f + 8 <= args.features) {
                         const __nv_bfloat162 p0 = __floats2bfloat162_rn(y[0], y[1]), p1 = __floats2bfloat162_rn(y[2], y[3]);
                         const __nv_bfloat162 p2 = __floats2bfloat162_rn(y[4], y[5]), p3 = __floats2bfloat162_rn(y[6], y[7]);
@@ -523,12 +540,10 @@ __device__ __forceinline__ void store_swiglu_bulk(uint32_t lane_addr, int first_
         }
 #pragma unroll
         for (int e0 = 0; e0 < 32; e0 += 8) {
-            float y[8];
+            float y[8], g[8], u[8];
 #pragma unroll
-            for (int e = 0; e < 8; ++e) {
-                const float g = tmem_loaded(gate[cur][e0 + e]), u = tmem_loaded(up[cur][e0 + e]);
-                y[e] = gated_unit(g, u, f_base + 32 * ci + e0 + e, args);
-            }
+            for (int e = 0; e < 8; ++e) { g[e] = tmem_loaded(gate[cur][e0 + e]); u[e] = tmem_loaded(up[cur][e0 + e]); }
+            gated_units(g, u, y, f_base + 32 * ci + e0, args);
             const __nv_bfloat162 p0 = __floats2bfloat162_rn(y[0], y[1]), p1 = __floats2bfloat162_rn(y[2], y[3]);
             const __nv_bfloat162 p2 = __floats2bfloat162_rn(y[4], y[5]), p3 = __floats2bfloat162_rn(y[6], y[7]);
             const int piece = (ci & 1) * 4 + (e0 >> 3);
