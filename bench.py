@@ -137,7 +137,8 @@ def zuvepel_pair(size: str) -> tuple[dict, dict]:
     """(Zuvepel config.json, Famalorn config.json) of one size from the table of named shapes: the same width, feed-forward
     width, vocabulary and number of layers (six, each run once).  Famalorn is the closest model: its delta layers have the same
     heads (a decay per head where Zuvepel's have one per key channel), its Mamba-2 scan is the like of the gla layers' scan (16 or
-    24 heads of 64 x 128), its attention branch has the same heads and a sink (Zuvepel's: chunks of 1,024)."""
+    24 heads of 64 x 128), its attention branch has the same heads and a sink (Zuvepel's: chunks of 8,192, so all keys
+    of the workload, at width 2,048 and of 1,536 at width 3,072)."""
     return json.loads(json.dumps(SHAPES[ZUVEPEL_SHAPES[size]])), json.loads(json.dumps(SHAPES[FAMALORN_SHAPES[size]]))
 
 

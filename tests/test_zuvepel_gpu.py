@@ -285,12 +285,12 @@ def test_what_the_cache_holds(folders):
     assert runtime.model.device_driven
     engine = runtime.new_engine(max_tokens=128, max_sequences=2)
     needs = [(g.need.kv_heads, g.need.head_dim, g.need.v_dim, g.need.window, len(g.runs)) for g in engine.cache.kv_groups]
-    assert needs == [(2, 16, 24, 21, 3)]
+    assert needs == [(2, 16, 24, 21, 2)]
     shapes = sorted((tuple(g.need.shape), len(g.runs)) for g in engine.cache.state_groups)
-    assert shapes == sorted([((4, 40, 24), 3), ((2, 2 * 48 + 160), 3), ((3, 12, 20), 1)])
+    assert shapes == sorted([((4, 40, 24), 2), ((2, 2 * 48 + 160), 2), ((3, 12, 20), 1)])
     engine = load(folders("c", "float32"), "float32").new_engine(max_tokens=128, max_sequences=2)
     needs = sorted((g.need.kv_heads, g.need.head_dim, len(g.runs)) for g in engine.cache.kv_groups)
-    assert needs == [(1, 128, 1), (2, 64, 2)]
+    assert needs == [(1, 128, 1), (2, 64, 3)]
 
 
 @pytest.mark.parametrize("name,dtype", [("a", "float32"), ("c", "bfloat16"), ("b", "bfloat16")])

@@ -19,10 +19,10 @@ def _dense(ff):
 
 
 CONFIGS = {
-    # a chunk inside the first block; three passes over the first two layers
+    # a chunk inside the first block; two passes over the first two layers
     "a": {
         "architecture": "Zuvepel", "vocab": 211, "width": 96, "norm": {"eps": 1e-5}, "residual_mult": 0.7, "embedding": {"scale": 1.5},
-        "loop": {"start": 0, "stop": 2, "times": 3},
+        "loop": {"start": 0, "stop": 2, "times": 2},
         "layers": [
             {"type": "attention", "mlp": _dense(136), "mixer": {
                 "heads": 6, "kv_heads": 2, "dim": 16, "vdim": 24, "mask": {"size": 21}, "rot": {"dims": 8, "base": 500.0}, "scale": 0.3}},
@@ -40,10 +40,10 @@ CONFIGS = {
             {"type": "channel_delta", "mlp": _dense(64), "mixer": {"heads": 3, "kv_heads": 1, "dim": 136, "vdim": 8, "conv": 1}},
         ],
     },
-    # attention heads of tensor-core sizes, one layer without chunks; the loop in the middle; the factor 1
+    # attention heads of tensor-core sizes, one layer without chunks; three passes over the layers in the middle; the factor 1
     "c": {
         "architecture": "Zuvepel", "vocab": 160, "width": 128, "norm": {"eps": 1e-6}, "residual_mult": 1.0, "embedding": {"scale": 2.0},
-        "loop": {"start": 1, "stop": 3, "times": 2},
+        "loop": {"start": 1, "stop": 3, "times": 3},
         "layers": [
             {"type": "channel_delta", "mlp": _dense(160), "mixer": {"heads": 2, "kv_heads": 2, "dim": 64, "vdim": 48, "conv": 5}},
             {"type": "attention", "mlp": _dense(192), "mixer": {
@@ -58,9 +58,11 @@ SEEDS = {"a": 3, "b": 4, "c": 6}
 
 
 def _rank(name: str, drawn: int) -> int:
-    """A rank for the products of low rank of layer ``l<i>.``, which is the tensors' alone: odd, and another one in every layer
-    and for the gate than for the decay."""
+    """A rank for the products of low rank of layer ``l<i>.``, which is the tensors' alone: another one in every layer and for the
+    gate than for the decay; multiples of eight (tensor-core products in bfloat16) in the first layer, odd in the others."""
     layer = int(name[1:name.index(".")])
+    if layer == 0:
+        return 8 if name[-2] == "a" else 32
     return 5 + 2 * layer if name[-2] == "a" else 9 + 2 * layer
 
 
