@@ -115,7 +115,7 @@ def attention_reference(q, keys, values, new_lens, heads, kv_heads, scale, windo
         total = k.shape[0]
         for i in range(new):
             pos = total - new + i
-            first = max(0, pos - window + 1) if window else 0
+            first = pos - pos % -window if window < 0 else max(0, pos - window + 1) if window else 0        # below zero: chunks
             for h in range(heads):
                 kh = h // group
                 s = (k[first: pos + 1, kh] @ q[t, h].double()) * scale
@@ -362,7 +362,7 @@ def test_attention_mma_decode_in_several_rounds(sequences, heads, kv_heads, head
 
 @pytest.mark.parametrize("write_cache", [True, False])
 @pytest.mark.parametrize("splits", [1, 3, 16])
-@pytest.mark.parametrize("window", [0, 100])
+@pytest.mark.parametrize("window", [0, 100, -90])
 @pytest.mark.parametrize("heads,kv_heads,head_dim", [(8, 2, 64), (3, 1, 64), (32, 8, 64), (10, 5, 64), (16, 1, 64)])
 def test_attention_decode_with_rotation_and_cache_write(splits, window, heads, kv_heads, head_dim, write_cache):
     """Decoding straight from the slices of the qkv product: the kernel rotates q and k, writes
