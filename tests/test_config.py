@@ -73,10 +73,11 @@ def test_config_errors(change, needle):
 
 
 def test_registry():
-    assert supported_architectures() == ["Famalorn", "Kerepel", "LlamaForCausalLM", "Neruzen", "Sogidra", "Zuvepel"]
+    assert supported_architectures() == ["Famalorn", "Kerepel", "LlamaForCausalLM", "Neruzen", "Sogidra", "Zezilix", "Zuvepel"]
     assert resolve_architecture({"architecture": "Sogidra"}).name == "Sogidra"
     assert resolve_architecture({"architecture": "Kerepel"}).name == "Kerepel"
     assert resolve_architecture({"architecture": "Zuvepel"}).name == "Zuvepel"
+    assert resolve_architecture({"architecture": "Zezilix"}).name == "Zezilix"
     assert resolve_architecture({"architecture": "Famalorn"}).name == "Famalorn"
     assert resolve_architecture({"architecture": "Neruzen"}).name == "Neruzen"
     assert resolve_architecture({"architectures": ["LlamaForCausalLM"]}).name == "LlamaForCausalLM"

@@ -447,7 +447,7 @@ def test_latent_attention_with_direct_queries(dtype, heads, dim, rot, vdim, rank
             part_ml = torch.zeros(tokens * heads * splits * 2, dtype=torch.float32, device=DEV)
             api.latent_attention(wide[:, :, front:front + q_cols], w_key.to(DEV), w_value.to(DEV), pool, step_table, i32(cu), i32([at[b] for b in live]),
                                  len(live), tokens, heads, dim, rot, vdim, rank, inv_freq, rot, scale, 0, splits, out, absorbed, part_acc, part_ml, word,
-                                 interleaved=True, rot_scale=factor, head_gate=wide[:, :, front + q_cols:] if gated else None)
+                                 interleaved=True, rot_scale=factor, gate=wide[:, :, front + q_cols:] if gated else None)
             assert int(word.item()) == 0
             for i, (b, n) in enumerate(zip(live, counts)):
                 expect = torch.stack(want[b][at[b]: at[b] + n])

@@ -108,7 +108,7 @@ def test_low_rank_products(tokens, weights, splits, rank_a, heads, dim, rank_b, 
     # the pieces of the form for many tokens
     for dtype in (torch.float32, torch.bfloat16):
         in_a, in_b = (torch.empty(tokens, n, dtype=dtype, device=DEV) for n in (rank_a, rank_b))
-        api.low_rank_inputs(proj, [(off, in_a), (off + rank_a + 2, in_b)])
+        api.low_rank_inputs(proj, [(off, in_a, False), (off + rank_a + 2, in_b, False)])
         for got, lo in ((in_a, off), (in_b, off + rank_a + 2)):
             want = x[:, lo: lo + got.shape[1]]
             assert float((got.double().cpu() - want).abs().max()) <= (1e-5 if dtype == torch.float32 else 5e-3) * float(want.abs().max())

@@ -1,7 +1,7 @@
-// Memory-bound kernels between the matrix products: embedding gather (also with a hashed
+// Memory-bound kernels between the matrix products: embedding gather (also with an RMS norm of the row, and with a hashed
 // row for the pair of the previous token and this one), residual add fused with RMSNorm (also with two scaled
 // branches added and two norms taken of the sum),
-// the token shift of a mixer's input, rotary encoding fused with the cache append, SwiGLU,
+// the token shift of a mixer's input (one blend, or several of the same rows), rotary encoding fused with the cache append, SwiGLU,
 // and the length bookkeeping of a step.  All statistics, angles and sums are float32.
 //
 // Counterparts in random-unknown-username/Thintensor (Triton, one token per launch):
@@ -59,6 +59,45 @@ extern "C" int tt_embed_gather(const void* table, int table_dtype, const int* to
         tt_launch_pdl(embed_gather_kernel<float>, dim3(n_tokens), dim3(threads), 0, stream, (const float*)table, tokens, residual, hidden, vocab, scale, status);
     else
         tt_launch_pdl(embed_gather_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(threads), 0, stream, (const __nv_bfloat16*)table, tokens, residual, hidden, vocab, scale, status);
+    TT_LAUNCH_CHECK();
+}
+
+// ------------------------------------------------------------------------------------
+// embedding gather with a norm: with e = table[token[t], :] * scale, residual[t, :] = e * rsqrt(mean(e^2) + eps) * weight.
+// The block reads its row twice, the second time from the L1.
+// ------------------------------------------------------------------------------------
+template <typename TW>
+__global__ void embed_norm_gather_kernel(const TW* __restrict__ table, const int* __restrict__ tokens, const float* __restrict__ weight,
+                                         float eps, float* __restrict__ residual, int hidden, int vocab, float scale, unsigned* status) {
+    tt_pdl_wait();                      // the first kernel of a step: see embed_gather_kernel
+    tt_pdl_launch_dependents();
+    __shared__ float reduce[32];
+    const int t = blockIdx.x;
+    const int id = tokens[t];
+    float* out = residual + (size_t)t * hidden;
+    if (id < 0 || id >= vocab) {
+        if (threadIdx.x == 0) atomicOr(status, TT_STATUS_BAD_TOKEN);
+        for (int j = threadIdx.x; j < hidden; j += blockDim.x) out[j] = 0.0f;
+        return;
+    }
+    const TW* row = table + (size_t)id * hidden;
+    float sumsq = 0.0f;
+    for (int j = threadIdx.x; j < hidden; j += blockDim.x) {
+        const float x = tt_to_float(row[j]) * scale;
+        sumsq = fmaf(x, x, sumsq);
+    }
+    const float gain = rsqrtf(tt_block_sum(sumsq, reduce) / (float)hidden + eps);
+    for (int j = threadIdx.x; j < hidden; j += blockDim.x) out[j] = tt_to_float(row[j]) * scale * gain * __ldg(weight + j);
+}
+
+extern "C" int tt_embed_norm_gather(const void* table, int table_dtype, const int* tokens, const float* weight, float eps, float* residual,
+                                    int n_tokens, int hidden, int vocab, float scale, unsigned* status, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    const int threads = hidden >= 1024 ? 256 : 128;
+    if (table_dtype == TT_F32)
+        tt_launch_pdl(embed_norm_gather_kernel<float>, dim3(n_tokens), dim3(threads), 0, stream, (const float*)table, tokens, weight, eps, residual, hidden, vocab, scale, status);
+    else
+        tt_launch_pdl(embed_norm_gather_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(threads), 0, stream, (const __nv_bfloat16*)table, tokens, weight, eps, residual, hidden, vocab, scale, status);
     TT_LAUNCH_CHECK();
 }
 
@@ -1025,6 +1064,80 @@ extern "C" int tt_token_shift(const void* x, int dtype, const float* mix, float*
 }
 
 // ------------------------------------------------------------------------------------
+// Several blends of the same rows at once: out[m][t] = x[t] + (x[t - 1] - x[t]) * mix[m], m < blends, with one state row per
+// sequence (its last x).  A thread takes VEC neighbouring channels through `tile` packed tokens with the row before in
+// registers; where the tile holds a sequence's first token of the step it reads that row from the sequence's state and moves
+// the state on to the step's last row, its own channels only.
+// ------------------------------------------------------------------------------------
+constexpr int SHIFT_BLENDS = 8;
+
+template <typename T, int VEC> struct alignas(VEC * sizeof(T)) ShiftPack { T v[VEC]; };
+
+template <typename T, int VEC>
+__global__ void token_shifts_kernel(const T* __restrict__ x, const float* __restrict__ mix, int blends, float* __restrict__ state,
+                                    T* __restrict__ out, size_t out_stride, const int* __restrict__ cu, const int* __restrict__ slots,
+                                    int sequences, int n_tokens, int hidden, int tile) {
+    tt_pdl_launch_dependents();
+    const int j = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
+    if (j >= hidden) return;
+    const int t0 = blockIdx.x * tile, t1 = min(t0 + tile, n_tokens);
+    int b = tt_find_sequence(cu, sequences, t0);
+    int first = cu[b], next = cu[b + 1];
+    float before[VEC];
+    tt_pdl_wait();
+    using Pack = ShiftPack<T, VEC>;
+    for (int t = t0; t < t1; ++t) {
+        while (t >= next) {                                     // the next sequence starts here
+            ++b;
+            first = next;
+            next = cu[b + 1];
+        }
+        if (t == first) {
+            float* st = state + (size_t)slots[b] * hidden + j;
+            const Pack tail = *reinterpret_cast<const Pack*>(x + (size_t)(next - 1) * hidden + j);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+                before[e] = st[e];
+                st[e] = tt_to_float(tail.v[e]);
+            }
+        } else if (t == t0) {
+            const Pack row = *reinterpret_cast<const Pack*>(x + (size_t)(t - 1) * hidden + j);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) before[e] = tt_to_float(row.v[e]);
+        }
+        const Pack row = *reinterpret_cast<const Pack*>(x + (size_t)t * hidden + j);
+        float now[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) now[e] = tt_to_float(row.v[e]);
+        for (int m = 0; m < blends; ++m) {
+            Pack o;
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) o.v[e] = tt_from_float<T>(fmaf(before[e] - now[e], __ldg(mix + (size_t)m * hidden + j + e), now[e]));
+            *reinterpret_cast<Pack*>(out + (size_t)m * out_stride + (size_t)t * hidden + j) = o;
+        }
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) before[e] = now[e];
+    }
+}
+
+// out: blend m starts out_stride numbers after blend m - 1
+extern "C" int tt_token_shifts(const void* x, int dtype, const float* mix, int blends, float* state, void* out, long long out_stride,
+                               const int* cu, const int* slots, int sequences, int n_tokens, int hidden, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (blends < 1 || blends > SHIFT_BLENDS || hidden <= 0) return (int)cudaErrorInvalidValue;
+    const int vec = dtype == TT_F32 ? 4 : 8, threads = 128;
+    const bool wide = hidden % vec == 0 && out_stride % vec == 0 && (((uintptr_t)x | (uintptr_t)out) & 15) == 0;
+    const int per_block = threads * (wide ? vec : 1), tile = n_tokens >= 1024 ? 8 : 1;
+    const dim3 grid((n_tokens + tile - 1) / tile, (hidden + per_block - 1) / per_block), block(threads);
+    if (grid.y > 65535) return (int)cudaErrorInvalidValue;
+#define TT_SHIFTS(T, V) tt_launch_pdl(token_shifts_kernel<T, V>, grid, block, 0, stream, (const T*)x, mix, blends, state, (T*)out, (size_t)out_stride, cu, slots, sequences, n_tokens, hidden, tile)
+    if (dtype == TT_F32) { if (wide) TT_SHIFTS(float, 4); else TT_SHIFTS(float, 1); }
+    else { if (wide) TT_SHIFTS(__nv_bfloat16, 8); else TT_SHIFTS(__nv_bfloat16, 1); }
+#undef TT_SHIFTS
+    TT_LAUNCH_CHECK();
+}
+
+// ------------------------------------------------------------------------------------
 // embedding with a learned position vector:
 //   residual[t, :] = table[token[t], :] * scale + positions[p, :],  p = len_before[b] + (t - cu[b])   (float32 out)
 // A token outside the table, or a position beyond the position table's rows, raises the bad-token bit and leaves zeros.
@@ -1066,10 +1179,11 @@ extern "C" int tt_embed_position_gather(const void* table, const void* positions
 
 // ------------------------------------------------------------------------------------
 // Ungated activation: act[t, j] = f(sum over slices of x[s][t, j]).  f by `activation`: 0 silu, 1 relu, 2 tanh-gelu (as
-// in tt_gate_activation), 4 the exact gelu 0.5 z (1 + erf(z / sqrt 2)), 3 xielu with two numbers a = softplus(p) and c = 1/2 + softplus(q) that the caller has formed:
+// in tt_gate_activation), 5 the square of relu, 4 the exact gelu 0.5 z (1 + erf(z / sqrt 2)), 3 xielu with two numbers a = softplus(p) and c = 1/2 + softplus(q) that the caller has formed:
 //   z > 0: a z^2 + z / 2;   z <= 0: c (exp(z) - 1 - z) + z / 2     (expm1f keeps small z exact)
 // ------------------------------------------------------------------------------------
 __device__ __forceinline__ float tt_unary_activation(float z, int activation, float a, float c) {
+    if (activation == 5) { const float p = fmaxf(z, 0.0f); return p * p; }
     if (activation == 4) return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f));        // the exact gelu
     if (activation == 3) return z > 0.0f ? fmaf(a * z, z, 0.5f * z) : fmaf(c, expm1f(z) - z, 0.5f * z);
     return tt_gate_activation(z, activation);
@@ -1102,7 +1216,7 @@ __global__ void activation_kernel(const float* __restrict__ x, int splits, size_
 extern "C" int tt_activation(const float* x, int splits, long long split_stride, void* act, int act_dtype, long long total,
                              int activation, float a, float c, cudaStream_t stream) {
     if (total <= 0) return 0;
-    if (activation < 0 || activation > 4) return (int)cudaErrorInvalidValue;
+    if (activation < 0 || activation > 5) return (int)cudaErrorInvalidValue;
     const int threads = 256;
     const unsigned blocks = (unsigned)(((total + 3) / 4 + threads - 1) / threads);      // a thread takes four numbers; the last one what is left
     if (act_dtype == TT_F32)

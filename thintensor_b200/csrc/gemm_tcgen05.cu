@@ -99,8 +99,16 @@ struct Args {
     // features below clamp_split use clamp_low as their limit, the others clamp_high (a limit of 0 or less: no clamp)
     float clamp_low, clamp_high, clamp_alpha;
     int clamp_split;
+    // plain forms: output features in groups of so many, each with activations of its own, the rows of which follow one another (x
+    // is [groups][tokens][k]; a tile's features lie in one group).  0: all features read the same activations
+    int group_features;
     unsigned* status;
 };
+
+// the first row of the activations that output feature `feature` reads
+__device__ __forceinline__ int group_rows(int feature, const Args& args) {
+    return args.group_features > 0 ? feature / args.group_features * args.tokens : 0;
+}
 
 // the gate's activation of the gated forms: act(gate) * up is what they store
 // (the tanh form of gelu is g times the logistic function of twice tanh's argument: (1 + tanh(z)) / 2 = 1 / (1 + exp(-2 z)))
@@ -180,12 +188,13 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
     constexpr bool paired_rows = FORM == FEATURES_ON_M_SWIGLU;     // 64 gate rows over the 64 up rows of the same features
     const int a_row = tile_m * (paired_rows ? BM / 2 : BM);       // tokens (TOKENS_ON_M*) or features (FEATURES_ON_M*)
     const int b_row = tile_n * BN;
+    const int x_row0 = group_rows(weights_are_a ? a_row : b_row, args);
     auto load_a = [&](uint8_t* stage, int kx, uint32_t bar) {
         if (paired_rows) {
             tma_load_2d(smem_u32(stage), &map_a, kx, a_row, bar);
             tma_load_2d(smem_u32(stage + S::a_bytes / 2), &map_a, kx, args.up_row_offset + a_row, bar);
         } else {
-            tma_load_2d(smem_u32(stage), &map_a, kx, a_row, bar);
+            tma_load_2d(smem_u32(stage), &map_a, kx, weights_are_a ? a_row : a_row + x_row0, bar);
         }
     };
 
@@ -205,7 +214,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                 }
             };
             auto load_activations = [&](uint8_t* stage, int kx, uint32_t bar) {
-                if (weights_are_a) tma_load_2d(smem_u32(stage + S::a_bytes), &map_b, kx, b_row, bar);
+                if (weights_are_a) tma_load_2d(smem_u32(stage + S::a_bytes), &map_b, kx, b_row + x_row0, bar);
                 else load_a(stage, kx, bar);
             };
             const int first = min(n_groups, RING);
@@ -789,7 +798,7 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const 
             bool ok = true;
             for (int j = 0; j < my_tiles && ok; ++j) {
                 const int item = (int)blockIdx.x + j * (int)gridDim.x, tile = item % tiles_total;
-                const int a_row = (tile % tiles_m) * BM, b_row = (tile / tiles_m) * TILE_N;
+                const int b_row = (tile / tiles_m) * TILE_N, a_row = (tile % tiles_m) * BM + group_rows(b_row, args);
                 int kb_begin;
                 const int n_kb = k_blocks_of(item, kb_begin);
                 for (int i = 0; i < n_kb; ++i, ++it) {
@@ -976,7 +985,7 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid
             for (int j = 0; j < my_tiles && ok; ++j) {
                 int tile, kb0, kb1;
                 item(j, tile, kb0, kb1);
-                const int a_row = (tile % tiles_m) * 2 * BM + rank * BM;
+                const int a_row = (tile % tiles_m) * 2 * BM + rank * BM + group_rows((tile / tiles_m) * TILE_N, args);
                 const int b_row = dual ? (rank == 0 ? 0 : args.up_row_offset) + (tile / tiles_m) * TILE_N
                                        : (tile / tiles_m) * TILE_N + rank * B_ROWS;
                 for (int i = kb0; i < kb1; ++i, ++it) {
@@ -1311,7 +1320,8 @@ struct GateClamp { float low, high, alpha; int split; };
 
 static int gemm_dispatch(const void* x, long long ldx, const void* w, long long ldw, const float* bias, void* out,
                          long long ld_out, long long split_stride, int tokens, int features, int k, int splits,
-                         int form, unsigned* status, cudaStream_t stream, void* shares, long long shares_bytes, const GateClamp clamp) {
+                         int form, unsigned* status, cudaStream_t stream, void* shares, long long shares_bytes, const GateClamp clamp,
+                         int group_features = 0) {
     if (tokens <= 0 || features <= 0) return 0;
     if (k <= 0 || (k % 8) || (ldx % 8) || (ldw % 8) || ((uintptr_t)x & 15) || ((uintptr_t)w & 15) || splits < 1)
         return (int)cudaErrorInvalidValue;
@@ -1331,6 +1341,9 @@ static int gemm_dispatch(const void* x, long long ldx, const void* w, long long 
     args.undelivered_bytes = undelivered_bytes_for_tests;
     args.bulk_out = 0;
     args.shares = nullptr;
+    args.group_features = group_features;
+    const long long x_rows = group_features > 0 ? (long long)tokens * ((features + group_features - 1) / group_features) : tokens;
+    if (x_rows > 2147483647LL) return (int)cudaErrorInvalidValue;
     CUtensorMap map_a, map_b;
     const int tiles_m = (tokens + BM - 1) / BM;
     if (form == 2 && !(tokens > 128 && tiles_m * ((features + 255) / 256) >= 8 && splits == 1)) return (int)cudaErrorInvalidValue;
@@ -1386,13 +1399,13 @@ static int gemm_dispatch(const void* x, long long ldx, const void* w, long long 
             int device = 0, sm_count = 0;
             if (cudaGetDevice(&device) != cudaSuccess || cudaDeviceGetAttribute(&sm_count, cudaDevAttrMultiProcessorCount, device) != cudaSuccess) return -1;
             if (form == 0 && tiles_m * ((features + 255) / 256) * 8 <= sm_count) {
-                if (!make_map(&map_a, x, tokens, k, ldx, BM) || !make_map(&map_b, w, features, k, ldw, 128)) return -1;
+                if (!make_map(&map_a, x, x_rows, k, ldx, BM) || !make_map(&map_b, w, features, k, ldw, 128)) return -1;
                 return launch_persistent<TOKENS_ON_M, 128>(map_a, map_b, map_out, args, tiles_m, tiles_m * ((features + 127) / 128), splits, stream);
             }
-            if (!make_map(&map_a, x, tokens, k, ldx, BM) || !make_map(&map_b, w, features, k, ldw, 256)) return -1;
+            if (!make_map(&map_a, x, x_rows, k, ldx, BM) || !make_map(&map_b, w, features, k, ldw, 256)) return -1;
             return launch_persistent<TOKENS_ON_M>(map_a, map_b, map_out, args, tiles_m, tiles_m * ((features + 255) / 256), splits, stream);
         }
-        if (!make_map(&map_a, x, tokens, k, ldx, BM) || !make_map(&map_b, w, features, k, ldw, 128)) return -1;
+        if (!make_map(&map_a, x, x_rows, k, ldx, BM) || !make_map(&map_b, w, features, k, ldw, 128)) return -1;
         const int pair_tiles_m = (tokens + 2 * BM - 1) / (2 * BM);
         const int pair_tiles = pair_tiles_m * ((features + 255) / 256);
         if (args.bulk_out && shares && (((uintptr_t)shares) & 15) == 0 && shares_bytes >= tt_gemm_tcgen05_shares_bytes()) {
@@ -1403,12 +1416,12 @@ static int gemm_dispatch(const void* x, long long ldx, const void* w, long long 
         return launch_pair<TOKENS_ON_M>(map_a, map_b, map_out, args, pair_tiles_m, pair_tiles, stream);
     }
     if (tokens > 128) {
-        if (!make_map(&map_a, x, tokens, k, ldx, BM) || !make_map(&map_b, w, features, k, ldw, 128)) return -1;
+        if (!make_map(&map_a, x, x_rows, k, ldx, BM) || !make_map(&map_b, w, features, k, ldw, 128)) return -1;
         const dim3 grid((features + 127) / 128, (tokens + BM - 1) / BM, splits);
         return launch<TOKENS_ON_M, 128, 3>(map_a, map_b, args, grid, stream);
     }
     const int bn = tokens <= 16 ? 16 : tokens <= 32 ? 32 : tokens <= 64 ? 64 : 128;
-    if (!make_map(&map_a, w, features, k, ldw, BM) || !make_map(&map_b, x, tokens, k, ldx, bn)) return -1;
+    if (!make_map(&map_a, w, features, k, ldw, BM) || !make_map(&map_b, x, x_rows, k, ldx, bn)) return -1;
     const dim3 grid(1, (features + BM - 1) / BM, splits);
     switch (bn) {
         case 16: return launch<FEATURES_ON_M, 16, 6, 2>(map_a, map_b, args, grid, stream);
@@ -1432,4 +1445,15 @@ extern "C" int tt_gemm_tcgen05_clamped(const void* x, long long ldx, const void*
                                        unsigned* status, cudaStream_t stream) {
     return gemm_dispatch(x, ldx, w, ldw, nullptr, out, ld_out, 0, tokens, features, k, 1, 1 + 16 * 3, status, stream, nullptr, 0,
                          GateClamp{clamp_low, clamp_high, clamp_alpha, clamp_split});
+}
+
+// The plain form with activations of their own for every `group_features` output features (the last group may be smaller):
+// x holds the groups' rows one after another, [groups][tokens][k].  group_features must be a multiple of the widest tile the
+// step's form uses: 256 for prompts (more than 128 tokens), 128 for fewer tokens.
+extern "C" int tt_gemm_tcgen05_groups(const void* x, long long ldx, const void* w, long long ldw, void* out, long long ld_out, long long split_stride,
+                                      int tokens, int features, int k, int splits, int group_features, unsigned* status, cudaStream_t stream,
+                                      void* shares, long long shares_bytes) {
+    if (group_features <= 0 || group_features % (tokens > 128 ? 256 : 128)) return (int)cudaErrorInvalidValue;
+    return gemm_dispatch(x, ldx, w, ldw, nullptr, out, ld_out, split_stride, tokens, features, k, splits, 0, status, stream, shares, shares_bytes,
+                         GateClamp{0.0f, 0.0f, 1.0f, 0}, group_features);
 }

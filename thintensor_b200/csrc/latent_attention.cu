@@ -15,7 +15,7 @@
 // key of a tile of 32 (16-byte loads along the row), online softmax, the weighted latents accumulated with every lane
 // taking 16 bytes of a latent at a time; the slice leaves (sum, maximum, denominator) in scratch memory.  (3) A block per
 // (token, head) combines the slices in order and applies Wv_h, a warp per output number, and multiplies the head by the
-// sigmoid of its gate number where the layer has one.
+// sigmoid of its gate number, or every output number by its own, where the layer has gates.
 //
 // Prompts may instead EXPAND the latents they can see into per-head keys and values for the step, laid out like blocks
 // of the ordinary cache (keys [block][head][64][dim + rot], values transposed [block][head][vdim][64]) with a table of
@@ -526,18 +526,20 @@ latent_decode_mma_kernel(const float* __restrict__ absorbed, const __nv_bfloat16
 template <typename TOut, typename TW>
 __global__ void latent_merge_expand_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml, int splits, int rank,
                                            int vdim, int heads, const TW* __restrict__ w_value, TOut* __restrict__ out,
-                                           const float* __restrict__ gate, int gate_splits, size_t gate_stride, int gate_row) {
+                                           const float* __restrict__ gate, int gate_splits, size_t gate_stride, int gate_row,
+                                           int gate_each) {
     tt_pdl_launch_dependents();
     tt_pdl_wait();
     extern __shared__ float lat_shared[];                       // rank, then splits
     const size_t row = blockIdx.x;
     const int h = (int)(row % heads);
-    float head_gate = 1.0f;                                     // sigmoid of the head's gate number, where the layer has one
-    if (gate) {
+    auto opened = [&](int column) {                             // sigmoid of the token's gate number at this column
         float z = 0.0f;
-        for (int s = 0; s < gate_splits; ++s) z += __ldg(gate + s * gate_stride + (row / heads) * (size_t)gate_row + h);
-        head_gate = 1.0f / (1.0f + expf(-z));
-    }
+        for (int s = 0; s < gate_splits; ++s) z += __ldg(gate + s * gate_stride + (row / heads) * (size_t)gate_row + column);
+        return 1.0f / (1.0f + expf(-z));
+    };
+    const float head_gate = gate && !gate_each ? opened(h) : 1.0f;
+    const bool each = gate && gate_each;
     const float* ml = part_ml + row * splits * 2;
     float m = -INFINITY;
     for (int s = 0; s < splits; ++s) m = fmaxf(m, ml[2 * s]);
@@ -560,6 +562,7 @@ __global__ void latent_merge_expand_kernel(const float* __restrict__ part_acc, c
     if (rank % VEC == 0) {                                      // 16 bytes of a row a load; four rows' loads in flight together
         for (int v0 = 4 * warp; v0 < vdim; v0 += 4 * warps) {
             float o[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+            const float own_gate = each && lane < 4 && v0 + lane < vdim ? opened(h * vdim + v0 + lane) : head_gate;     // asked for before the products
             for (int r = lane * VEC; r < rank; r += 32 * VEC) {
                 float w[4][VEC];
 #pragma unroll
@@ -575,7 +578,7 @@ __global__ void latent_merge_expand_kernel(const float* __restrict__ part_acc, c
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
                 const float total = tt_warp_sum(o[i]);
-                if (lane == 0 && v0 + i < vdim) out[row * vdim + v0 + i] = tt_from_float<TOut>(total * head_gate);
+                if (lane == i && v0 + i < vdim) out[row * vdim + v0 + i] = tt_from_float<TOut>(total * own_gate);
             }
         }
         return;
@@ -585,7 +588,7 @@ __global__ void latent_merge_expand_kernel(const float* __restrict__ part_acc, c
         float o = 0.0f;
         for (int r = lane; r < rank; r += 32) o = fmaf(lat_weight(wrow + r), lat_shared[r], o);
         o = tt_warp_sum(o);
-        if (lane == 0) out[row * vdim + v] = tt_from_float<TOut>(o * head_gate);
+        if (lane == 0) out[row * vdim + v] = tt_from_float<TOut>(o * (each ? opened(h * vdim + v) : head_gate));
     }
 }
 
@@ -614,7 +617,7 @@ extern "C" int tt_latent_attention(const float* q, int q_splits, long long q_str
                                    int vdim, int rank, const float* inv_freq, int rotary_dim, int interleaved, float rot_scale, float scale,
                                    int window, int splits, void* out, float* absorbed, float* part_acc, float* part_ml,
                                    int one_token_each, const float* gate, int gate_splits, long long gate_stride, int gate_row,
-                                   unsigned* status, cudaStream_t stream) {
+                                   int gate_each, unsigned* status, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (rank <= 0 || rank > LAT_MAX_RANK || rank + rot > LAT_MAX_ROW || dim <= 0 || dim > LAT_MAX_DIM || vdim <= 0 || splits < 1 ||
         splits > 65535 || rotary_dim > rot || (rotary_dim & 1) || !absorbed || !part_acc || !part_ml || q_row < heads * (dim + rot))
@@ -626,7 +629,7 @@ extern "C" int tt_latent_attention(const float* q, int q_splits, long long q_str
     const dim3 grid((unsigned)blocks, splits), block(LAT_WARPS * 32);
 #define TT_ABSORB(TW) tt_launch_pdl(latent_absorb_kernel<TW>, dim3((unsigned)rows), dim3(rank >= 512 ? 512 : rank >= 256 ? 256 : 128), (size_t)(dim + rot) * sizeof(float), stream, q, q_splits, (size_t)q_stride, q_row, (const TW*)w_key, cu, len_before, sequences, heads, dim, rot, rank, inv_freq, rotary_dim, interleaved, rot_scale, scale, absorbed)
 #define TT_ATT(TA) tt_launch_pdl(latent_attention_kernel<TA>, grid, block, shared, stream, (const float*)absorbed, (const TA*)pool, table, table_width, pool_blocks, cu, len_before, sequences, n_tokens, heads, rot, rank, window, splits, part_acc, part_ml, status)
-#define TT_MERGE(TA, TW) tt_launch_pdl(latent_merge_expand_kernel<TA, TW>, dim3((unsigned)rows), dim3(256), (size_t)(rank + splits) * sizeof(float), stream, (const float*)part_acc, (const float*)part_ml, splits, rank, vdim, heads, (const TW*)w_value, (TA*)out, gate, gate_splits, (size_t)gate_stride, gate_row)
+#define TT_MERGE(TA, TW) tt_launch_pdl(latent_merge_expand_kernel<TA, TW>, dim3((unsigned)rows), dim3(256), (size_t)(rank + splits) * sizeof(float), stream, (const float*)part_acc, (const float*)part_ml, splits, rank, vdim, heads, (const TW*)w_value, (TA*)out, gate, gate_splits, (size_t)gate_stride, gate_row, gate_each)
     if (weight_dtype == TT_F32) TT_ABSORB(float); else TT_ABSORB(__nv_bfloat16);
 #define TT_ATT_ROWS(TA) tt_launch_pdl(latent_attention_rows_kernel<TA>, grid, block, 0, stream, (const float*)absorbed, (const TA*)pool, table, table_width, pool_blocks, cu, len_before, sequences, n_tokens, heads, rot, rank, window, splits, part_acc, part_ml, status)
     const int piece = act_dtype == TT_F32 ? 4 : 8;              // numbers in 16 bytes of a cache row

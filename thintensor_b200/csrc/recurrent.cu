@@ -258,13 +258,15 @@ extern "C" int tt_causal_conv(const float* proj, int splits, long long split_str
 // what bounds the kernel once the grid fills the GPU (batches of prompts).
 // ROWS: every token brings a decay for each state row of its head (row_decay, float32 [tokens][groups * N], one more
 // vector staged beside B and C) instead of one for the head; step sizes are one and there is no skip.
-template <int K, int G, int C, bool ROWS>
+// BONUS (with ROWS): the token reads the state as it was before it and its own contribution by a weight for every state row of
+// its head (row_bonus, float32 [groups * N]): y = (S + diag(bonus) B x^T)^T C, then S = diag(decay) S + B x^T.
+template <int K, int G, int C, bool ROWS, bool BONUS>
 __global__ void __launch_bounds__(G* REC_LANES)
 mamba2_scan_kernel(const float* __restrict__ xbc, int xbc_cols, const float* __restrict__ proj, int splits, size_t split_stride,
                    int cols, int dt_col, const float* __restrict__ dt_bias, const float* __restrict__ a_log,
                    const float* __restrict__ d_skip, float* __restrict__ state, float* __restrict__ y,
                    const int* __restrict__ cu, const int* __restrict__ slots, int heads, int P, int N, int groups, int chunk,
-                   int vec, const float* __restrict__ fixed_decay, const float* __restrict__ row_decay) {
+                   int vec, const float* __restrict__ fixed_decay, const float* __restrict__ row_decay, const float* __restrict__ row_bonus) {
     tt_pdl_launch_dependents();
     tt_pdl_wait();
     extern __shared__ __align__(16) float rec_shared[];
@@ -285,6 +287,11 @@ mamba2_scan_kernel(const float* __restrict__ xbc, int xbc_cols, const float* __r
     const float neg_a = plain ? 0.0f : -expf(__ldg(a_log + h)), bias = plain ? 0.0f : __ldg(dt_bias + h);
     const float skip = plain ? 0.0f : __ldg(d_skip + h);
     const bool vec_x = vec && (width & 3) == 0;
+    float uv[BONUS ? K : 1];
+    if constexpr (BONUS) {
+#pragma unroll
+        for (int i = 0; i < K; ++i) uv[i] = rec_row(lane, i) < N ? __ldg(row_bonus + (size_t)g * N + rec_row(lane, i)) : 0.0f;
+    }
 
     auto stage = [&](int c0, float* base) {                      // asynchronous: B, C and x of tokens c0 .. of this sequence
         const int count = min(chunk, n - c0);
@@ -348,6 +355,14 @@ mamba2_scan_kernel(const float* __restrict__ xbc, int xbc_cols, const float* __r
                 float part0 = 0.0f, part1 = 0.0f;                // two chains, so that neighbouring rows do not wait for each other
 #pragma unroll
                 for (int i = 0; i < K; i += 2) {
+                    if constexpr (BONUS) {
+                        const float b0 = dx * bv[i], b1 = dx * bv[i + 1];
+                        part0 = fmaf(fmaf(uv[i], b0, s[c][i]), cv[i], part0);
+                        part1 = fmaf(fmaf(uv[i + 1], b1, s[c][i + 1]), cv[i + 1], part1);
+                        s[c][i] = fmaf(av[i], s[c][i], b0);
+                        s[c][i + 1] = fmaf(av[i + 1], s[c][i + 1], b1);
+                        continue;
+                    }
                     s[c][i] = fmaf(dx, bv[i], (ROWS ? av[ROWS ? i : 0] : a) * s[c][i]);
                     part0 = fmaf(s[c][i], cv[i], part0);
                     s[c][i + 1] = fmaf(dx, bv[i + 1], (ROWS ? av[ROWS ? i + 1 : 0] : a) * s[c][i + 1]);
@@ -403,8 +418,9 @@ static bool rec_aligned(const void* p, int a, int b, int c, int d) { return (((u
 static int mamba2_scan_launch(const float* xbc, int xbc_cols, const float* proj, int splits, long long split_stride, int cols,
                               int dt_col, const float* dt_bias, const float* a_log, const float* d_skip, float* state, float* y,
                               const int* cu, const int* slots, int sequences, int heads, int P, int N, int groups, int mode,
-                              const float* fixed_decay, const float* row_decay, cudaStream_t stream) {
+                              const float* fixed_decay, const float* row_decay, const float* row_bonus, cudaStream_t stream) {
     if (sequences <= 0) return 0;
+    if (row_bonus && !row_decay) return (int)cudaErrorInvalidValue;
     if (N <= 0 || N > REC_MAX_ROWS || P <= 0 || groups <= 0 || heads % groups || sequences > 65535) return (int)cudaErrorInvalidValue;
     const int vec = rec_aligned(xbc, xbc_cols, N, P, 0) && ((uintptr_t)row_decay & 15) == 0 ? 1 : 0;          // every row piece starts on 16 bytes
     const bool wide = rec_wide(mode, (long long)heads * sequences * ((P + REC_COLS - 1) / REC_COLS), N);
@@ -412,8 +428,8 @@ static int mamba2_scan_launch(const float* xbc, int xbc_cols, const float* proj,
     const dim3 grid(heads, sequences, (P + tile - 1) / tile), block((wide ? REC_WIDE_GROUPS : REC_COLS) * REC_LANES);
     const int vectors = row_decay ? 3 : 2, chunk = rec_chunk(N, tile, vectors);
     const size_t shared = rec_shared_bytes(N, chunk, tile, vectors);
-#define TT_SCAN_FORM(K, G, C, ROWS) tt_launch_pdl(mamba2_scan_kernel<K, G, C, ROWS>, grid, block, shared, stream, xbc, xbc_cols, proj, splits, (size_t)split_stride, cols, dt_col, dt_bias, a_log, d_skip, state, y, cu, slots, heads, P, N, groups, chunk, vec, fixed_decay, row_decay)
-#define TT_SCAN(K, G, C) do { if (row_decay) TT_SCAN_FORM(K, G, C, true); else TT_SCAN_FORM(K, G, C, false); } while (0)
+#define TT_SCAN_FORM(K, G, C, ROWS, BONUS) tt_launch_pdl(mamba2_scan_kernel<K, G, C, ROWS, BONUS>, grid, block, shared, stream, xbc, xbc_cols, proj, splits, (size_t)split_stride, cols, dt_col, dt_bias, a_log, d_skip, state, y, cu, slots, heads, P, N, groups, chunk, vec, fixed_decay, row_decay, row_bonus)
+#define TT_SCAN(K, G, C) do { if (row_bonus) TT_SCAN_FORM(K, G, C, true, true); else if (row_decay) TT_SCAN_FORM(K, G, C, true, false); else TT_SCAN_FORM(K, G, C, false, false); } while (0)
     if (wide) {
         if (N <= 8 * REC_LANES) TT_SCAN(8, REC_WIDE_GROUPS, REC_WIDE_COLS);
         else TT_SCAN(16, REC_WIDE_GROUPS, REC_WIDE_COLS);
@@ -432,7 +448,7 @@ extern "C" int tt_mamba2_scan(const float* xbc, int xbc_cols, const float* proj,
                               const int* cu, const int* slots, int sequences, int heads, int P, int N, int groups, int mode,
                               cudaStream_t stream) {
     return mamba2_scan_launch(xbc, xbc_cols, proj, splits, split_stride, cols, dt_col, dt_bias, a_log, d_skip, state, y, cu, slots,
-                              sequences, heads, P, N, groups, mode, nullptr, nullptr, stream);
+                              sequences, heads, P, N, groups, mode, nullptr, nullptr, nullptr, stream);
 }
 
 // ------------------------------------------------------------------------------------
@@ -445,16 +461,17 @@ extern "C" int tt_decay_scan(const float* vkq, int vkq_cols, const float* decay,
                              const int* slots, int sequences, int heads, int V, int D, int mode, cudaStream_t stream) {
     if (!decay) return (int)cudaErrorInvalidValue;
     return mamba2_scan_launch(vkq, vkq_cols, nullptr, 0, 0, 0, 0, nullptr, nullptr, nullptr, state, out, cu, slots, sequences, heads, V, D,
-                              heads, mode, decay, nullptr, stream);
+                              heads, mode, decay, nullptr, nullptr, stream);
 }
 
 // The same with decays that a token brings: S_t = diag(a_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t, a_t one number per head and
-// key channel (row_decay: float32 [tokens][heads * D]).
-extern "C" int tt_row_decay_scan(const float* vkq, int vkq_cols, const float* row_decay, float* state, float* out, const int* cu,
+// key channel (row_decay: float32 [tokens][heads * D]).  With a bonus (float32 [heads * D]) the token reads the state before it:
+// o_t = (S_(t-1) + diag(bonus) k_t v_t^T)^T q_t, the update as before.
+extern "C" int tt_row_decay_scan(const float* vkq, int vkq_cols, const float* row_decay, const float* bonus, float* state, float* out, const int* cu,
                                  const int* slots, int sequences, int heads, int V, int D, int mode, cudaStream_t stream) {
     if (!row_decay) return (int)cudaErrorInvalidValue;
     return mamba2_scan_launch(vkq, vkq_cols, nullptr, 0, 0, 0, 0, nullptr, nullptr, nullptr, state, out, cu, slots, sequences, heads, V, D,
-                              heads, mode, nullptr, row_decay, stream);
+                              heads, mode, nullptr, row_decay, bonus, stream);
 }
 
 // q, k and v of a linear attention from the partial sums of its input projection (columns [q | k | v | ...], q and k
@@ -722,6 +739,7 @@ struct RowScan {
     int splits, cols, b_col;
     size_t split_stride;
     float q_scale;
+    const float* bonus;         // [heads * D]: a token reads the state before it and its own contribution times this (not with the delta rule)
     float* state;               // [slots][heads][V][D]
     float* out;                 // [tokens][heads * V]
     const int* cu;
@@ -750,7 +768,7 @@ __device__ __forceinline__ float rb_scatter_sum(float (&v)[N], int lane) {
 constexpr uint32_t RB_T = 1u | 2u << 2 | 2u << 4 | 3u << 6 | 3u << 8 | 3u << 10 | 0u << 12 | 1u << 14 | 1u << 16 | 2u << 18 | 2u << 20 | 2u << 22 | 3u << 24 | 3u << 26 | 3u << 28 | 3u << 30;
 constexpr uint32_t RB_J = 0u | 0u << 2 | 1u << 4 | 0u << 6 | 1u << 8 | 2u << 10 | 0u << 12 | 0u << 14 | 1u << 16 | 0u << 18 | 1u << 20 | 2u << 22 | 0u << 24 | 1u << 26 | 2u << 28 | 3u << 30;
 
-template <int K, bool DELTA>
+template <int K, bool DELTA, bool BONUS>
 __global__ void __launch_bounds__(RB_THREADS)
 row_decay_blocks_kernel(const RowScan a) {
     tt_pdl_launch_dependents();
@@ -774,6 +792,11 @@ row_decay_blocks_kernel(const RowScan a) {
         const int mine = warp - RB_SCAN_WARPS, g = h / (a.heads / a.qk_heads);
         auto row_of = [&](int e) { return E == 8 ? 4 * lane + 128 * (e >> 2) + (e & 3) : E * lane + e; };
         float q[4][E], k[4][E], d[4][E], v[2], raw = 0.0f;
+        float bonus[BONUS ? E : 1];
+        if constexpr (BONUS) {
+#pragma unroll
+            for (int e = 0; e < E; ++e) bonus[e] = row_of(e) < D ? __ldg(a.bonus + (size_t)h * D + row_of(e)) : 0.0f;
+        }
         const int v_token = lane >> 3, v_col = 2 * (lane & 7);
         auto load_row = [&](float (&x)[E], const float* row, float missing, bool live) {
             constexpr int W = E < 4 ? E : 4;                    // numbers of a load
@@ -833,9 +856,14 @@ row_decay_blocks_kernel(const RowScan a) {
 #pragma unroll
                     for (int j = 0; j < 4; ++j) {
                         float w = k[j][e];
-                        sums[B_AT + j * (j + 1) / 2 + j] = fmaf(q[j][e], w, sums[B_AT + j * (j + 1) / 2 + j]);
+                        sums[B_AT + j * (j + 1) / 2 + j] = fmaf(q[j][e], BONUS ? bonus[BONUS ? e : 0] * w : w, sums[B_AT + j * (j + 1) / 2 + j]);
 #pragma unroll
                         for (int t = j + 1; t < 4; ++t) {
+                            if (BONUS) {                        // the query meets the state before its own token's decay
+                                sums[B_AT + t * (t + 1) / 2 + j] = fmaf(q[t][e], w, sums[B_AT + t * (t + 1) / 2 + j]);
+                                w *= d[t][e];
+                                continue;
+                            }
                             w *= d[t][e];
                             if (DELTA) sums[A_AT + t * (t - 1) / 2 + j] = fmaf(k[t][e], w, sums[A_AT + t * (t - 1) / 2 + j]);
                             sums[B_AT + t * (t + 1) / 2 + j] = fmaf(q[t][e], w, sums[B_AT + t * (t + 1) / 2 + j]);
@@ -880,7 +908,11 @@ row_decay_blocks_kernel(const RowScan a) {
                 for (int t = 0; t < 4; ++t) {
                     float x[E];
 #pragma unroll
-                    for (int e = 0; e < E; ++e) { p[e] *= d[t][e]; x[e] = q[t][e] * p[e] * nq[t]; }
+                    for (int e = 0; e < E; ++e) {
+                        const float before = p[e];
+                        p[e] *= d[t][e];
+                        x[e] = q[t][e] * (BONUS ? before : p[e]) * nq[t];
+                    }
                     put(base + Q_AT + t * DP, x);
                     if (DELTA) {
 #pragma unroll
@@ -1018,44 +1050,49 @@ row_decay_blocks_kernel(const RowScan a) {
         }
 }
 
-template <int K, bool DELTA>
+template <int K, bool DELTA, bool BONUS>
 static int row_decay_blocks_launch(const RowScan& scan, int sequences, cudaStream_t stream) {
     constexpr size_t shared = (size_t)2 * RB_BLOCKS * (((DELTA ? 3 : 2) * RB_BLOCK + 1) * K * RB_LANES + RB_SCALARS) * sizeof(float);
     static bool allowed = false;
     if (!allowed) {
-        const cudaError_t code = cudaFuncSetAttribute(row_decay_blocks_kernel<K, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
+        const cudaError_t code = cudaFuncSetAttribute(row_decay_blocks_kernel<K, DELTA, BONUS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
         if (code != cudaSuccess) return (int)code;
         allowed = true;
     }
-    tt_launch_pdl(row_decay_blocks_kernel<K, DELTA>, dim3(scan.heads, sequences, (scan.V + RB_TILE - 1) / RB_TILE), dim3(RB_THREADS), shared, stream, scan);
+    tt_launch_pdl(row_decay_blocks_kernel<K, DELTA, BONUS>, dim3(scan.heads, sequences, (scan.V + RB_TILE - 1) / RB_TILE), dim3(RB_THREADS), shared, stream, scan);
     TT_LAUNCH_CHECK();
 }
 
 // delta != 0: the delta rule (q and k are made unit vectors, q also times q_scale; beta from proj); else linear attention (q times q_scale)
 extern "C" int tt_row_decay_blocks(const float* q, const float* k, const float* v, long long row_stride, const float* decay, int delta,
-                                   const float* proj, int splits, long long split_stride, int cols, int b_col, float q_scale, float* state,
+                                   const float* proj, int splits, long long split_stride, int cols, int b_col, float q_scale, const float* bonus, float* state,
                                    float* out, const int* cu, const int* slots, int sequences, int heads, int qk_heads, int D, int V,
                                    cudaStream_t stream) {
     if (sequences <= 0) return 0;
     if (!q || !k || !v || !decay || D <= 0 || D > REC_MAX_ROWS || V <= 0 || qk_heads <= 0 || heads % qk_heads || sequences > 65535) return (int)cudaErrorInvalidValue;
-    if (delta && !proj) return (int)cudaErrorInvalidValue;
+    if (delta && (!proj || bonus)) return (int)cudaErrorInvalidValue;
     const uintptr_t bases = (uintptr_t)q | (uintptr_t)k | (uintptr_t)decay;
-    const RowScan scan{q, k, v, (size_t)row_stride, decay, proj, splits, cols, b_col, (size_t)split_stride, q_scale, state, out, cu, slots,
+    const RowScan scan{q, k, v, (size_t)row_stride, decay, proj, splits, cols, b_col, (size_t)split_stride, q_scale, bonus, state, out, cu, slots,
                        heads, qk_heads, D, V, (bases & 15) == 0 && !(D & 3) && !(row_stride & 3) ? 1 : 0};
-    if (D <= 4 * RB_LANES) return delta ? row_decay_blocks_launch<4, true>(scan, sequences, stream) : row_decay_blocks_launch<4, false>(scan, sequences, stream);
-    if (D <= 8 * RB_LANES) return delta ? row_decay_blocks_launch<8, true>(scan, sequences, stream) : row_decay_blocks_launch<8, false>(scan, sequences, stream);
-    return delta ? row_decay_blocks_launch<16, true>(scan, sequences, stream) : row_decay_blocks_launch<16, false>(scan, sequences, stream);
+#define TT_BLOCKS(K) (delta ? row_decay_blocks_launch<K, true, false>(scan, sequences, stream) : bonus ? row_decay_blocks_launch<K, false, true>(scan, sequences, stream) \
+                                                                                               : row_decay_blocks_launch<K, false, false>(scan, sequences, stream))
+    if (D <= 4 * RB_LANES) return TT_BLOCKS(4);
+    if (D <= 8 * RB_LANES) return TT_BLOCKS(8);
+    return TT_BLOCKS(16);
+#undef TT_BLOCKS
 }
 
 // ------------------------------------------------------------------------------------
 // Products of low rank: z[t, j] = sum_r W[j, r] * x[t, r] with x the columns x_col .. x_col + rank - 1 of a projection's
 // partial sums, and what is made of z at once (kind):
 //   0: z      1: exp(-exp(a_log[h]) * softplus(z + bias[j])), h = j / per_head      2: sigmoid(z + bias[j]) ^ inv_tau
+//   3: exp(-exp(z + bias[j]))
+// x may pass tanh first (tanh_x).
 // Up to two such products of one projection in one launch (blockIdx.z).  All float32; W is stored [rank][n] (transposed, so
 // that neighbouring threads read neighbouring numbers) in either element type.
 // ------------------------------------------------------------------------------------
 struct LowRankPart {
-    int x_col, rank, n, kind, per_head;
+    int x_col, rank, n, kind, per_head, tanh_x;
     const void* w;
     const float* bias;
     const float* a_log;
@@ -1067,6 +1104,7 @@ struct LowRankParts { LowRankPart part[2]; };
 __device__ __forceinline__ float low_rank_finish(const LowRankPart& p, float z, int j) {
     if (p.kind == 1) return expf(-expf(__ldg(p.a_log + j / p.per_head)) * rec_softplus(z + __ldg(p.bias + j)));
     if (p.kind == 2) return expf(-rec_softplus(-(z + __ldg(p.bias + j))) * p.inv_tau);
+    if (p.kind == 3) return expf(-expf(z + __ldg(p.bias + j)));
     return z;
 }
 
@@ -1119,7 +1157,7 @@ low_rank_few_kernel(const float* __restrict__ proj, int splits, size_t split_str
                     for (int s = 0; s < LRF_SLICES; ++s) total += v[s];
                 }
             }
-            xs[r * LRF_TOKENS + t] = total;
+            xs[r * LRF_TOKENS + t] = p.tanh_x ? tanhf(total) : total;
         }
         __syncthreads();
 #pragma unroll
@@ -1152,26 +1190,27 @@ low_rank_few_kernel(const float* __restrict__ proj, int splits, size_t split_str
 // Prompts: the products themselves are matrix products like any other (the caller's); here are their inputs, columns of a
 // projection's partial sums in the activation dtype, and what is made of their results, in place.
 template <typename TAct>
-__global__ void low_rank_inputs_kernel(const float* __restrict__ proj, int splits, size_t split_stride, int cols, int col0, int width0,
-                                       TAct* __restrict__ out0, int col1, int width1, TAct* __restrict__ out1) {
+__global__ void low_rank_inputs_kernel(const float* __restrict__ proj, int splits, size_t split_stride, int cols, int col0, int width0, int tanh0,
+                                       TAct* __restrict__ out0, int col1, int width1, int tanh1, TAct* __restrict__ out1) {
     tt_pdl_launch_dependents();
     tt_pdl_wait();
     const float* row = proj + (size_t)blockIdx.x * cols;
     for (int r = threadIdx.x; r < width0 + width1; r += blockDim.x) {
         const bool second = r >= width0;
-        const float x = rec_sum_slices(row + (second ? col1 + r - width0 : col0 + r), splits, split_stride);
+        float x = rec_sum_slices(row + (second ? col1 + r - width0 : col0 + r), splits, split_stride);
+        if (second ? tanh1 : tanh0) x = tanhf(x);
         if (second) out1[(size_t)blockIdx.x * width1 + r - width0] = tt_from_float<TAct>(x);
         else out0[(size_t)blockIdx.x * width0 + r] = tt_from_float<TAct>(x);
     }
 }
 
-extern "C" int tt_low_rank_inputs(const float* proj, int splits, long long split_stride, int cols, int col0, int width0, void* out0, int col1,
-                                  int width1, void* out1, int out_dtype, int n_tokens, cudaStream_t stream) {
+extern "C" int tt_low_rank_inputs(const float* proj, int splits, long long split_stride, int cols, int col0, int width0, int tanh0, void* out0,
+                                  int col1, int width1, int tanh1, void* out1, int out_dtype, int n_tokens, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (width0 < 1 || width1 < 0 || col0 < 0 || col0 + width0 > cols || (width1 && (!out1 || col1 < 0 || col1 + width1 > cols))) return (int)cudaErrorInvalidValue;
     const int threads = width0 + width1 <= 64 ? 64 : (width0 + width1 <= 128 ? 128 : 256);
-    if (out_dtype == TT_F32) tt_launch_pdl(low_rank_inputs_kernel<float>, dim3(n_tokens), dim3(threads), 0, stream, proj, splits, (size_t)split_stride, cols, col0, width0, (float*)out0, col1, width1, (float*)out1);
-    else tt_launch_pdl(low_rank_inputs_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(threads), 0, stream, proj, splits, (size_t)split_stride, cols, col0, width0, (__nv_bfloat16*)out0, col1, width1, (__nv_bfloat16*)out1);
+    if (out_dtype == TT_F32) tt_launch_pdl(low_rank_inputs_kernel<float>, dim3(n_tokens), dim3(threads), 0, stream, proj, splits, (size_t)split_stride, cols, col0, width0, tanh0, (float*)out0, col1, width1, tanh1, (float*)out1);
+    else tt_launch_pdl(low_rank_inputs_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(threads), 0, stream, proj, splits, (size_t)split_stride, cols, col0, width0, tanh0, (__nv_bfloat16*)out0, col1, width1, tanh1, (__nv_bfloat16*)out1);
     TT_LAUNCH_CHECK();
 }
 
@@ -1185,14 +1224,14 @@ __global__ void low_rank_finish_kernel(const float* z, int splits, size_t split_
     const size_t at = (size_t)blockIdx.x * p.n + j;
     float x = bias;
     for (int s = 0; s < splits; ++s) x += z[(size_t)s * split_stride + at];
-    p.out[at] = p.kind == 1 ? expf(rate * rec_softplus(x)) : expf(-rec_softplus(-x) * p.inv_tau);
+    p.out[at] = p.kind == 1 ? expf(rate * rec_softplus(x)) : p.kind == 2 ? expf(-rec_softplus(-x) * p.inv_tau) : expf(-expf(x));
 }
 
 extern "C" int tt_low_rank_finish(const float* z, int splits, long long split_stride, int n, int kind, int per_head, const float* bias,
                                   const float* a_log, float inv_tau, float* out, int n_tokens, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (n < 1 || (kind != 1 && kind != 2) || !bias || (kind == 1 && (!a_log || per_head < 1))) return (int)cudaErrorInvalidValue;
-    const LowRankPart p{0, 0, n, kind, per_head, nullptr, bias, a_log, inv_tau, out};
+    if (n < 1 || kind < 1 || kind > 3 || !bias || (kind == 1 && (!a_log || per_head < 1))) return (int)cudaErrorInvalidValue;
+    const LowRankPart p{0, 0, n, kind, per_head, 0, nullptr, bias, a_log, inv_tau, out};
     const int threads = 256;
     const unsigned blocks = (unsigned)((n + threads - 1) / threads);
     if (blocks > 65535) return (int)cudaErrorInvalidValue;
@@ -1201,18 +1240,18 @@ extern "C" int tt_low_rank_finish(const float* z, int splits, long long split_st
 }
 
 extern "C" int tt_low_rank(const float* proj, int splits, long long split_stride, int cols, int n_parts, int w_dtype,
-                           int x_col0, int rank0, int n0, int kind0, int per_head0, const void* w0, const float* bias0, const float* a_log0, float inv_tau0, float* out0,
-                           int x_col1, int rank1, int n1, int kind1, int per_head1, const void* w1, const float* bias1, const float* a_log1, float inv_tau1, float* out1,
+                           int x_col0, int rank0, int n0, int kind0, int per_head0, int tanh0, const void* w0, const float* bias0, const float* a_log0, float inv_tau0, float* out0,
+                           int x_col1, int rank1, int n1, int kind1, int per_head1, int tanh1, const void* w1, const float* bias1, const float* a_log1, float inv_tau1, float* out1,
                            int n_tokens, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (n_parts < 1 || n_parts > 2) return (int)cudaErrorInvalidValue;
     LowRankParts parts;
-    parts.part[0] = LowRankPart{x_col0, rank0, n0, kind0, per_head0, w0, bias0, a_log0, inv_tau0, out0};
-    parts.part[1] = n_parts > 1 ? LowRankPart{x_col1, rank1, n1, kind1, per_head1, w1, bias1, a_log1, inv_tau1, out1} : parts.part[0];
+    parts.part[0] = LowRankPart{x_col0, rank0, n0, kind0, per_head0, tanh0, w0, bias0, a_log0, inv_tau0, out0};
+    parts.part[1] = n_parts > 1 ? LowRankPart{x_col1, rank1, n1, kind1, per_head1, tanh1, w1, bias1, a_log1, inv_tau1, out1} : parts.part[0];
     int widest = 0;
     for (int i = 0; i < n_parts; ++i) {
         const LowRankPart& p = parts.part[i];
-        if (p.rank < 1 || p.n < 1 || p.x_col < 0 || p.x_col + p.rank > cols || p.kind < 0 || p.kind > 2) return (int)cudaErrorInvalidValue;
+        if (p.rank < 1 || p.n < 1 || p.x_col < 0 || p.x_col + p.rank > cols || p.kind < 0 || p.kind > 3) return (int)cudaErrorInvalidValue;
         if ((p.kind && !p.bias) || (p.kind == 1 && (!p.a_log || p.per_head < 1))) return (int)cudaErrorInvalidValue;
         widest = p.n > widest ? p.n : widest;
     }

@@ -14,6 +14,8 @@
 //
 // tt_expert_activation: the clamped gated unit of every expert's columns times the token's gate for that expert.
 //
+// tt_expert_unary_activation: the same for experts without a gate projection.
+//
 // tt_scale_expert_columns: act[t][e * width + j] *= gates[t][e] for the first experts * width columns of act; the next
 // shared_width columns (an always-on expert's) are multiplied by gates[t][experts], and columns behind those stay as they are.
 #include "common.cuh"
@@ -36,6 +38,7 @@ __device__ __forceinline__ void route_argmax(float& value, int& index) {
 //   correction (float32 [experts] or null): added to the scores for the CHOICE only (groups and top); weights use the scores.
 //   group_top2: a group's score is the sum of its two largest choice scores (its only one, for groups of one expert).
 //   plain_weights: the weights are the chosen scores themselves instead of score / (sum of the chosen + 1e-20).
+//   weight_scale: a factor on the weights, however they are made (not on the always-on experts' gates).
 //   extra: so many more logits follow the experts'; gates[t][experts + k] = sigmoid(logit) for each (the gate of an
 //   expert that every token uses).  A row of `gates` has experts + extra numbers.
 struct RouteOptions {
@@ -44,6 +47,7 @@ struct RouteOptions {
     int group_top2;
     int plain_weights;
     int extra;
+    float weight_scale;
 };
 
 // One warp routes token t from its logits (`splits` partial sums `split_stride` apart); group_best: 32 floats of the warp's own.
@@ -154,7 +158,7 @@ __device__ __forceinline__ void route_token(const float* __restrict__ logits, in
         sum += score;
         if (lane == round) { mine = e; mine_score = score; }
     }
-    const float scale = opt.plain_weights ? 1.0f : 1.0f / (sum + 1e-20f);
+    const float scale = opt.weight_scale * (opt.plain_weights ? 1.0f : 1.0f / (sum + 1e-20f));
     if (lane < top) {
         chosen[(size_t)t * top + lane] = mine;
         weights[(size_t)t * top + lane] = mine >= 0 ? mine_score * scale : 0.0f;
@@ -226,12 +230,12 @@ __global__ void scale_expert_columns_kernel(T* __restrict__ act, int row_stride,
 
 extern "C" int tt_route_topk(const float* logits, int splits, long long split_stride, int n_tokens, int experts, int top, int groups,
                              int keep, float* gates, int* chosen, float* weights, int sigmoid, const float* correction,
-                             int group_top2, int plain_weights, int extra, cudaStream_t stream) {
+                             int group_top2, int plain_weights, int extra, float weight_scale, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (experts <= 0 || experts > ROUTE_MAX_EXPERTS || top < 1 || top > 32 || top > experts || groups < 1 || groups > 32 ||
         experts % groups || keep < 1 || keep > groups || extra < 0 || extra > 32)
         return (int)cudaErrorInvalidValue;
-    const RouteOptions opt{sigmoid, correction, group_top2, plain_weights, extra};
+    const RouteOptions opt{sigmoid, correction, group_top2, plain_weights, extra, weight_scale};
     tt_launch_pdl(route_topk_kernel, dim3((n_tokens + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), 0, stream, logits, splits,
                   (size_t)split_stride, n_tokens, experts, top, groups, keep, gates, chosen, weights, opt);
     TT_LAUNCH_CHECK();
@@ -259,12 +263,12 @@ __global__ void scale_expert_columns_vec_kernel(T* __restrict__ act, int row_str
 
 extern "C" int tt_route_rows(const void* x, int x_dtype, const void* w, int w_dtype, int hidden, int n_tokens, int experts, int top,
                              int groups, int keep, float* gates, int* chosen, float* weights, int sigmoid, const float* correction,
-                             int group_top2, int plain_weights, int extra, cudaStream_t stream) {
+                             int group_top2, int plain_weights, int extra, float weight_scale, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (experts <= 0 || experts > ROUTE_MAX_EXPERTS || top < 1 || top > 32 || top > experts || groups < 1 || groups > 32 ||
         experts % groups || keep < 1 || keep > groups || extra < 0 || extra > 32)
         return (int)cudaErrorInvalidValue;
-    const RouteOptions opt{sigmoid, correction, group_top2, plain_weights, extra};
+    const RouteOptions opt{sigmoid, correction, group_top2, plain_weights, extra, weight_scale};
     const size_t shared = (size_t)(hidden + experts + extra + 32) * sizeof(float);
     if (shared > 48 * 1024) return (int)cudaErrorInvalidValue;
 #define TT_ROUTE(TX, TW) tt_launch_pdl(route_rows_kernel<TX, TW>, dim3(n_tokens), dim3(n_tokens <= 256 ? 512 : 128), shared, stream, (const TX*)x, (const TW*)w, hidden, n_tokens, experts, top, groups, keep, gates, chosen, weights, opt)
@@ -347,5 +351,66 @@ extern "C" int tt_expert_activation(const float* gate_up, int splits, long long 
         tt_launch_pdl(expert_activation_kernel<float>, dim3((unsigned)blocks), dim3(threads), 0, stream, gate_up, splits, (size_t)split_stride, (float*)act, experts, width, shared_width, limit, shared_limit, alpha, gates, gate_row, shared_gated, total);
     else
         tt_launch_pdl(expert_activation_kernel<__nv_bfloat16>, dim3((unsigned)blocks), dim3(threads), 0, stream, gate_up, splits, (size_t)split_stride, (__nv_bfloat16*)act, experts, width, shared_width, limit, shared_limit, alpha, gates, gate_row, shared_gated, total);
+    TT_LAUNCH_CHECK();
+}
+
+// ------------------------------------------------------------------------------------
+// Experts without a gate projection: act[t][c] = f(sum over slices of up[s][t][c]) * gates[t][c / width].
+// up: float32 [splits][tokens][experts * width].  f by `activation`: 0 silu, 1 relu, 2 the tanh form of gelu, 4 the exact gelu, 5 the
+// square of relu.  Columns of experts the token did not choose are zero without being read.  A thread takes VEC neighbouring
+// columns of one expert.
+// ------------------------------------------------------------------------------------
+__device__ __forceinline__ float expert_unary(float z, int activation) {
+    if (activation == 5) { const float p = fmaxf(z, 0.0f); return p * p; }
+    if (activation == 1) return fmaxf(z, 0.0f);
+    if (activation == 2) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+    if (activation == 4) return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f));
+    return z / (1.0f + expf(-z));
+}
+
+template <typename T, int N> struct alignas(N * sizeof(T)) ExpertPack { T v[N]; };
+
+template <typename TAct, int VEC>
+__global__ void expert_unary_activation_kernel(const float* __restrict__ up, int splits, size_t split_stride, TAct* __restrict__ act, int experts,
+                                               int width, int activation, const float* __restrict__ gates, int gate_row, long long total) {
+    tt_pdl_launch_dependents();
+    tt_pdl_wait();
+    const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * VEC;
+    if (i >= total) return;
+    const int cols = experts * width;
+    const long long t = i / cols;
+    const int c = (int)(i - t * cols);
+    const float weight = gates[t * gate_row + c / width];
+    float z[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) z[e] = 0.0f;
+    if (weight != 0.0f) {
+        for (int s = 0; s < splits; ++s) {
+            const ExpertPack<float, VEC> x = *reinterpret_cast<const ExpertPack<float, VEC>*>(up + (size_t)s * split_stride + i);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) z[e] += x.v[e];
+        }
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) z[e] = expert_unary(z[e], activation) * weight;
+    }
+    ExpertPack<TAct, VEC> o;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) o.v[e] = tt_from_float<TAct>(z[e]);
+    *reinterpret_cast<ExpertPack<TAct, VEC>*>(act + i) = o;
+}
+
+extern "C" int tt_expert_unary_activation(const float* up, int splits, long long split_stride, void* act, int act_dtype, int n_tokens, int experts,
+                                          int width, int activation, const float* gates, int gate_row, cudaStream_t stream) {
+    const long long total = (long long)n_tokens * experts * width;
+    if (total <= 0) return 0;
+    if (activation < 0 || activation > 5 || activation == 3 || gate_row < experts) return (int)cudaErrorInvalidValue;
+    const bool wide = width % 4 == 0 && split_stride % 4 == 0 && (((uintptr_t)up | (uintptr_t)act) & 15) == 0;
+    const int threads = 256;
+    const long long per_block = (long long)threads * (wide ? 4 : 1), blocks = (total + per_block - 1) / per_block;
+    if (blocks > 2147483647LL) return (int)cudaErrorInvalidValue;
+#define TT_UNARY(T, V) tt_launch_pdl(expert_unary_activation_kernel<T, V>, dim3((unsigned)blocks), dim3(threads), 0, stream, up, splits, (size_t)split_stride, (T*)act, experts, width, activation, gates, gate_row, total)
+    if (act_dtype == TT_F32) { if (wide) TT_UNARY(float, 4); else TT_UNARY(float, 1); }
+    else { if (wide) TT_UNARY(__nv_bfloat16, 4); else TT_UNARY(__nv_bfloat16, 1); }
+#undef TT_UNARY
     TT_LAUNCH_CHECK();
 }

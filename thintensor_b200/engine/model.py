@@ -15,7 +15,7 @@ import torch
 
 from ..cache.cache import SequenceCache
 from ..parts import ARRANGEMENTS, EMBEDDINGS, HEADS, NORMS, REGISTRIES
-from ..parts.base import Delta, Part, WeightDecl
+from ..parts.base import Delta, Part, StreamStep, WeightDecl
 from ..parts.spec import ModelSpec, PartSpec
 from .context import StepContext
 
@@ -166,13 +166,15 @@ class DecoderModel:
         matrix whatever the number of positions) are not run and nothing is returned."""
         if not self.bound:
             raise RuntimeError("the model has no weights yet")
-        residual = ctx.scratch("model.residual", (ctx.n_tokens, self.spec.hidden_size), torch.float32)
-        self.embedding.part.forward(ctx, ctx.tokens, residual, None if self.embedding_entry is None else cache.run_state(self.embedding_entry))
+        copies = self.spec.streams          # a stream in several copies; the embedding fills the first, the first norm spreads it
+        shape = (ctx.n_tokens, self.spec.hidden_size)
+        residual = ctx.scratch("model.residual", shape if copies is None else (copies, *shape), torch.float32)
+        self.embedding.part.forward(ctx, ctx.tokens, residual if copies is None else residual[0], None if self.embedding_entry is None else cache.run_state(self.embedding_entry))
         embedded = None
         if any(run.add_embedding for run in self.spec.schedule):          # kept for the runs that start by adding it
             embedded = ctx.scratch("model.embedded", (ctx.n_tokens, self.spec.hidden_size), torch.float32)
             embedded.copy_(residual)
-        pending: Delta | None = None
+        pending: Delta | None = None if copies is None else Delta(None, streams=StreamStep(spread=True))
         for index, run in enumerate(self.spec.schedule):
             users = self.users[index]
             if run.add_embedding:

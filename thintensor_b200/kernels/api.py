@@ -74,6 +74,14 @@ def _need(t: torch.Tensor, dtype: torch.dtype, name: str) -> None:
         raise KernelError(f"{name} must be contiguous")
 
 
+def _need_columns(t: torch.Tensor, dtype: torch.dtype, name: str) -> None:
+    """Like :func:`_need` for a product's output, which may be a range of the columns of a wider matrix."""
+    if t.dtype != dtype:
+        raise KernelError(f"{name} must be {dtype}, got {t.dtype}")
+    if t.stride(-1) != 1:
+        raise KernelError(f"{name} must have its columns side by side")
+
+
 _functions: dict[str, object] = {}
 
 
@@ -167,6 +175,21 @@ def embed_gather(table: torch.Tensor, tokens: torch.Tensor, residual: torch.Tens
     _check(fn(_ptr(table), dtype_code(table.dtype), _ptr(tokens), _ptr(residual), n, hidden, table.shape[0], scale, _ptr(status), _stream()), "embed_gather")
 
 
+def embed_norm_gather(table: torch.Tensor, tokens: torch.Tensor, weight: torch.Tensor, eps: float, residual: torch.Tensor, scale: float,
+                      status: torch.Tensor) -> None:
+    """residual[t] = rmsnorm(table[tokens[t]] * scale) * weight, float32 out."""
+    _need(tokens, torch.int32, "tokens")
+    _need(residual, torch.float32, "residual")
+    _need(weight, torch.float32, "norm weight")
+    n, hidden = tokens.numel(), table.shape[1]
+    if not table.is_contiguous() or weight.numel() != hidden or tuple(residual.shape) != (n, hidden):
+        raise KernelError("embed_norm_gather: shapes do not fit")
+    fn = _fn("elementwise", "tt_embed_norm_gather", [c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_float, c_void_p,
+                                                     c_void_p])
+    _check(fn(_ptr(table), dtype_code(table.dtype), _ptr(tokens), _ptr(weight), eps, _ptr(residual), n, hidden, table.shape[0], scale, _ptr(status),
+              _stream()), "embed_norm_gather")
+
+
 def embed_position_gather(table: torch.Tensor, positions: torch.Tensor, tokens: torch.Tensor, cu: torch.Tensor, len_before: torch.Tensor,
                           sequences: int, residual: torch.Tensor, scale: float, status: torch.Tensor) -> None:
     """residual[t] = table[tokens[t]] * scale + positions[p] with p the position of packed token t in its sequence."""
@@ -217,6 +240,68 @@ def token_shift(x: torch.Tensor, mix: torch.Tensor, state: torch.Tensor, out: to
     fn = _fn("elementwise", "tt_token_shift", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
     _check(fn(_ptr(x), dtype_code(x.dtype), _ptr(mix), _ptr(state), _ptr(out), _ptr(cu), _ptr(slots), sequences, tokens, hidden, _stream()),
            "token_shift")
+
+
+SHIFT_BLENDS = 8            # most blends of one token_shifts call (SHIFT_BLENDS in csrc/elementwise.cu)
+
+
+def token_shifts(x: torch.Tensor, mix: torch.Tensor, state: torch.Tensor, out: torch.Tensor, cu: torch.Tensor, slots: torch.Tensor,
+                 sequences: int) -> None:
+    """Several blends of the same rows, ``out[m, t] = x[t] + (x[t - 1] - x[t]) * mix[m]`` (``mix`` float32 ``[blends, hidden]``,
+    ``out`` ``[blends, tokens, hidden]``); the state as for :func:`token_shift`, one row per sequence."""
+    _need(mix, torch.float32, "shift weights")
+    _need(state, torch.float32, "shift state")
+    tokens, hidden = x.shape
+    blends = mix.shape[0]
+    if (x.dtype != out.dtype or not x.is_contiguous() or not out.is_contiguous() or tuple(out.shape) != (blends, tokens, hidden)
+            or tuple(mix.shape) != (blends, hidden) or state.shape[1] != hidden):
+        raise KernelError("token_shifts: shapes do not fit")
+    if not 1 <= blends <= SHIFT_BLENDS:
+        raise KernelError(f"token_shifts makes 1 to {SHIFT_BLENDS} blends, not {blends}")
+    fn = _fn("elementwise", "tt_token_shifts", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int,
+                                                c_int, c_void_p])
+    _check(fn(_ptr(x), dtype_code(x.dtype), _ptr(mix), blends, _ptr(state), _ptr(out), out.stride(0), _ptr(cu), _ptr(slots), sequences, tokens,
+              hidden, _stream()), "token_shifts")
+
+
+MAX_STREAMS = 16            # STREAMS_MAX in csrc/streams.cu
+
+
+def stream_norm(streams: torch.Tensor, delta: torch.Tensor | None, scale: float, gain: torch.Tensor | None, mix: torch.Tensor | None,
+                write: torch.Tensor | None, read: torch.Tensor | None, spread: bool, weight: torch.Tensor, weight_offset: float, eps: float,
+                out: torch.Tensor, rows: torch.Tensor | None = None) -> None:
+    """A residual stream in several copies, ``streams`` float32 ``[copies, tokens, hidden]`` (or ``[tokens, hidden]``: one): with
+    ``y = scale * gain * sum(delta)`` copy t becomes ``sum(mix[s, t] * x_s) + write[t] * y``, all at once from the old copies, and
+    ``out`` is the RMS norm of ``sum(read[t] * x_t)``.  ``mix`` None: the copies stay; ``write``, ``read``, ``gain`` None: ones.
+    ``spread``: only copy 0 is there, and all start equal to it.  ``rows`` as for :func:`add_rmsnorm`."""
+    _need(streams, torch.float32, "streams")
+    _need(weight, torch.float32, "norm weight")
+    copies = 1 if streams.dim() == 2 else streams.shape[0]
+    tokens, hidden = streams.shape[-2:]
+    if not 1 <= copies <= MAX_STREAMS:
+        raise KernelError(f"stream_norm takes 1 to {MAX_STREAMS} streams, got {copies}")
+    for t, count, name in ((gain, hidden, "channel factors"), (mix, copies * copies, "mixing weights"), (write, copies, "writing weights"),
+                           (read, copies, "reading weights"), (weight, hidden, "norm weight")):
+        if t is not None:
+            _need(t, torch.float32, name)
+            if t.numel() != count:
+                raise KernelError(f"stream_norm: {count} {name}, got {t.numel()}")
+    splits, stride = 0, 0
+    if delta is not None:
+        _need(delta, torch.float32, "delta")
+        if tuple(delta.shape[1:]) != (tokens, hidden):
+            raise KernelError("stream_norm: the delta does not fit the streams")
+        splits, stride = delta.shape[0], delta.stride(0)
+    if rows is not None:
+        _need(rows, torch.int32, "rows")
+    n_rows = rows.numel() if rows is not None else tokens
+    if tuple(out.shape) != (n_rows, hidden) or not out.is_contiguous():
+        raise KernelError("stream_norm: the output does not fit")
+    fn = _fn("streams", "tt_stream_norm", [c_void_p, c_int, c_longlong, c_void_p, c_int, c_longlong, c_float, c_void_p, c_void_p, c_void_p, c_void_p,
+                                           c_int, c_void_p, c_float, c_float, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p])
+    _check(fn(_ptr(streams), copies, tokens * hidden, _ptr(delta), splits, stride, scale, _ptr(gain), _ptr(mix), _ptr(write), _ptr(read),
+              1 if spread else 0, _ptr(weight), weight_offset, eps, _ptr(out), dtype_code(out.dtype), _ptr(rows), n_rows, hidden, _stream()),
+           "stream_norm")
 
 
 def add_rmsnorm(residual: torch.Tensor, delta: torch.Tensor | None, weight: torch.Tensor, eps: float, out: torch.Tensor,
@@ -445,7 +530,7 @@ def swiglu(gate_up: torch.Tensor, act: torch.Tensor, activation: str = "silu") -
               GATE_ACTIVATIONS[activation], _stream()), "swiglu")
 
 
-UNARY_ACTIVATIONS = {**GATE_ACTIVATIONS, "xielu": 3, "gelu": 4}      # gelu: the exact one, with erf
+UNARY_ACTIVATIONS = {**GATE_ACTIVATIONS, "xielu": 3, "gelu": 4, "relu2": 5}      # gelu: the exact one, with erf; relu2: the square of relu
 
 
 def activation(x: torch.Tensor, act: torch.Tensor, activation: str = "gelu_tanh", a: float = 0.0, c: float = 0.0) -> None:
@@ -906,28 +991,37 @@ def decay_scan(vkq: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, out:
 
 
 def row_decay_scan(vkq: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, out: torch.Tensor, cu: torch.Tensor, slots: torch.Tensor,
-                   sequences: int, heads: int, key_dim: int, value_dim: int, form: str = "auto") -> None:
+                   sequences: int, heads: int, key_dim: int, value_dim: int, form: str = "auto", bonus: torch.Tensor | None = None) -> None:
     """:func:`decay_scan` with decays that every token brings for every head and key channel: ``S = diag(a_t) S + k v^T``,
-    ``o = S^T q``, ``decay`` float32 ``[tokens, heads * key_dim]``."""
+    ``o = S^T q``, ``decay`` float32 ``[tokens, heads * key_dim]``.  ``bonus`` (float32 ``[heads * key_dim]``): a token reads the
+    state before it and its own contribution with this weight, ``o = (S + diag(bonus) k v^T)^T q``, and S moves on afterwards."""
+    if bonus is not None:
+        _need(bonus, torch.float32, "bonus")
+        if bonus.numel() != heads * key_dim:
+            raise KernelError("row_decay_scan: the bonus does not fit the sizes")
     for t, name in ((vkq, "v/k/q"), (decay, "decays"), (state, "recurrent state"), (out, "recurrence output")):
         _need(t, torch.float32, name)
     if (vkq.shape[1] != heads * value_dim + 2 * heads * key_dim or tuple(state.shape[1:]) != (heads, value_dim, key_dim)
             or out.shape[1] != heads * value_dim or tuple(decay.shape) != (vkq.shape[0], heads * key_dim)):
         raise KernelError("row_decay_scan: shapes do not fit the sizes")
-    fn = _fn("recurrent", "tt_row_decay_scan", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+    fn = _fn("recurrent", "tt_row_decay_scan", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                                 c_int, c_void_p])
-    _check(fn(_ptr(vkq), vkq.shape[1], _ptr(decay), _ptr(state), _ptr(out), _ptr(cu), _ptr(slots), sequences, heads, value_dim, key_dim,
-              SCAN_FORMS[form], _stream()), "row_decay_scan")
+    _check(fn(_ptr(vkq), vkq.shape[1], _ptr(decay), _ptr(bonus), _ptr(state), _ptr(out), _ptr(cu), _ptr(slots), sequences, heads, value_dim,
+              key_dim, SCAN_FORMS[form], _stream()), "row_decay_scan")
 
 
 def row_decay_blocks(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, out: torch.Tensor,
                      cu: torch.Tensor, slots: torch.Tensor, sequences: int, heads: int, qk_heads: int, key_dim: int, value_dim: int,
-                     q_scale: float, write: tuple[torch.Tensor, int] | None = None) -> None:
+                     q_scale: float, write: tuple[torch.Tensor, int] | None = None, bonus: torch.Tensor | None = None) -> None:
     """The recurrences with a decay per head and key channel, four tokens at a time (for prompts; token by token they are
     :func:`delta_scan` with ``row_decay`` and :func:`row_decay_scan`).  ``q``, ``k``, ``v``: float32 ``[tokens, columns]`` of
     ``qk_heads * key_dim`` and ``heads * value_dim`` columns, views of one matrix (equal row strides).  ``write`` = (projection
     partial sums, first column of the raw write strengths): the delta rule, which makes q and k unit vectors; without it: linear
-    attention.  q is multiplied by ``q_scale``."""
+    attention.  q is multiplied by ``q_scale``.  ``bonus`` as for :func:`row_decay_scan` (not with the delta rule)."""
+    if bonus is not None:
+        _need(bonus, torch.float32, "bonus")
+        if bonus.numel() != heads * key_dim or qk_heads != heads or write is not None:
+            raise KernelError("row_decay_blocks: a bonus has a number per head and key channel and does not go with the delta rule")
     for t, cols, name in ((q, qk_heads * key_dim, "q"), (k, qk_heads * key_dim, "k"), (v, heads * value_dim, "v")):
         if t.dtype != torch.float32 or t.dim() != 2 or t.stride(1) != 1 or t.stride(0) != q.stride(0) or t.shape[1] != cols:
             raise KernelError(f"row_decay_blocks: {name} must be float32 [tokens, {cols}] with the row stride of q")
@@ -943,17 +1037,18 @@ def row_decay_blocks(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: t
         if b_col < 0 or b_col + heads > cols:
             raise KernelError("row_decay_blocks: the write strengths lie outside the projection")
     fn = _fn("recurrent", "tt_row_decay_blocks", [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_int, c_longlong, c_int,
-                                                  c_int, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                                                  c_void_p])
+                                                  c_int, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                                                  c_int, c_void_p])
     _check(fn(_ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(decay), 0 if write is None else 1, p, splits, stride, cols, b_col, q_scale,
-              _ptr(state), _ptr(out), _ptr(cu), _ptr(slots), sequences, heads, qk_heads, key_dim, value_dim, _stream()), "row_decay_blocks")
+              _ptr(bonus), _ptr(state), _ptr(out), _ptr(cu), _ptr(slots), sequences, heads, qk_heads, key_dim, value_dim, _stream()), "row_decay_blocks")
 
 
 @dataclass(frozen=True)
 class LowRank:
     """One product of :func:`low_rank`: ``z = W x`` with x the ``rank`` columns of a projection from ``col`` on and ``weight`` the
     transposed matrix, ``[rank, n]``.  ``kind``: ``plain`` (z), ``delta_decay`` (``exp(-exp(a_log_h) * softplus(z + bias))``, h the
-    head of ``per_head`` neighbouring columns) or ``sigmoid_root`` (``sigmoid(z + bias) ** (1 / tau)``)."""
+    head of ``per_head`` neighbouring columns), ``sigmoid_root`` (``sigmoid(z + bias) ** (1 / tau)``) or ``exp_decay``
+    (``exp(-exp(z + bias))``).  ``tanh``: x passes tanh first."""
 
     col: int
     weight: torch.Tensor
@@ -963,9 +1058,10 @@ class LowRank:
     a_log: torch.Tensor | None = None
     per_head: int = 1
     tau: float = 1.0
+    tanh: bool = False
 
 
-LOW_RANK_KINDS = {"plain": 0, "delta_decay": 1, "sigmoid_root": 2}
+LOW_RANK_KINDS = {"plain": 0, "delta_decay": 1, "sigmoid_root": 2, "exp_decay": 3}
 
 
 def low_rank(proj: torch.Tensor, products: list[LowRank]) -> None:
@@ -985,35 +1081,35 @@ def low_rank(proj: torch.Tensor, products: list[LowRank]) -> None:
                 _need(t, torch.float32, name)
                 if t.numel() != count:
                     raise KernelError(f"low_rank: {name} has {t.numel()} numbers, needs {count}")
-        args += [p.col, rank, n, LOW_RANK_KINDS[p.kind], p.per_head, _ptr(p.weight), _ptr(p.bias), _ptr(p.a_log), 1.0 / p.tau, _ptr(p.out)]
-    types = [c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_float, c_void_p]
+        args += [p.col, rank, n, LOW_RANK_KINDS[p.kind], p.per_head, 1 if p.tanh else 0, _ptr(p.weight), _ptr(p.bias), _ptr(p.a_log), 1.0 / p.tau, _ptr(p.out)]
+    types = [c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_float, c_void_p]
     if len(products) == 1:
-        args += [0, 0, 0, 0, 1, c_void_p(0), c_void_p(0), c_void_p(0), 0.0, c_void_p(0)]
+        args += [0, 0, 0, 0, 1, 0, c_void_p(0), c_void_p(0), c_void_p(0), 0.0, c_void_p(0)]
     fn = _fn("recurrent", "tt_low_rank", [c_void_p, c_int, c_longlong, c_int, c_int, c_int, *types, *types, c_int, c_void_p])
     _check(fn(ptr, splits, stride, cols, len(products), dtype_code(products[0].weight.dtype), *args, tokens, _stream()), "low_rank")
 
 
-def low_rank_inputs(proj: torch.Tensor, columns: list[tuple[int, torch.Tensor]]) -> None:
+def low_rank_inputs(proj: torch.Tensor, columns: list[tuple[int, torch.Tensor, bool]]) -> None:
     """One or two ranges of a projection's columns (float32 partial sums, summed) as matrices of their own: ``columns`` lists
-    (first column, out ``[tokens, width]``)."""
+    (first column, out ``[tokens, width]``, whether they pass tanh)."""
     ptr, splits, stride, cols = _projection(proj)
-    if not 1 <= len(columns) <= 2 or len({out.dtype for _, out in columns}) != 1:
+    if not 1 <= len(columns) <= 2 or len({out.dtype for _, out, _ in columns}) != 1:
         raise KernelError("low_rank_inputs takes one or two ranges into one dtype")
     args = []
-    for col, out in columns:
+    for col, out, tanh in columns:
         if out.dim() != 2 or out.shape[0] != proj.shape[1] or not out.is_contiguous() or col < 0 or col + out.shape[1] > cols:
             raise KernelError("low_rank_inputs: shapes do not fit")
-        args += [col, out.shape[1], _ptr(out)]
+        args += [col, out.shape[1], 1 if tanh else 0, _ptr(out)]
     if len(columns) == 1:
-        args += [0, 0, c_void_p(0)]
-    fn = _fn("recurrent", "tt_low_rank_inputs", [c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_int,
-                                                 c_void_p])
+        args += [0, 0, 0, c_void_p(0)]
+    fn = _fn("recurrent", "tt_low_rank_inputs", [c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_int,
+                                                 c_int, c_void_p])
     _check(fn(ptr, splits, stride, cols, *args, dtype_code(columns[0][1].dtype), proj.shape[1], _stream()), "low_rank_inputs")
 
 
 def low_rank_finish(z: torch.Tensor, kind: str, bias: torch.Tensor, out: torch.Tensor, a_log: torch.Tensor | None = None, per_head: int = 1,
                     tau: float = 1.0) -> None:
-    """What :class:`LowRank` makes of its product (``delta_decay`` or ``sigmoid_root``), from the product's partial sums; ``out``
+    """What :class:`LowRank` makes of its product (``delta_decay``, ``sigmoid_root`` or ``exp_decay``), from the product's partial sums; ``out``
     (float32 ``[tokens, n]``) may be the first slice of ``z``."""
     ptr, splits, stride, n = _projection(z)
     for t, name in ((bias, "bias"), (a_log, "A_log"), (out, "decays")):
@@ -1080,7 +1176,7 @@ def latent_attention(q: torch.Tensor, w_key: torch.Tensor, w_value: torch.Tensor
                      inv_freq: torch.Tensor, rotary_dim: int, scale: float, window: int, splits: int, out: torch.Tensor,
                      absorbed: torch.Tensor, part_acc: torch.Tensor, part_ml: torch.Tensor, status: torch.Tensor,
                      tensor_cores: bool = False, interleaved: bool = False, rot_scale: float = 1.0,
-                     head_gate: torch.Tensor | None = None) -> None:
+                     gate: torch.Tensor | None = None) -> None:
     """Causal softmax attention over a latent cache.  ``q``: float32 partial sums ``[slices, tokens, heads * (dim + rot)]`` of
     the queries (per head ``dim`` unrotated numbers, then ``rot`` of which the first ``rotary_dim`` are rotated here);
     ``w_key`` ``[heads * dim, rank]`` and ``w_value`` ``[heads * vdim, rank]`` expand a latent into a head's keys and values;
@@ -1092,8 +1188,8 @@ def latent_attention(q: torch.Tensor, w_key: torch.Tensor, w_value: torch.Tensor
     sequence whose sizes :func:`latent_decode_tensor_cores` takes runs both products on the tensor cores, with the heads of a
     token as the rows; ``splits`` must then cover every key a token can see in slices of ``LATENT_DECODE_SLICE`` keys.
     ``q`` may be a range of a wider projection's columns.  ``interleaved`` / ``rot_scale``: as in :func:`latent_prepare`.
-    ``head_gate``: float32 partial sums ``[slices, tokens, heads]`` (possibly such a range); every head's output is multiplied
-    by the sigmoid of its number."""
+    ``gate``: float32 partial sums ``[slices, tokens, heads]`` or ``[slices, tokens, heads * vdim]`` (possibly such a range); every
+    head's output, or every output number, is multiplied by the sigmoid of its number."""
     if tensor_cores and (n_tokens != sequences or not latent_decode_tensor_cores(out.dtype, rank, rot)):
         raise KernelError("latent_attention: the tensor-core form is for steps of one token per sequence and sizes it takes")
     _need(inv_freq, torch.float32, "inverse frequencies")
@@ -1101,11 +1197,11 @@ def latent_attention(q: torch.Tensor, w_key: torch.Tensor, w_value: torch.Tensor
         raise KernelError(f"latent attention takes latents of up to {LATENT_MAX_RANK}, rows of up to {LATENT_MAX_ROW} and "
                           f"{LATENT_MAX_DIM} unrotated numbers per head; got {rank}, {rank + rot}, {dim}")
     p, q_splits, q_stride, q_row, q_cols = _projection_view(q)
-    g_ptr, g_splits, g_stride, g_row = c_void_p(0), 0, 0, 0
-    if head_gate is not None:
-        g_ptr, g_splits, g_stride, g_row, g_cols = _projection_view(head_gate)
-        if g_cols != heads or head_gate.shape[1] != n_tokens:
-            raise KernelError("latent_attention: the gate has one number per head and token")
+    g_ptr, g_splits, g_stride, g_row, g_cols = c_void_p(0), 0, 0, 0, 0
+    if gate is not None:
+        g_ptr, g_splits, g_stride, g_row, g_cols = _projection_view(gate)
+        if g_cols not in (heads, heads * vdim) or gate.shape[1] != n_tokens:
+            raise KernelError("latent_attention: the gate has one number per token and head, or per token and output number")
     if (q_cols != heads * (dim + rot) or tuple(w_key.shape) != (heads * dim, rank) or tuple(w_value.shape) != (heads * vdim, rank)
             or w_key.dtype != w_value.dtype or not w_key.is_contiguous() or not w_value.is_contiguous()
             or tuple(pool.shape[1:]) != (1, BLOCK_TOKENS, rank + rot) or pool.dtype != out.dtype
@@ -1119,11 +1215,12 @@ def latent_attention(q: torch.Tensor, w_key: torch.Tensor, w_value: torch.Tensor
     fn = _fn("latent_attention", "tt_latent_attention", [c_void_p, c_int, c_longlong, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p,
                                                          c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                                                          c_void_p, c_int, c_int, c_float, c_float, c_int, c_int, c_void_p, c_void_p, c_void_p,
-                                                         c_void_p, c_int, c_void_p, c_int, c_longlong, c_int, c_void_p, c_void_p])
+                                                         c_void_p, c_int, c_void_p, c_int, c_longlong, c_int, c_int, c_void_p, c_void_p])
     _check(fn(p, q_splits, q_stride, q_row, _ptr(w_key), _ptr(w_value), dtype_code(w_key.dtype), _ptr(pool), dtype_code(out.dtype), _ptr(table),
               table.shape[1], pool.shape[0], _ptr(cu), _ptr(len_before), sequences, n_tokens, heads, dim, rot, vdim, rank, _ptr(inv_freq),
               rotary_dim, 1 if interleaved else 0, float(rot_scale), scale, window, splits, _ptr(out), _ptr(absorbed), _ptr(part_acc),
-              _ptr(part_ml), 2 if tensor_cores else 0, g_ptr, g_splits, g_stride, g_row, _ptr(status), _stream()), "latent_attention", 3)
+              _ptr(part_ml), 2 if tensor_cores else 0, g_ptr, g_splits, g_stride, g_row, 1 if g_cols != heads else 0, _ptr(status), _stream()),
+           "latent_attention", 3)
 
 
 LATENT_DECODE_SLICE = 64        # keys of one slice of the tensor-core decode form (LT_KEYS in csrc/latent_attention.cu)
@@ -1244,7 +1341,8 @@ def sigmoid_gate(y: torch.Tensor, gate: torch.Tensor, head_width: int = 0) -> No
 ROUTE_MAX_EXPERTS = 512
 
 
-def _route_options(experts: int, score: str, correction: torch.Tensor | None, group_score: str, renormalize: bool, extra: int) -> tuple:
+def _route_options(experts: int, score: str, correction: torch.Tensor | None, group_score: str, renormalize: bool, extra: int,
+                   weight_scale: float) -> tuple:
     if score not in ("softmax", "sigmoid") or group_score not in ("max", "top2"):
         raise KernelError("routing scores are 'softmax' or 'sigmoid', group scores 'max' or 'top2'")
     if correction is not None:
@@ -1253,12 +1351,13 @@ def _route_options(experts: int, score: str, correction: torch.Tensor | None, gr
             raise KernelError(f"a correction per expert: {experts} numbers, got {correction.numel()}")
     if not 0 <= extra <= 32:
         raise KernelError("up to 32 always-on gates")
-    return (1 if score == "sigmoid" else 0, _ptr(correction), 1 if group_score == "top2" else 0, 0 if renormalize else 1, int(extra))
+    return (1 if score == "sigmoid" else 0, _ptr(correction), 1 if group_score == "top2" else 0, 0 if renormalize else 1, int(extra),
+            float(weight_scale))
 
 
 def route_topk(logits: torch.Tensor, top: int, groups: int, keep: int, gates: torch.Tensor, chosen: torch.Tensor,
                weights: torch.Tensor, score: str = "softmax", correction: torch.Tensor | None = None, group_score: str = "max",
-               renormalize: bool = True, extra: int = 0) -> None:
+               renormalize: bool = True, extra: int = 0, weight_scale: float = 1.0) -> None:
     """Routing of a mixture of experts from the router's logits (float32 partial sums ``[slices, tokens, experts]``): scores
     are the softmax over all experts; experts form ``groups`` equal groups of neighbours, a group's score is its largest
     expert score, and only experts of the ``keep`` best groups can be chosen; the ``top`` largest of those are chosen (ties:
@@ -1267,10 +1366,11 @@ def route_topk(logits: torch.Tensor, top: int, groups: int, keep: int, gates: to
     ``score`` "sigmoid": scores are the logits' sigmoids.  ``correction`` (float32, one per expert) is added to the scores for
     the choice only (groups and experts); weights stay the scores.  ``group_score`` "top2": a group's score is the sum of its
     two largest choice scores.  ``renormalize`` off: the weights are the chosen scores themselves.  ``extra``: so many more
-    logits follow the experts'; ``gates`` then has ``experts + extra`` columns, the last ones the sigmoids of those logits."""
+    logits follow the experts'; ``gates`` then has ``experts + extra`` columns, the last ones the sigmoids of those logits.
+    ``weight_scale``: a factor on the chosen experts' weights."""
     p, splits, stride, experts = _projection(logits)
     experts -= extra
-    options = _route_options(experts, score, correction, group_score, renormalize, extra)
+    options = _route_options(experts, score, correction, group_score, renormalize, extra, weight_scale)
     tokens = logits.shape[1]
     _need(gates, torch.float32, "gates")
     _need(weights, torch.float32, "routing weights")
@@ -1282,19 +1382,19 @@ def route_topk(logits: torch.Tensor, top: int, groups: int, keep: int, gates: to
     if tuple(gates.shape) != (tokens, experts + extra) or tuple(chosen.shape) != (tokens, top) or tuple(weights.shape) != (tokens, top):
         raise KernelError("route_topk: outputs do not fit the sizes")
     fn = _fn("routing", "tt_route_topk", [c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
-                                          c_int, c_void_p, c_int, c_int, c_int, c_void_p])
+                                          c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p])
     _check(fn(p, splits, stride, tokens, experts, top, groups, keep, _ptr(gates), _ptr(chosen), _ptr(weights), *options, _stream()),
            "route_topk")
 
 
 def route_rows(x: torch.Tensor, w: torch.Tensor, top: int, groups: int, keep: int, gates: torch.Tensor, chosen: torch.Tensor,
                weights: torch.Tensor, score: str = "softmax", correction: torch.Tensor | None = None, group_score: str = "max",
-               renormalize: bool = True, extra: int = 0) -> None:
+               renormalize: bool = True, extra: int = 0, weight_scale: float = 1.0) -> None:
     """:func:`route_topk` with the router's product ``x @ w.T`` (float32 sums) in front, in one kernel: ``x`` ``[tokens,
     hidden]`` and ``w`` ``[experts + extra, hidden]``, each float32 or bfloat16."""
     tokens, hidden = x.shape
     experts = w.shape[0] - extra
-    options = _route_options(experts, score, correction, group_score, renormalize, extra)
+    options = _route_options(experts, score, correction, group_score, renormalize, extra, weight_scale)
     _need(gates, torch.float32, "gates")
     _need(weights, torch.float32, "routing weights")
     _need(chosen, torch.int32, "chosen experts")
@@ -1309,7 +1409,7 @@ def route_rows(x: torch.Tensor, w: torch.Tensor, top: int, groups: int, keep: in
     if tuple(gates.shape) != (tokens, experts + extra) or tuple(chosen.shape) != (tokens, top) or tuple(weights.shape) != (tokens, top):
         raise KernelError("route_rows: outputs do not fit the sizes")
     fn = _fn("routing", "tt_route_rows", [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
-                                          c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p])
+                                          c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p])
     _check(fn(_ptr(x), dtype_code(x.dtype), _ptr(w), dtype_code(w.dtype), hidden, tokens, experts, top, groups, keep, _ptr(gates),
               _ptr(chosen), _ptr(weights), *options, _stream()), "route_rows")
 
@@ -1339,31 +1439,55 @@ def scale_expert_columns(act: torch.Tensor, width: int, gates: torch.Tensor, exp
 
 
 def expert_activation(gate_up: torch.Tensor, act: torch.Tensor, experts: int, width: int, shared_width: int, limit: float,
-                      shared_limit: float, alpha: float, gates: torch.Tensor, shared_gated: bool) -> None:
+                      shared_limit: float, alpha: float, gates: torch.Tensor | None, shared_gated: bool) -> None:
     """The clamped gated unit of a mixture's experts with the routing weights applied: ``gate_up`` float32 partial sums
     ``[slices, tokens, 2 * cols]`` (gate columns first), ``cols = experts * width + shared_width``.  With ``g' = min(g, limit)``
     and ``u' = clamp(u, -limit, limit)``: ``act[t, c] = g' sigmoid(alpha g') (u' + 1) * gates[t, c // width]`` for the routed
     experts' columns; the always-on expert's columns behind them use ``shared_limit`` and ``gates[t, experts]`` (``shared_gated``)
-    or no weight.  A limit of 0 or less: no clamp."""
+    or no weight.  A limit of 0 or less: no clamp.  Without routed experts (a dense feed-forward: ``shared_width`` columns) ``gates`` may be None."""
     p, splits, stride, cols2 = _projection(gate_up)
-    _need(gates, torch.float32, "gates")
     tokens = gate_up.shape[1]
+    if gates is None:
+        if experts or shared_gated:
+            raise KernelError("expert_activation: routed experts and a gated expert need the gates")
+    else:
+        _need(gates, torch.float32, "gates")
+        if gates.shape[0] != tokens:
+            raise KernelError("expert_activation: the gates do not fit the tokens")
     cols = experts * width + shared_width
-    if cols2 != 2 * cols or tuple(act.shape) != (tokens, cols) or not act.is_contiguous() or gates.shape[0] != tokens:
+    if cols2 != 2 * cols or tuple(act.shape) != (tokens, cols) or not act.is_contiguous():
         raise KernelError("expert_activation: shapes do not fit the sizes")
-    if gates.shape[1] < experts + (1 if shared_gated else 0):
+    if gates is not None and gates.shape[1] < experts + (1 if shared_gated else 0):
         raise KernelError("expert_activation: too few gates a token")
     fn = _fn("routing", "tt_expert_activation", [c_void_p, c_int, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
                                                  c_float, c_void_p, c_int, c_int, c_void_p])
     _check(fn(p, splits, stride, _ptr(act), dtype_code(act.dtype), tokens, experts, width, shared_width, float(limit or 0.0),
-              float(shared_limit or 0.0), float(alpha), _ptr(gates), gates.shape[1], 1 if shared_gated else 0, _stream()), "expert_activation")
+              float(shared_limit or 0.0), float(alpha), _ptr(gates), 0 if gates is None else gates.shape[1], 1 if shared_gated else 0, _stream()),
+           "expert_activation")
+
+
+def expert_unary_activation(up: torch.Tensor, act: torch.Tensor, width: int, activation: str, gates: torch.Tensor) -> None:
+    """Experts without a gate projection, with the routing weights applied: ``act[t, c] = f(sum of the float32 slices up[s, t, c]) *
+    gates[t, c // width]`` for the experts' ``width`` columns each, side by side; f is an ungated activation without parameters.
+    Columns of experts with a zero gate are zero."""
+    p, splits, stride, cols = _projection(up)
+    _need(gates, torch.float32, "gates")
+    tokens, experts = up.shape[1], cols // width
+    if cols != experts * width or tuple(act.shape) != (tokens, cols) or not act.is_contiguous() or gates.shape[0] != tokens or gates.shape[1] < experts:
+        raise KernelError("expert_unary_activation: shapes do not fit the sizes")
+    if activation not in UNARY_ACTIVATIONS or activation == "xielu":
+        raise KernelError(f"expert_unary_activation: {activation!r} is not an activation without parameters")
+    fn = _fn("routing", "tt_expert_unary_activation", [c_void_p, c_int, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
+                                                       c_void_p])
+    _check(fn(p, splits, stride, _ptr(act), dtype_code(act.dtype), tokens, experts, width, UNARY_ACTIVATIONS[activation], _ptr(gates),
+              gates.shape[1], _stream()), "expert_unary_activation")
 
 
 # -------------------------------------------------------------------------------- gemm
 def gemm_simt(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None, out: torch.Tensor) -> None:
     """out[s] = x @ w[:, k-slice s].T in float32 FMA; ``out`` is float32
-    [splits, m, n]; bias (float32 [n]) goes into slice 0."""
-    _need(out, torch.float32, "gemm output")
+    [splits, m, n] (possibly a range of a wider matrix's columns); bias (float32 [n]) goes into slice 0."""
+    _need_columns(out, torch.float32, "gemm output")
     if x.stride(-1) != 1 or w.stride(-1) != 1:
         raise KernelError("gemm operands must be contiguous along k")
     m, k = x.shape
@@ -1508,12 +1632,12 @@ def gemm_tcgen05_shares_words() -> int:
 def gemm_tcgen05(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None, out: torch.Tensor, status: torch.Tensor,
                  operands_checked: bool = False, accumulate: bool = False, shares: torch.Tensor | None = None) -> None:
     """out[s] = x @ w[:, k-slice s].T on the tensor cores; bfloat16 operands, float32
-    ``out`` [splits, tokens, features]; bias (float32) goes into slice 0.  ``operands_checked``: the
+    ``out`` [splits, tokens, features] (possibly a range of a wider matrix's columns); bias (float32) goes into slice 0.  ``operands_checked``: the
     caller has already called :func:`gemm_tcgen05_usable` on these operands.  ``accumulate``: the
     product is added to ``out`` [1, tokens, features] (only where :func:`gemm_tcgen05_accumulates`).
     ``shares``: zeroed int32 scratch memory of :func:`gemm_tcgen05_shares_words` words; with it, prompts on
     CTA pairs whose tiles would leave pairs idle share the tiles' k among the pairs."""
-    _need(out, torch.float32, "gemm output")
+    _need_columns(out, torch.float32, "gemm output")
     tokens, k = x.shape
     features = w.shape[0]
     if accumulate and (out.shape[0] != 1 or not gemm_tcgen05_accumulates(tokens, features, k)):
@@ -1531,6 +1655,32 @@ def gemm_tcgen05(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None, ou
     _check(fn(_ptr(x), x.stride(0), _ptr(w), w.stride(0), _ptr(bias), _ptr(out), out.stride(1), out.stride(0), tokens, features, k,
               out.shape[0], 2 if accumulate else 0, _ptr(status), _stream(), _ptr(shares), 0 if shares is None else shares.numel() * 4),
            "gemm_tcgen05")
+
+
+def gemm_tcgen05_groups_takes(x: torch.Tensor, w: torch.Tensor, group_features: int) -> bool:
+    """Whether one product can give every ``group_features`` output features activations of their own: ``x`` ``[groups, tokens, k]``,
+    no tile across two groups."""
+    groups, tokens, _ = x.shape
+    return (x.is_contiguous() and gemm_tcgen05_usable(x[0], w) and group_features % (256 if tokens > SKINNY_TOKENS else 128) == 0
+            and -(-w.shape[0] // group_features) == groups)
+
+
+def gemm_tcgen05_groups(x: torch.Tensor, w: torch.Tensor, group_features: int, out: torch.Tensor, status: torch.Tensor,
+                        shares: torch.Tensor | None = None) -> None:
+    """:func:`gemm_tcgen05` with activations of their own for every ``group_features`` output features (the last group may be
+    smaller): ``x`` ``[groups, tokens, k]``, ``out[s, t, f] = x[f // group_features, t] . w[f]`` over k-slice s.  Only where
+    :func:`gemm_tcgen05_groups_takes`."""
+    _need(out, torch.float32, "gemm output")
+    groups, tokens, k = x.shape
+    features = w.shape[0]
+    if not gemm_tcgen05_groups_takes(x, w, group_features) or w.shape[1] != k or tuple(out.shape[1:]) != (tokens, features):
+        raise KernelError(f"grouped tcgen05 gemm cannot take x {tuple(x.shape)} / w {tuple(w.shape)} / out {tuple(out.shape)} in groups of {group_features}")
+    if out.shape[0] > -(-k // 64):
+        raise KernelError(f"{out.shape[0]} k-slices for k = {k}: a slice needs at least one block of 64")
+    fn = _fn("gemm_tcgen05", "tt_gemm_tcgen05_groups", [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_longlong, c_int, c_int,
+                                                        c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_longlong])
+    _check(fn(_ptr(x), x.stride(1), _ptr(w), w.stride(0), _ptr(out), out.stride(1), out.stride(0), tokens, features, k, out.shape[0],
+              group_features, _ptr(status), _stream(), _ptr(shares), 0 if shares is None else shares.numel() * 4), "gemm_tcgen05_groups")
 
 
 def gemm_tcgen05_qkv_rope_takes(x: torch.Tensor, w: torch.Tensor, head_dim: int, rotary_dim: int) -> bool:

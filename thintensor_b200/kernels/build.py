@@ -40,6 +40,7 @@ SOURCES: dict[str, list[str]] = {
     "recurrent": [],
     "latent_attention": [],
     "routing": [],
+    "streams": [],
 }
 
 

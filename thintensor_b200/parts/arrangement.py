@@ -16,25 +16,38 @@ norm, or the final norm).
 """
 from __future__ import annotations
 
+from dataclasses import replace
+
 import torch
 
 from ..kernels import api
-from .base import ARRANGEMENTS, Arrangement, Delta, DepthStep
+from .base import ARRANGEMENTS, Arrangement, Delta, DepthStep, StreamStep
 
 
 @ARRANGEMENTS.register("pre_norm")
 class PreNorm(Arrangement):
     """A layer without a feed-forward leaves out ``ffn_norm`` and ``ffn``: its mixer's output is then what the next
     layer's norm adds.  ``side`` (optional): a side input at the layer's end, which reads the stream with the last
-    sublayer's output added and hands on what it adds itself."""
+    sublayer's output added and hands on what it adds itself.  ``scale`` (a constant) and ``mixer_scale`` / ``ffn_scale`` (factors
+    per channel) multiply a sublayer's output before the stream takes it.  ``mixer_streams`` / ``ffn_streams``: the stream comes in
+    several copies (the model's ``streams``), which each sublayer reads and writes with weights of its own."""
 
-    roles = {"mixer_norm": "norm", "mixer": "mixer", "ffn_norm": "norm", "ffn": "ffn", "side": "side"}
-    optional = ("ffn_norm", "ffn", "side")
+    roles = {"mixer_norm": "norm", "mixer": "mixer", "mixer_scale": "scale", "mixer_streams": "streams", "ffn_norm": "norm", "ffn": "ffn",
+             "ffn_scale": "scale", "ffn_streams": "streams", "side": "side"}
+    optional = ("mixer_scale", "mixer_streams", "ffn_norm", "ffn", "ffn_scale", "ffn_streams", "side")
 
-    def __init__(self, parts):
+    def __init__(self, parts, scale: float = 1.0):
         super().__init__(parts)
         if ("ffn" in parts) != ("ffn_norm" in parts):
             raise ValueError("a pre-norm layer has a feed-forward and its norm, or neither")
+        if "ffn" not in parts and ("ffn_scale" in parts or "ffn_streams" in parts):
+            raise ValueError("a scale or stream weights of a feed-forward go with one")
+        if "ffn" in parts and ("mixer_streams" in parts) != ("ffn_streams" in parts):
+            raise ValueError("both sublayers read and write the streams with weights of their own, or neither does")
+        self.scale = float(scale)
+        self.plain = self.scale == 1.0 and not {"mixer_scale", "mixer_streams", "ffn_scale", "ffn_streams"} & set(parts)
+        if "side" in parts and not self.plain:
+            raise ValueError("a side input goes with a single stream and unscaled sublayers")
 
     def mixers(self):
         return [self.parts["mixer"]]
@@ -45,17 +58,33 @@ class PreNorm(Arrangement):
     def run(self, ctx, residual, pending: Delta | None, caches, states) -> Delta:
         hidden = residual.shape[-1]
         # Between a part's output and the norm that follows nothing else reads the stream, so a part
-        # may add its output into it directly instead of handing it on.
-        ctx.residual = residual
+        # may add its output into it directly instead of handing it on (not one that is scaled or mixed on its way).
+        ctx.residual = residual if self.plain else None
         normed = ctx.scratch("block.normed", (ctx.n_tokens, hidden))
-        self.parts["mixer_norm"].forward(ctx, residual, pending, normed)
-        last = self.parts["mixer"].forward(ctx, normed, caches[0], states[0])
+        self.parts["mixer_norm"].forward(ctx, residual, self.reading("mixer", pending), normed)
+        last = self.written("mixer", self.parts["mixer"].forward(ctx, normed, caches[0], states[0]))
         if "ffn" in self.parts:
-            self.parts["ffn_norm"].forward(ctx, residual, last, normed)
-            last = self.parts["ffn"].forward(ctx, normed)
+            self.parts["ffn_norm"].forward(ctx, residual, self.reading("ffn", last), normed)
+            last = self.written("ffn", self.parts["ffn"].forward(ctx, normed))
         if "side" in self.parts:
             last = self.parts["side"].forward(ctx, residual, last)
         return last
+
+    def reading(self, sublayer: str, pending: Delta | None) -> Delta | None:
+        """The pending delta with the weights with which this sublayer's norm reads the streams."""
+        streams = self.parts.get(sublayer + "_streams")
+        if streams is None:
+            return pending
+        pending = pending or Delta(None)
+        return replace(pending, streams=replace(pending.streams or StreamStep(), read=streams.read))
+
+    def written(self, sublayer: str, delta: Delta) -> Delta:
+        """The sublayer's output with its factors and the weights with which the streams take it."""
+        if self.plain:
+            return delta
+        scale, streams = self.parts.get(sublayer + "_scale"), self.parts.get(sublayer + "_streams")
+        return Delta(delta.tensor, scale=self.scale, gain=None if scale is None else scale.weight,
+                     streams=None if streams is None else StreamStep(streams.mix, streams.write))
 
 
 @ARRANGEMENTS.register("pre_norm_pair")

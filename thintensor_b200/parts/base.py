@@ -26,6 +26,8 @@ Roles and what each must provide:
   step's tokens (a gated slice of a second token embedding, say).
 * ``DepthMix``: the weights with which a layer's end mixes the results of the layers so far (``weights()`` only; the
   arrangement hands them to the norm that follows).
+* ``StreamMix``: the weights with which a sublayer reads and writes a residual stream that comes in several copies, and
+  ``Scale``: a factor per channel on a sublayer's output (both ``weights()`` only, for the norm kernels as well).
 * ``Arrangement``: wires norms, mixer and feed-forward around the residual stream.
 """
 from __future__ import annotations
@@ -40,7 +42,7 @@ import torch
 class WeightDecl:
     """A tensor a part needs.  ``init`` tells the random-weights mode how to draw it:
     ``normal`` is N(0, 0.02), ``norm`` is 1 + N(0, 0.1), ``small`` is N(0, 0.1), ``depth`` is N(0, 0.3) with one added to the last number,
-    ``zeros`` is zero.  ``free`` lists axes whose extent the checkpoint decides (the rank of a product of low rank, say); ``shape``
+    ``identity`` is N(0, 0.1) with one added on the diagonal of a square matrix, ``zeros`` is zero.  ``free`` lists axes whose extent the checkpoint decides (the rank of a product of low rank, say); ``shape``
     then holds what random weights are drawn with, and the part reads the real extent off the tensor it is bound to.
     ``alias_of`` names a checkpoint tensor (full name) to use instead when this one is
     absent from the checkpoint; with ``prefer_alias`` it is used even when this one is
@@ -105,6 +107,19 @@ class DepthStep:
     weights: torch.Tensor | None    # float32 [index + 1]
 
 
+@dataclass(frozen=True)
+class StreamStep:
+    """A residual stream in several copies ``x_s`` (float32 ``[streams, tokens, hidden]``).  With y the sublayer's output (after its
+    scales), copy t becomes ``sum(mix[s, t] * x_s) + write[t] * y`` and what the norm takes is ``sum(read[t] * x_t)`` of the new
+    copies.  ``mix`` None: the copies stay; ``write`` / ``read`` None: ones.  ``spread``: only the first copy is there so far (the
+    embedding's output), and the others start equal to it."""
+
+    mix: torch.Tensor | None = None     # float32 [streams, streams], from (row) and to (column)
+    write: torch.Tensor | None = None   # float32 [streams]
+    read: torch.Tensor | None = None    # float32 [streams]
+    spread: bool = False
+
+
 @dataclass
 class Delta:
     """What a mixer or feed-forward adds to the residual stream: float32
@@ -116,6 +131,9 @@ class Delta:
     addition the stream is kept as a layer's result and replaced by a weighted sum of the results so far.
     Both are carried out by the norm that follows, in its one pass over the row.
 
+    ``gain`` (float32 ``[hidden]``) multiplies the sum channel by channel.  ``streams``: the stream comes in several copies, into
+    which the sum goes and from which the norm that follows reads as the step says.
+
     ``second``: another sublayer's partial sums, added to the first's.  ``scale`` multiplies both.  ``addend`` (float32
     ``[tokens, hidden]``) is added as it is.  The norm that follows does these too."""
 
@@ -125,11 +143,18 @@ class Delta:
     second: torch.Tensor | None = None
     scale: float = 1.0
     addend: torch.Tensor | None = None
+    gain: torch.Tensor | None = None
+    streams: "StreamStep | None" = None
 
     @property
     def plain(self) -> bool:
         """Whether the delta is nothing but the sum of ``tensor``."""
-        return self.post is None and self.depth is None and not self.branched
+        return self.post is None and self.depth is None and not self.branched and not self.streamed
+
+    @property
+    def streamed(self) -> bool:
+        """Whether the delta goes through the kernel for scaled outputs and several streams."""
+        return self.gain is not None or self.streams is not None
 
     @property
     def branched(self) -> bool:
@@ -326,6 +351,8 @@ POSITION_ENCODINGS = Registry("position encoding")
 MIXERS = Registry("mixer")
 FEED_FORWARDS = Registry("feed-forward")
 DEPTH_MIXES = Registry("depth mix")
+STREAM_MIXES = Registry("stream mix")
+SCALES = Registry("scale")
 EMBEDDINGS = Registry("embedding")
 SHIFTS = Registry("input shift")
 SIDES = Registry("side input")
@@ -338,6 +365,8 @@ REGISTRIES = {
     "mixer": MIXERS,
     "ffn": FEED_FORWARDS,
     "depth": DEPTH_MIXES,
+    "streams": STREAM_MIXES,
+    "scale": SCALES,
     "embedding": EMBEDDINGS,
     "shift": SHIFTS,
     "side": SIDES,

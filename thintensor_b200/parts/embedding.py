@@ -3,7 +3,7 @@
 ``h0 = E[token] * scale`` with scale 1 for Llama (thinruntime/gpu_runtime.py:10072,
 thinruntime/model_arch.py:234-238).  The head is ``lm_head.weight`` when the checkpoint
 has one and the embedding table otherwise (thinruntime/gpu_runtime.py:10395-10401);
-logits are float32.  Two more embeddings add a second row to the token's: one chosen by the pair of the
+logits are float32.  The row may pass an RMS norm first.  Two more embeddings add a second row to the token's: one chosen by the pair of the
 previous token and this one, one by the token's position.
 """
 from __future__ import annotations
@@ -17,22 +17,32 @@ from .linear import Linear
 
 @EMBEDDINGS.register("table")
 class TokenEmbedding(Embedding):
-    def __init__(self, vocab: int, hidden: int, scale: float = 1.0, name: str = "weight"):
+    """``norm_eps``: the row (times ``scale``) is divided by its root mean square and multiplied by a weight (``norm_name``)."""
+
+    def __init__(self, vocab: int, hidden: int, scale: float = 1.0, name: str = "weight", norm_eps: float | None = None,
+                 norm_name: str = "norm.weight"):
         self.vocab, self.hidden, self.scale = int(vocab), int(hidden), float(scale)
         self.name = name                        # what the checkpoint calls the table, behind the part's prefix
+        self.norm_eps, self.norm_name = None if norm_eps is None else float(norm_eps), norm_name
         self.table: torch.Tensor | None = None
+        self.norm: torch.Tensor | None = None
 
     def weights(self) -> dict[str, WeightDecl]:
-        return {self.name: WeightDecl((self.vocab, self.hidden))}
+        norm = {} if self.norm_eps is None else {self.norm_name: WeightDecl((self.hidden,), init="norm")}
+        return {self.name: WeightDecl((self.vocab, self.hidden)), **norm}
 
     def bind(self, tensors, dtype, device) -> None:
         self.table = tensors[self.name].contiguous()
+        self.norm = None if self.norm_eps is None else tensors[self.norm_name].to(torch.float32).contiguous()
 
     def device_driven(self) -> bool:
         return True
 
     def forward(self, ctx, tokens, residual, states=None) -> None:
-        api.embed_gather(self.table, tokens, residual, self.scale, ctx.status)
+        if self.norm is not None:
+            api.embed_norm_gather(self.table, tokens, self.norm, self.norm_eps, residual, self.scale, ctx.status)
+        else:
+            api.embed_gather(self.table, tokens, residual, self.scale, ctx.status)
 
 
 @EMBEDDINGS.register("table_positions")

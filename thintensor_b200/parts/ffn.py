@@ -1,9 +1,10 @@
 """Dense feed-forwards.  Gated: ``down(f(gate(x)) * up(x))``, f = ``silu(g) = g / (1 + exp(-g))`` by default
 (thinruntime/gpu_runtime.py:10286-10366; the activation at :10351 and
-thinruntime/triton_kernels.py:2760-2774), or ``relu`` or ``gelu_tanh`` (``activation``).  ``names`` gives the
+thinruntime/triton_kernels.py:2760-2774), or ``relu`` or ``gelu_tanh`` (``activation``).  With ``activation="clamped"`` the unit is
+``g' sigmoid(alpha g') (u' + 1)`` with ``g' = min(gate(x), limit)`` and ``u' = clamp(up(x), -limit, limit)``.  ``names`` gives the
 checkpoint's names of the gate, up and down matrices behind the part's prefix.
 
-Ungated (``mlp``): ``down(f(up(x)))`` with f one of the gate activations or ``xielu``, which has two learned numbers
+Ungated (``mlp``): ``down(f(up(x)))`` with f one of the gate activations, ``relu2`` (the square of relu) or ``xielu``, which has two learned numbers
 (p, q) per layer: ``softplus(p) z^2 + z / 2`` for z > 0 and ``(1 / 2 + softplus(q)) (exp(z) - 1 - z) + z / 2`` otherwise."""
 from __future__ import annotations
 
@@ -18,11 +19,12 @@ from .linear import GatedLinear, Linear
 class SwiGLU(FeedForward):
     NAMES = {"gate": "gate_proj.weight", "up": "up_proj.weight", "down": "down_proj.weight"}
 
-    def __init__(self, hidden: int, inter: int, bias: bool = False, activation: str = "silu", names: dict | None = None):
+    def __init__(self, hidden: int, inter: int, bias: bool = False, activation: str = "silu", names: dict | None = None,
+                 limit: float = 0.0, alpha: float = 1.702):
         self.hidden, self.inter, self.bias = int(hidden), int(inter), bool(bias)
-        if activation not in api.GATE_ACTIVATIONS:
-            raise ValueError(f"gate activation {activation!r} is not one of {sorted(api.GATE_ACTIVATIONS)}")
-        self.activation = activation
+        if activation != "clamped" and activation not in api.GATE_ACTIVATIONS:
+            raise ValueError(f"gate activation {activation!r} is not 'clamped' or one of {sorted(api.GATE_ACTIVATIONS)}")
+        self.activation, self.limit, self.alpha = activation, float(limit), float(alpha)
         self.names = {**self.NAMES, **(names or {})}
         self.gate_up: GatedLinear | None = None
         self.down: Linear | None = None
@@ -42,7 +44,8 @@ class SwiGLU(FeedForward):
     def bind(self, tensors, dtype, device) -> None:
         n = self.names
         self.gate_up = GatedLinear(tensors[n["gate"]], tensors[n["up"]],
-                                   tensors.get("gate_proj.bias"), tensors.get("up_proj.bias"), self.activation)
+                                   tensors.get("gate_proj.bias"), tensors.get("up_proj.bias"), self.activation,
+                                   self.limit, self.alpha)
         self.down = Linear(tensors[n["down"]], tensors.get("down_proj.bias"))
 
     def projections(self) -> list:

@@ -9,7 +9,8 @@ concatenated heads.
 
 Options: no low-rank query path at all (``q_rank`` None: ``q = W_q x``, tensor ``q``); a rotation that pairs neighbouring
 numbers and multiplies cosines and sines by a constant (the position encoding's ``interleaved`` and
-``attention_scaling``); every head's output multiplied by ``sigmoid(W_g x)_h``, one number per head (``gate="head"``).  Where
+``attention_scaling``); every head's output multiplied by ``sigmoid(W_g x)_h``, one number per head (``gate="head"``) or one per
+output number (``gate="elementwise"``, W_g with ``heads * value_dim`` rows).  Where
 the queries are projected directly, ONE product makes ``[kv latent | shared key part | queries | gate]``.
 
 Only ``[c | k_rot]`` is cached: one row per token, one key/value head, no value pool.  Decoding (and every step
@@ -44,9 +45,10 @@ class LatentAttention(Mixer):
                  gate: str | None = None):
         self.hidden, self.heads, self.dim, self.rot_dim = int(hidden), int(heads), int(dim), int(rot_dim)
         self.value_dim, self.q_rank, self.kv_rank = int(value_dim), int(q_rank or 0), int(kv_rank)
-        if gate not in (None, "head"):
-            raise ValueError(f"latent attention gates its heads ('head') or nothing, not {gate!r}")
+        if gate not in (None, "head", "elementwise"):
+            raise ValueError(f"latent attention gates its heads ('head'), its output numbers ('elementwise') or nothing, not {gate!r}")
         self.gate = gate
+        self.gate_rows = {None: 0, "head": self.heads, "elementwise": self.heads * self.value_dim}[gate]
         self.scale, self.eps = float(scale), float(eps)
         self.window = None if not window else int(window)
         if self.kv_rank > api.LATENT_MAX_RANK or self.kv_rank + self.rot_dim > api.LATENT_MAX_ROW or self.dim > api.LATENT_MAX_DIM:
@@ -69,7 +71,7 @@ class LatentAttention(Mixer):
                        n["uq"]: WeightDecl((self.heads * (self.dim + self.rot_dim), self.q_rank))}
         else:
             queries = {n["q"]: WeightDecl((self.heads * (self.dim + self.rot_dim), self.hidden))}
-        gate = {n["g"]: WeightDecl((self.heads, self.hidden))} if self.gate else {}
+        gate = {n["g"]: WeightDecl((self.gate_rows, self.hidden))} if self.gate else {}
         return {
             **queries,
             n["dkv"]: WeightDecl((self.kv_rank + self.rot_dim, self.hidden)),
@@ -105,7 +107,7 @@ class LatentAttention(Mixer):
             rows = [tensors[n["dkv"]], tensors[n["q"]]]                     # [kv latent | shared key part | queries]
             self.up_q, self.q_norm = None, None
         if self.gate:
-            rows.append(tensors[n["g"]])                                    # one gate number per head behind everything else
+            rows.append(tensors[n["g"]])                                    # the gate numbers behind everything else
         self.down = Linear(torch.cat(rows, dim=0))
         self.out = Linear(tensors[n["o"]])
         self.kv_norm = tensors[n["dkv_norm"]].to(torch.float32).contiguous()
@@ -128,7 +130,7 @@ class LatentAttention(Mixer):
         rot = self.rot
         down = self.down(ctx, x, "latent.down")
         front = self.q_rank + self.kv_rank + self.rot_dim
-        head_gate = down[:, :, down.shape[2] - self.heads:] if self.gate else None
+        gate = down[:, :, down.shape[2] - self.gate_rows:] if self.gate else None
         q_latent = ctx.scratch("latent.q_latent", (ctx.n_tokens, self.q_rank)) if self.q_rank else None
         api.latent_prepare(down[:, :, :front], self.q_rank, self.kv_rank, self.rot_dim, self.q_norm, self.kv_norm, self.eps, rot.inv_freq,
                            rot.rotary_dim, q_latent, cache.k_pool if cache.writes else None, table, ctx.cu, ctx.len_before,
@@ -140,8 +142,8 @@ class LatentAttention(Mixer):
         mixed = ctx.scratch("latent.mixed", (ctx.n_tokens, self.heads * self.value_dim))
         if self.expands(ctx, x):
             self.attend_expanded(ctx, q, cache, table, mixed)
-            if head_gate is not None:
-                api.sigmoid_gate(mixed, head_gate, self.value_dim)
+            if gate is not None:
+                api.sigmoid_gate(mixed, gate, self.value_dim if self.gate == "head" else 0)
             return self.out.delta(ctx, mixed, "latent.out")
         splits, tensor_cores = 1, False
         reach = ctx.max_total if self.window is None else min(self.window, ctx.max_total)
@@ -158,7 +160,7 @@ class LatentAttention(Mixer):
         api.latent_attention(q, self.w_key, self.w_value, cache.k_pool, table, ctx.cu, ctx.len_before, ctx.sequences, ctx.n_tokens,
                              self.heads, self.dim, self.rot_dim, self.value_dim, self.kv_rank, rot.inv_freq, rot.rotary_dim, self.scale,
                              self.window or 0, splits, mixed, absorbed, part_acc, part_ml, ctx.status, tensor_cores,
-                             interleaved=rot.interleaved, rot_scale=rot.attention_scaling, head_gate=head_gate)
+                             interleaved=rot.interleaved, rot_scale=rot.attention_scaling, gate=gate)
         return self.out.delta(ctx, mixed, "latent.out")
 
     # ------------------------------------------------------------ prompts on the tensor cores

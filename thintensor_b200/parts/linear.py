@@ -77,12 +77,48 @@ class Linear:
         return Delta(self(ctx, x, name))
 
 
+class GroupedLinear:
+    """Matrices ``W_i`` ``[n_i, in]`` that each multiply rows of their own: ``x`` ``[groups, tokens, in]`` -> float32 partial sums
+    ``[slices, tokens, sum(n_i)]`` with ``x_i @ W_i.T`` side by side.  All ``n_i`` but the last are equal.
+    One tensor-core product does it where its tiles fit the groups; otherwise one product per group writes its columns."""
+
+    def __init__(self, weights: list[torch.Tensor]):
+        self.rows = weights[0].shape[0]
+        if any(w.shape[0] != self.rows for w in weights[:-1]):
+            raise ValueError("grouped projections but the last have equally many rows")
+        self.fused = Linear(torch.cat(weights, dim=0))
+        self.groups = len(weights)
+
+    def __call__(self, ctx, x: torch.Tensor, name: str) -> torch.Tensor:
+        tokens, k = x.shape[1:]
+        total, w = self.fused.out_features, self.fused.weight
+        if api.gemm_tcgen05_groups_takes(x, w, self.rows):
+            out = ctx.scratch(name, (api.gemm_tcgen05_splits(tokens, total, k), tokens, total), torch.float32)
+            api.set_label(name)
+            api.gemm_tcgen05_groups(x, w, self.rows, out, ctx.status, Linear.shares(ctx, tokens))
+            return out
+        tensor_cores = api.gemm_tcgen05_usable(x[0], w)
+        # every group's product fills the same slices (an empty one with zeros, which the kernel for few tokens does)
+        splits = api.gemm_tcgen05_splits(tokens, self.rows, k) if tensor_cores and tokens <= api.SKINNY_TOKENS else 1
+        out = ctx.scratch(name, (splits, tokens, total), torch.float32)
+        for i in range(self.groups):
+            columns = slice(i * self.rows, (i + 1) * self.rows if i + 1 < self.groups else total)
+            api.set_label(name)
+            if tensor_cores:
+                api.gemm_tcgen05(x[i], w[columns], None, out[:, :, columns], ctx.status, operands_checked=True)
+            else:
+                api.gemm_simt(x[i], w[columns], None, out[:, :, columns])
+        return out
+
+
 class GatedLinear:
     """gate and up projections as one ``[2 * inter, in]`` matrix (gate rows first) and
-    ``f(gate) * up`` in the activation dtype (f: silu, relu or gelu_tanh)."""
+    ``f(gate) * up`` in the activation dtype (f: silu, relu or gelu_tanh), or the clamped unit ``g' sigmoid(alpha g') (u' + 1)``
+    with ``g' = min(gate, limit)`` and ``u' = clamp(up, -limit, limit)`` (``activation="clamped"``)."""
 
     def __init__(self, gate: torch.Tensor, up: torch.Tensor, gate_bias: torch.Tensor | None, up_bias: torch.Tensor | None,
-                 activation: str = "silu"):
+                 activation: str = "silu", limit: float = 0.0, alpha: float = 1.702):
+        self.limit, self.alpha = float(limit), float(alpha)
         self.inter = gate.shape[0]
         self.activation = activation
         bias = None
@@ -101,7 +137,13 @@ class GatedLinear:
             # into slices, so it is taken only where the plain product would not slice either
             # (measured on a B200: 3 % faster for 14336 x 4096 at 8 tokens, 2 % slower for 8192 x 2048).
             api.set_label(name)
-            api.gemm_tcgen05_swiglu(x, w.weight, act, ctx.status, self.activation)
+            if self.activation == "clamped":
+                api.gemm_tcgen05_clamped(x, w.weight, act, ctx.status, self.limit, self.limit, self.inter, self.alpha)
+            else:
+                api.gemm_tcgen05_swiglu(x, w.weight, act, ctx.status, self.activation)
+            return act
+        if self.activation == "clamped":
+            api.expert_activation(w(ctx, x, name), act, 0, 0, self.inter, self.limit, self.limit, self.alpha, None, False)
             return act
         api.swiglu(w(ctx, x, name), act, self.activation)
         return act

@@ -11,7 +11,8 @@ the scores for the choice of groups and experts only); ``group_score="top2"`` (a
 choice scores); ``renormalize`` off (the weights are the chosen scores as they are); ``activation="clamped"``: an expert is
 ``down(g' sigmoid(alpha g') (u' + 1))`` with ``g' = min(gate x, limit)`` and ``u' = clamp(up x, -limit, limit)``, the shared expert
 with a limit of its own; ``shared_gate``: the shared expert's output is multiplied by ``sigmoid(w_sg . x)``, one number a token,
-whose row rides behind the router's rows in one product.
+whose row rides behind the router's rows in one product; ``gated`` off: an expert is ``down(f(up x))`` with f one of the ungated
+activations; ``weight_scale`` multiplies the routing weights.
 
 The experts run as ONE gated product over the concatenation of all experts' gate and up rows (the shared expert's
 behind them) and ONE down product over the concatenated columns: a token's activations are multiplied by its
@@ -37,11 +38,14 @@ class MixtureOfExperts(FeedForward):
     def __init__(self, hidden: int, experts: int, top: int, inter: int, groups: int = 1, keep: int = 1, shared_inter: int = 0,
                  activation: str = "silu", names: dict | None = None, score: str = "softmax", correction: bool = False,
                  group_score: str = "max", renormalize: bool = True, limit: float = 0.0, shared_limit: float = 0.0, alpha: float = 1.702,
-                 shared_gate: bool = False):
+                 shared_gate: bool = False, gated: bool = True, weight_scale: float = 1.0):
         self.hidden, self.experts, self.top, self.inter = int(hidden), int(experts), int(top), int(inter)
         self.groups, self.keep, self.shared_inter = int(groups), int(keep), int(shared_inter or 0)
-        if activation != "clamped" and activation not in api.GATE_ACTIVATIONS:
+        self.gated, self.weight_scale = bool(gated), float(weight_scale)
+        if self.gated and activation != "clamped" and activation not in api.GATE_ACTIVATIONS:
             raise ValueError(f"gate activation {activation!r} is not 'clamped' or one of {sorted(api.GATE_ACTIVATIONS)}")
+        if not self.gated and (activation not in api.UNARY_ACTIVATIONS or activation == "xielu" or shared_inter):
+            raise ValueError("ungated experts have an activation without parameters and no shared expert beside them")
         if score not in ("softmax", "sigmoid") or group_score not in ("max", "top2"):
             raise ValueError("routing scores are 'softmax' or 'sigmoid', group scores 'max' or 'top2'")
         self.score, self.group_score, self.renormalize = score, group_score, bool(renormalize)
@@ -58,6 +62,7 @@ class MixtureOfExperts(FeedForward):
         self.names = {**self.NAMES, **(names or {})}
         self.router: Linear | None = None
         self.gate_up: GatedLinear | None = None
+        self.up: Linear | None = None           # ungated experts: all up rows
         self.down: Linear | None = None
 
     def _expert_names(self, prefix: str) -> tuple[str, str, str]:
@@ -74,7 +79,8 @@ class MixtureOfExperts(FeedForward):
         out = {}
         for prefix, inter in self._prefixes():
             gate, up, down = self._expert_names(prefix)
-            out[gate] = WeightDecl((inter, self.hidden))
+            if self.gated:
+                out[gate] = WeightDecl((inter, self.hidden))
             out[up] = WeightDecl((inter, self.hidden))
             out[down] = WeightDecl((self.hidden, inter))
         out[self.names["router"]] = WeightDecl((self.experts, self.hidden))
@@ -86,8 +92,12 @@ class MixtureOfExperts(FeedForward):
 
     def bind(self, tensors, dtype, device) -> None:
         names = [self._expert_names(prefix) for prefix, _ in self._prefixes()]
-        self.gate_up = GatedLinear(torch.cat([tensors[g] for g, _, _ in names], dim=0), torch.cat([tensors[u] for _, u, _ in names], dim=0),
-                                   None, None, "silu" if self.activation == "clamped" else self.activation)
+        up = torch.cat([tensors[u] for _, u, _ in names], dim=0)
+        if self.gated:
+            self.gate_up = GatedLinear(torch.cat([tensors[g] for g, _, _ in names], dim=0), up, None, None,
+                                       "silu" if self.activation == "clamped" else self.activation)
+        else:
+            self.up = Linear(up)
         self.down = Linear(torch.cat([tensors[d] for _, _, d in names], dim=1))
         # the router's sums are float32 in both dtypes; its matrix stays as stored (widening bfloat16 changes nothing)
         router = tensors[self.names["router"]]
@@ -98,7 +108,7 @@ class MixtureOfExperts(FeedForward):
             self.correction = tensors[self.names["correction"]].to(torch.float32).contiguous()
 
     def projections(self) -> list:
-        return [self.router, self.gate_up.fused, self.down]
+        return [self.router, self.gate_up.fused if self.gated else self.up, self.down]
 
     def device_driven(self) -> bool:
         return True
@@ -110,13 +120,15 @@ class MixtureOfExperts(FeedForward):
         chosen = ctx.scratch("moe.chosen", (tokens, self.top), torch.int32)
         weights = ctx.scratch("moe.weights", (tokens, self.top), torch.float32)
         options = {"score": self.score, "correction": self.correction, "group_score": self.group_score, "renormalize": self.renormalize,
-                   "extra": extra}
+                   "extra": extra, "weight_scale": self.weight_scale}
         if api.route_rows_takes(self.hidden, self.experts + extra):
             api.route_rows(x, self.router.weight, self.top, self.groups, self.keep, gates, chosen, weights, **options)
         else:                                   # rows too wide to stage: the exact product, then the routing
             logits = ctx.scratch("moe.router", (1, tokens, self.experts + extra), torch.float32)
             api.gemm_simt(x, self.router.weight, None, logits)
             api.route_topk(logits, self.top, self.groups, self.keep, gates, chosen, weights, **options)
+        if not self.gated:
+            return self.down.delta(ctx, self.ungated(ctx, x, gates), "moe.down")
         if self.activation == "clamped":
             act = ctx.scratch("moe.gate_up.act", (tokens, self.experts * self.inter + self.shared_inter))
             w = self.gate_up.fused.weight
@@ -135,3 +147,9 @@ class MixtureOfExperts(FeedForward):
         if extra:
             raise NotImplementedError("a gated shared expert goes with the clamped unit")
         return self.down.delta(ctx, act, "moe.down")
+
+    def ungated(self, ctx, x, gates) -> torch.Tensor:
+        """``f(up x)`` of every expert's columns times the token's weight for the expert."""
+        act = ctx.scratch("moe.up.act", (ctx.n_tokens, self.experts * self.inter))
+        api.expert_unary_activation(self.up(ctx, x, "moe.up"), act, self.inter, self.activation, gates)
+        return act

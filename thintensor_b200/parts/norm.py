@@ -9,14 +9,15 @@ The delta that a norm adds may ask for more on the way (see :class:`~thintensor_
 normalised itself before the stream takes it, and for the stream to be replaced, after the addition, by a weighted sum
 of the layers' results so far.  The RMS norm's kernel does all of it in its one pass over a row.  Or it may bring two
 sublayers' outputs with a common factor and something else to add; both norms' kernels take those, and two norms of the
-same kind over the same stream (a parallel layer's) are one kernel.
+same kind over the same stream (a parallel layer's) are one kernel.  Or it may bring a factor per channel, and weights with
+which a stream in several copies takes the delta and is read: the RMS norm has a kernel for those.
 """
 from __future__ import annotations
 
 import torch
 
 from ..kernels import api
-from .base import NORMS, Delta, Norm, PostNorm, WeightDecl
+from .base import NORMS, Delta, Norm, PostNorm, StreamStep, WeightDecl
 
 
 @NORMS.register("rmsnorm")
@@ -48,7 +49,7 @@ class RMSNorm(Norm):
     def forward(self, ctx, residual, delta: Delta | None, out, rows=None) -> None:
         if delta is not None and (delta.post is not None or delta.depth is not None):
             post, depth = delta.post, delta.depth
-            if delta.branched:
+            if delta.branched or delta.streamed:
                 raise NotImplementedError("a delta that is normalised or mixed on its way brings one sublayer's output without a factor")
             if post is not None and delta.tensor is None:
                 raise RuntimeError("a delta that is already in the stream cannot be normalised on its way there")
@@ -57,6 +58,13 @@ class RMSNorm(Norm):
                                   0 if depth is None else depth.index, None if depth is None else depth.weights, self.weight,
                                   self.weight_offset, self.eps, out, rows)
             return
+        if delta is not None and delta.streamed:
+            if delta.second is not None or delta.addend is not None:
+                raise NotImplementedError("a delta with factors per channel or several streams brings one sublayer's output")
+            step = delta.streams or StreamStep()
+            api.stream_norm(residual, delta.tensor, delta.scale, delta.gain, step.mix, step.write, step.read, step.spread, self.weight,
+                            self.weight_offset, self.eps, out, rows)
+            return
         if delta is not None and delta.branched:
             api.add_norms(residual, delta.tensor, delta.second, delta.scale, delta.addend, self.weight, None, out, self.eps, False,
                           self.weight_offset, rows=rows)
@@ -64,7 +72,7 @@ class RMSNorm(Norm):
         api.add_rmsnorm(residual, None if delta is None else delta.tensor, self.weight, self.eps, out, rows, self.weight_offset)   # an empty delta is already in the stream
 
     def forward_pair(self, ctx, residual, delta: Delta | None, out, other, other_out) -> None:
-        special = delta is not None and (delta.post is not None or delta.depth is not None)
+        special = delta is not None and (delta.post is not None or delta.depth is not None or delta.streamed)
         if special or not isinstance(other, RMSNorm) or (other.eps, other.weight_offset) != (self.eps, self.weight_offset):
             return super().forward_pair(ctx, residual, delta, out, other, other_out)
         delta = delta or Delta(None)
@@ -101,15 +109,15 @@ class LayerNorm(Norm):
         return True
 
     def forward(self, ctx, residual, delta: Delta | None, out, rows=None) -> None:
-        if delta is not None and (delta.post is not None or delta.depth is not None):
-            raise NotImplementedError("the layer norm's kernel neither normalises a delta nor mixes results")
+        if delta is not None and (delta.post is not None or delta.depth is not None or delta.streamed):
+            raise NotImplementedError("the layer norm's kernel neither normalises a delta nor mixes results or streams")
         if delta is not None and delta.branched:
             api.add_norms(residual, delta.tensor, delta.second, delta.scale, delta.addend, self.weight, self.shift, out, self.eps, True, rows=rows)
             return
         api.add_layernorm(residual, None if delta is None else delta.tensor, self.weight, self.shift, self.eps, out, rows)
 
     def forward_pair(self, ctx, residual, delta: Delta | None, out, other, other_out) -> None:
-        special = delta is not None and (delta.post is not None or delta.depth is not None)
+        special = delta is not None and (delta.post is not None or delta.depth is not None or delta.streamed)
         if special or not isinstance(other, LayerNorm) or other.eps != self.eps:
             return super().forward_pair(ctx, residual, delta, out, other, other_out)
         delta = delta or Delta(None)

@@ -62,14 +62,16 @@ def _low_rank_decls(down: str, up: str, inputs: int, rank: int, outputs: int) ->
 
 class LowRankProduct:
     """The second half of a product of low rank, ``W_up`` on columns ``col ..`` of an input product (which ends with the ``W_down``
-    rows), and what is made of it: nothing (``plain``), a ``delta_decay`` or a ``sigmoid_root`` (see :class:`api.LowRank`).  Few
+    rows), and what is made of it: nothing (``plain``), a ``delta_decay``, a ``sigmoid_root`` or an ``exp_decay`` (see
+    :class:`api.LowRank`).  ``tanh``: the columns pass tanh first.  Few
     tokens run one kernel that does all of it in float32 for up to two such products of one layer; for many the columns become
     a matrix of the activation dtype and the product one like any other."""
 
     FEW_TOKENS = 128
 
     def __init__(self, tensors, down: str, up: str, col: int, name: str, kind: str = "plain", bias: torch.Tensor | None = None,
-                 a_log: torch.Tensor | None = None, per_head: int = 1, tau: float = 1.0):
+                 a_log: torch.Tensor | None = None, per_head: int = 1, tau: float = 1.0, tanh: bool = False):
+        self.tanh = bool(tanh)
         if tensors[down].shape[0] != tensors[up].shape[1]:
             raise ValueError(f"{down!r} makes {tensors[down].shape[0]} numbers, {up!r} takes {tensors[up].shape[1]}")
         self.up = Linear(tensors[up])
@@ -83,7 +85,7 @@ class LowRankProduct:
         tokens = proj.shape[1]
         if tokens <= LowRankProduct.FEW_TOKENS:
             out = [ctx.scratch(p.name, (1, tokens, p.cols), torch.float32) for p in products]
-            jobs = [api.LowRank(p.col, p.transposed, o[0], p.kind, p.bias, p.a_log, p.per_head, p.tau) for p, o in zip(products, out)]
+            jobs = [api.LowRank(p.col, p.transposed, o[0], p.kind, p.bias, p.a_log, p.per_head, p.tau, p.tanh) for p, o in zip(products, out)]
             if len({p.transposed.dtype for p in products}) == 1:
                 api.low_rank(proj, jobs)
             else:
@@ -91,7 +93,7 @@ class LowRankProduct:
                     api.low_rank(proj, [job])
             return out
         inputs = [ctx.scratch(p.name + ".in", (tokens, p.rank)) for p in products]
-        api.low_rank_inputs(proj, [(p.col, x) for p, x in zip(products, inputs)])
+        api.low_rank_inputs(proj, [(p.col, x, p.tanh) for p, x in zip(products, inputs)])
         out = []
         for p, x in zip(products, inputs):
             z = p.up(ctx, x, p.name)
@@ -102,7 +104,7 @@ class LowRankProduct:
         return out
 
 
-def _in_blocks(ctx) -> bool:
+def in_blocks(ctx) -> bool:
     """Whether a recurrence with decays per channel takes its tokens four at a time: prompts do (decided by the step's
     shape alone, so a replayed step and the step it was captured from agree)."""
     return not ctx.decode and ctx.n_tokens >= 4 * ctx.sequences
@@ -272,7 +274,7 @@ class GatedDelta(Mixer):
         qkv = ctx.scratch("delta.qkv", (tokens, self.channels), torch.float32)
         api.causal_conv(proj, 0, self.channels, self.conv_weight, None, True, tail, qkv, ctx.cu, ctx.slots, ctx.sequences, tokens, ctx.decode)
         read = ctx.scratch("delta.read", (tokens, self.v), torch.float32)
-        if decay is not None and _in_blocks(ctx):
+        if decay is not None and in_blocks(ctx):
             api.row_decay_blocks(qkv[:, :self.qk], qkv[:, self.qk: 2 * self.qk], qkv[:, 2 * self.qk:], decay, recurrent, read, ctx.cu, ctx.slots,
                                  ctx.sequences, self.heads, self.qk_heads, self.key_dim, self.value_dim, self.key_dim ** -0.5, (proj, self.b_col))
         else:
@@ -381,7 +383,7 @@ class DecayLinearAttention(Mixer):
         decay = None
         if self.low_rank is not None:
             decay = LowRankProduct.run(ctx, proj, [self.low_rank])[0][0]
-        blocks = decay is not None and _in_blocks(ctx)
+        blocks = decay is not None and in_blocks(ctx)
         if blocks and proj.shape[0] == 1 and not rotary_dim and self.activation is None and self.key_scale == 1.0:
             q, k, v = proj[0].split((self.qk, self.qk, self.v, proj.shape[2] - 2 * self.qk - self.v), dim=1)[:3]     # the product as it is
             api.row_decay_blocks(q, k, v, decay, recurrent, read, ctx.cu, ctx.slots, ctx.sequences, self.heads, self.heads, self.key_dim,

@@ -60,8 +60,16 @@ class ModelSpec:
     schedule: tuple[Run, ...]
     final_norm: PartSpec
     head: PartSpec
+    streams: int | None = None      # copies of the residual stream (None: one, without an axis of its own)
 
     def validate(self) -> None:
+        if self.streams is not None and self.streams < 1:
+            raise ValueError(f"a model has at least one residual stream, not {self.streams}")
+        if self.streams is not None and any(run.add_embedding for run in self.schedule):
+            raise ValueError("runs that add the embedding's output go with a single residual stream")
+        for index, layer in enumerate(self.layers):
+            if ("mixer_streams" in layer.parts) != (self.streams is not None):
+                raise ValueError(f"layer {index}: a model with several residual streams has weights for them in every layer, another in none")
         for index, run in enumerate(self.schedule):
             if run.add_embedding and index == 0:
                 raise ValueError("the schedule's first run already starts from the embedding's output")

@@ -35,6 +35,8 @@ def draw(decl: WeightDecl, generator: torch.Generator) -> torch.Tensor:
         weights = 0.3 * noise
         weights.view(-1)[-1] += 1.0
         return weights
+    if decl.init == "identity":
+        return torch.eye(*decl.shape) + 0.1 * noise
     raise ValueError(f"unknown initialisation {decl.init!r}")
 
 
