@@ -113,6 +113,7 @@ NERUZEN_SHAPES = {"1b": "neruzen-w2048", "3b": "neruzen-w3072"}
 SOGIDRA_SHAPES = {"1b": "sogidra-w2048", "3b": "sogidra-w3072"}
 KEREPEL_SHAPES = {"1b": "kerepel-w2048", "3b": "kerepel-w3072"}
 ZUVEPEL_SHAPES = {"1b": "zuvepel-w2048", "3b": "zuvepel-w3072"}
+ZEZILIX_SHAPES = {"1b": "zezilix-w2048", "3b": "zezilix-w3072"}
 
 
 def neruzen_pair(size: str) -> tuple[dict, dict]:
@@ -142,6 +143,16 @@ def zuvepel_pair(size: str) -> tuple[dict, dict]:
     return json.loads(json.dumps(SHAPES[ZUVEPEL_SHAPES[size]])), json.loads(json.dumps(SHAPES[FAMALORN_SHAPES[size]]))
 
 
+def zezilix_pair(size: str) -> tuple[dict, dict]:
+    """(Zezilix config.json, Neruzen config.json) of one size from the table of named shapes: the same width, vocabulary and
+    number of layers (six, each run once), two of them latent attention.  Neruzen is the closest model: latent attention with
+    the same ranks, softmax-routed experts, linear attentions behind a token shift.  Zezilix's other four layers are wkv (16 or
+    24 heads of 128); its mixtures have 16 ungated experts of 2,048 of which a token takes 6, so a token's feed-forward
+    multiplies with as many numbers as Neruzen's (and as the dense ones of 8,192); its stream comes in 2 copies at width 2,048 and in 4
+    at width 3,072, where one latent layer's heads have 96 numbers."""
+    return json.loads(json.dumps(SHAPES[ZEZILIX_SHAPES[size]])), json.loads(json.dumps(SHAPES[NERUZEN_SHAPES[size]]))
+
+
 def sogidra_pair(size: str) -> tuple[dict, dict]:
     """(Sogidra config.json, Llama config.json) of one size from the table of named shapes: the same width, feed-forward
     width, vocabulary and number of layers (six).  The Llama decoder is the closest model: both are attention over the
@@ -167,7 +178,8 @@ def design_bench(args) -> int:
     """``--design famalorn``: prefill and decode of the Famalorn design beside the Llama decoder at equal size (random
     weights, bfloat16), with each step's time by class of kernel against that class's bound.  ``--design neruzen``: the
     same for the Neruzen design beside Famalorn, ``--design sogidra`` for the Sogidra design beside Llama, ``--design kerepel``
-    for the Kerepel design beside Neruzen, ``--design zuvepel`` for the Zuvepel design beside Famalorn.  One JSON line."""
+    for the Kerepel design beside Neruzen, ``--design zuvepel`` for the Zuvepel design beside Famalorn,
+    ``--design zezilix`` for the Zezilix design beside Neruzen.  One JSON line."""
     import thintensor_b200
     from thintensor_b200.benchmark import class_fractions, measure_classes, measure_decode, measure_prefill
 
@@ -175,7 +187,7 @@ def design_bench(args) -> int:
     import torch
     names, pair = {"famalorn": (("famalorn", "llama"), famalorn_pair), "neruzen": (("neruzen", "famalorn"), neruzen_pair),
                    "sogidra": (("sogidra", "llama"), sogidra_pair), "kerepel": (("kerepel", "neruzen"), kerepel_pair),
-                   "zuvepel": (("zuvepel", "famalorn"), zuvepel_pair)}[args.design]
+                   "zuvepel": (("zuvepel", "famalorn"), zuvepel_pair), "zezilix": (("zezilix", "neruzen"), zezilix_pair)}[args.design]
     out = {"bench": f"{names[0].capitalize()} beside {names[1].capitalize()} at equal width, feed-forward, vocabulary and layers; random weights, bfloat16",
            "prompt_len": args.prompt_len, "batch": args.batch, "peaks": pk, "sizes": {}}
     for size in args.sizes.split(","):
@@ -224,8 +236,8 @@ def main() -> int:
     parser.add_argument("--batch", type=int, default=BATCH, help="with --only decode: sequences decoded together")
     parser.add_argument("--shape", choices=sorted(SHAPE_NAMES), default="1b", help="with --only: layer sizes of another model of the family")
     parser.add_argument("--prompt-len", type=int, default=PROMPT, help="with --only: tokens per prompt (the context is this plus room for the steps)")
-    parser.add_argument("--design", choices=["famalorn", "neruzen", "sogidra", "kerepel", "zuvepel"],
-                        help="measure this design beside the closest model the library has at equal size (Famalorn beside Llama, Neruzen beside Famalorn, Sogidra beside Llama, Kerepel beside Neruzen, Zuvepel beside Famalorn) instead of the headline")
+    parser.add_argument("--design", choices=["famalorn", "neruzen", "sogidra", "kerepel", "zuvepel", "zezilix"],
+                        help="measure this design beside the closest model the library has at equal size (Famalorn beside Llama, Neruzen beside Famalorn, Sogidra beside Llama, Kerepel beside Neruzen, Zuvepel beside Famalorn, Zezilix beside Neruzen) instead of the headline")
     parser.add_argument("--sizes", default="1b,3b", help="with --design: which sizes (1b: width 2,048; 3b: width 3,072)")
     args = parser.parse_args()
     if args.design:

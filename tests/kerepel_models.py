@@ -144,7 +144,8 @@ def oracle_logits(folder: Path, tokens: list[int]) -> torch.Tensor:
 
 def oracle_sensitivity(folder: Path, tokens: list[int]) -> torch.Tensor:
     """Per position, one minus the cosine between the plain implementation's logits and its logits with every operand of
-    a matrix product narrowed to bfloat16 on the way: how far the rounding of activations alone carries that position."""
+    a matrix product narrowed to bfloat16 on the way: how far the rounding of activations alone carries that position.  The
+    larger of two roundings of the same precision, on grids a little apart: a router's close call may fall with one and stand with the other."""
     import plain_kerepel
 
     key = ("sensitivity", str(folder), tuple(tokens))
@@ -152,8 +153,8 @@ def oracle_sensitivity(folder: Path, tokens: list[int]) -> torch.Tensor:
         want = oracle_logits(folder, tokens)
         cfg, weights = _oracle[("model", str(folder))]
         with torch.no_grad():
-            other = plain_kerepel.forward(cfg, weights, tokens, narrow=lambda x: x.to(torch.bfloat16).to(x.dtype))
-        _oracle[key] = 1.0 - torch.nn.functional.cosine_similarity(want, other, dim=-1)
+            others = [plain_kerepel.forward(cfg, weights, tokens, narrow=lambda x, f=factor: (x * f).to(torch.bfloat16).to(x.dtype) / f) for factor in (1.0, 1.37)]
+        _oracle[key] = torch.stack([1.0 - torch.nn.functional.cosine_similarity(want, other, dim=-1) for other in others]).max(dim=0).values
     return _oracle[key]
 
 

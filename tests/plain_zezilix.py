@@ -109,8 +109,9 @@ def latent_attention(h, w, p, m, eps, low_rank_queries, gated):
     c = nar(rms(down[:, :C], eps) * w[p + "dkv.norm"])
     k_rot = nar(rotate_pairs(down[:, None, C:], torch.arange(T), m["rot"])[:, 0])
     q_rot = nar(rotate_pairs(q[..., D:], torch.arange(T), m["rot"]))
-    k = (c @ w[p + "uk"].T).reshape(T, H, D)
-    v = (c @ w[p + "uv"].T).reshape(T, H, V)
+    q = nar(q)
+    k = nar(c @ w[p + "uk"].T).reshape(T, H, D)
+    v = nar(c @ w[p + "uv"].T).reshape(T, H, V)
     out = torch.zeros(T, H, V, dtype=h.dtype)
     for t in range(T):
         s = (torch.einsum("hd,jhd->hj", q[t, :, :D], k[:t + 1]) + q_rot[t] @ k_rot[:t + 1].T) * m["scale"]
@@ -141,7 +142,7 @@ def wkv(h, w, p, m, eps):
     mixed = {s: nar(shifted(h, w[p + "mu." + s])) for s in "rkvgw"}
     r, k, v = ((mixed[s] @ w[p + s].T).reshape(T, H, D) for s in "rkv")
     gate = silu(mixed["g"] @ w[p + "g"].T)
-    decay = torch.exp(-torch.exp(torch.tanh(mixed["w"] @ w[p + "w1"].T) @ w[p + "w2"].T + w[p + "w0"])).reshape(T, H, D)
+    decay = torch.exp(-torch.exp(nar(torch.tanh(mixed["w"] @ w[p + "w1"].T)) @ w[p + "w2"].T + w[p + "w0"])).reshape(T, H, D)
     o = rms(bonus_recurrence(r, k, v, decay, w[p + "u"]), eps).reshape(T, H * D)
     return nar(o * w[p + "norm"] * gate) @ w[p + "o"].T
 

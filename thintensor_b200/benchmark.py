@@ -19,7 +19,7 @@ from .sampling.sampler import SamplingParams
 
 # Named shapes for benchmarks with random weights, each a whole config.json: the three Llama 3
 # models the reference's reports measure, two tiny ones that differ in every size and option, and
-# two Famalorn, two Neruzen, two Sogidra, two Kerepel and two Zuvepel models of six layers at the widths of the 1B and 3B Llama shapes.
+# two Famalorn, two Neruzen, two Sogidra, two Kerepel, two Zuvepel and two Zezilix models of six layers at the widths of the 1B and 3B Llama shapes.
 # They are data (config/shapes.json), read here and by bench.py.
 SHAPES: dict[str, dict] = json.loads((Path(__file__).resolve().parent / "config" / "shapes.json").read_text(encoding="utf-8"))
 
@@ -201,7 +201,7 @@ def class_fractions(model, classes: dict, pk: dict, prefill_prompts: list[list[i
     one after another (see :func:`measure_classes`)."""
     attention_kernels = ("tt_attention", "tt_latent_attention", "tt_differential_attention", "tt_pooled_window_attention")
     recurrent = ("tt_mamba2_scan", "tt_delta_scan", "tt_causal_conv", "tt_gated_group_norm", "tt_decay_scan", "tt_row_decay_scan", "tt_row_decay_blocks",
-                 "tt_low_rank", "tt_low_rank_inputs", "tt_low_rank_finish", "tt_linear_attention_prepare")
+                 "tt_low_rank", "tt_low_rank_inputs", "tt_low_rank_finish", "tt_linear_attention_prepare", "tt_token_shifts")
 
     def split(spans: dict) -> dict:
         out = {"products": 0.0, "attention": 0.0, "recurrence": 0.0, "rest": 0.0}

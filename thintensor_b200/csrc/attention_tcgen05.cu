@@ -93,6 +93,7 @@ struct Args {
     float scale_log2;
     int window;
     __nv_bfloat16* out;
+    int out_dim;            // numbers of a head's output that are written (the head size, or fewer for padded heads)
     unsigned* status;
     const float* sinks;     // one per query head, or null: exp(sink) joins the softmax denominator, with no key, no value and no scale
     // the SHAPED instances only: a scaled score s becomes softcap * tanh(s / softcap) (softcap > 0), slopes[head] * (query
@@ -428,7 +429,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             fence_after_sync();
             const float inv = l > 0.0f ? 1.0f / l : 0.0f;
             const int token = seq_begin + tok0 + local, head = kh * args.group + (r - local * args.group);
-            __nv_bfloat16* dst = args.out + ((size_t)token * args.heads + head) * HD + half * O_COLS;
+            __nv_bfloat16* dst = args.out + ((size_t)token * args.heads + head) * args.out_dim + half * O_COLS;
             const bool gated = SHAPED && args.gate != nullptr && row_ok;
             float head_gate = 1.0f;
             if (gated && args.gate_per_head) {
@@ -457,6 +458,13 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                 if (row_ok) {
 #pragma unroll
                     for (int e = 0; e < 32; e += 8) {
+                        const int room = args.out_dim - (half * O_COLS + c + e);     // numbers of a head's output left (all eight, but for heads that are padded)
+                        if (room < 8 || (args.out_dim & 7)) {
+#pragma unroll
+                            for (int i = 0; i < 8; ++i)
+                                if (i < room) dst[c + e + i] = __float2bfloat16_rn(o[e + i] * inv);
+                            continue;
+                        }
                         uint4 v;
                         __nv_bfloat162 h0 = __floats2bfloat162_rn(o[e] * inv, o[e + 1] * inv), h1 = __floats2bfloat162_rn(o[e + 2] * inv, o[e + 3] * inv);
                         __nv_bfloat162 h2 = __floats2bfloat162_rn(o[e + 4] * inv, o[e + 5] * inv), h3 = __floats2bfloat162_rn(o[e + 6] * inv, o[e + 7] * inv);
@@ -514,17 +522,20 @@ extern "C" int tt_attention_tcgen05_supports(int heads, int kv_heads, int head_d
 }
 
 // Packed prompts (any number of tokens per sequence) attending over the block cache; the
-// new tokens' keys and values are already in the cache.  Returns a cudaError_t value, or -1
+// new tokens' keys and values are already in the cache.  out_dim: the first so many numbers of a head's output are written, side by
+// side (head_dim, but for heads that are padded to a size the kernel takes).  Returns a cudaError_t value, or -1
 // if the tensor maps could not be made.
 extern "C" int tt_attention_tcgen05(const void* q, const void* k_pool, const void* v_pool, const int* table, int table_width,
                                     int pool_blocks, const int* cu, const int* len_before, int sequences, int n_tokens,
                                     int heads, int kv_heads, int head_dim, float scale, const float* sinks, int window, void* out,
                                     unsigned* status, float softcap, const float* slopes, const float* gate, int gate_splits,
-                                    long long gate_split_stride, int gate_row, int gate_per_head, cudaStream_t stream) {
+                                    long long gate_split_stride, int gate_row, int gate_per_head, int out_dim, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (!tt_attention_tcgen05_supports(heads, kv_heads, head_dim) || ((uintptr_t)q & 15) || ((uintptr_t)k_pool & 15) || ((uintptr_t)v_pool & 15))
         return (int)cudaErrorInvalidValue;
+    if (out_dim < 1 || out_dim > head_dim || (gate && out_dim != head_dim)) return (int)cudaErrorInvalidValue;
     Args args;
+    args.out_dim = out_dim;
     args.table = table; args.table_width = table_width; args.pool_blocks = pool_blocks; args.cu = cu; args.len_before = len_before;
     args.sequences = sequences; args.heads = heads; args.kv_heads = kv_heads; args.group = heads / kv_heads;
     args.tokens_per_tile = ROWS / args.group;

@@ -94,7 +94,13 @@ struct Args {
     QkvRope rope;            // qkv form only
     int rope_head_dim;       // 64 or 128
     int undelivered_bytes;   // 0 in every real call; tests: the first stage's barrier expects this many bytes that no copy brings
-    int activation;          // SWIGLU forms: what the gate passes through: 0 silu, 1 relu, 2 the tanh form of gelu, 3 the clamped unit
+    int activation;          // SWIGLU forms: what the gate passes through: 0 silu, 1 relu, 2 the tanh form of gelu, 3 the clamped unit; 4: no gate (see below)
+    // no gate (persistent and pair kernels with tiled copies only): the "gate" and "up" rows are the two halves of one matrix, and
+    // each half's products leave as f(z) * scales[token][feature / scale_width], f by `unary`: 0 silu, 1 relu, 2 the tanh form of gelu,
+    // 5 the square of relu.  scale_width is a multiple of a tile's 128 features, so a tile's half has one factor a token.
+    int unary;
+    const float* scales;
+    int scale_row, scale_width;
     // the clamped unit: with g' = min(g, limit) and u' = clamp(u, -limit, limit) the output is g' sigmoid(alpha g') (u' + 1); output
     // features below clamp_split use clamp_low as their limit, the others clamp_high (a limit of 0 or less: no clamp)
     float clamp_low, clamp_high, clamp_alpha;
@@ -572,6 +578,68 @@ __device__ __forceinline__ void store_swiglu_bulk(uint32_t lane_addr, int first_
     }
 }
 
+// The form without a gate: columns 0..127 of the accumulator are 128 features from f_base, columns 128..255 the 128 features from
+// args.features (half of all) + f_base.  Each becomes f(z) times its token's factor and leaves through a slab of its own, so both
+// slabs must be free before a chunk's are filled.
+__device__ __forceinline__ void store_unary_bulk(uint32_t lane_addr, int first_token, int f_base, const Args& args, const CUtensorMap* map_out,
+                                                 uint8_t* slabs, int lane) {
+    const bool wanted = first_token < args.tokens;                             // the same for the whole warp
+    const int token = first_token + lane;
+    float factor[2] = {1.0f, 1.0f};
+    if (args.scales && token < args.tokens) {
+#pragma unroll
+        for (int half = 0; half < 2; ++half)
+            factor[half] = __ldg(args.scales + (size_t)token * args.scale_row + (f_base + half * args.features) / args.scale_width);
+    }
+    uint32_t z[2][2][32];                                                      // [buffer][half]
+    tmem_load32_issue(lane_addr, z[0][0]);
+    tmem_load32_issue(lane_addr + 128, z[0][1]);
+#pragma unroll
+    for (int ci = 0; ci < 4; ++ci) {
+        const int cur = ci & 1;
+        tmem_load_wait();
+        if (ci + 1 < 4) {
+            tmem_load32_issue(lane_addr + 32 * ci + 32, z[cur ^ 1][0]);
+            tmem_load32_issue(lane_addr + 128 + 32 * ci + 32, z[cur ^ 1][1]);
+        }
+        if (!wanted) continue;
+        if ((ci & 1) == 0) {
+            if (lane == 0) bulk_wait_group_read<0>();
+            __syncwarp();
+        }
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+#pragma unroll
+            for (int e0 = 0; e0 < 32; e0 += 8) {
+                float y[8];
+                if (args.unary == 5) {
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) { const float p = fmaxf(tmem_loaded(z[cur][half][e0 + e]), 0.0f); y[e] = p * p * factor[half]; }
+                } else {
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) y[e] = gate_activation(tmem_loaded(z[cur][half][e0 + e]), args.unary) * factor[half];
+                }
+                const __nv_bfloat162 p0 = __floats2bfloat162_rn(y[0], y[1]), p1 = __floats2bfloat162_rn(y[2], y[3]);
+                const __nv_bfloat162 p2 = __floats2bfloat162_rn(y[4], y[5]), p3 = __floats2bfloat162_rn(y[6], y[7]);
+                const int piece = (ci & 1) * 4 + (e0 >> 3);
+                *reinterpret_cast<uint4*>(slabs + half * 4096 + lane * 128 + ((piece ^ (lane & 7)) << 4)) =
+                    make_uint4(*reinterpret_cast<const uint32_t*>(&p0), *reinterpret_cast<const uint32_t*>(&p1),
+                               *reinterpret_cast<const uint32_t*>(&p2), *reinterpret_cast<const uint32_t*>(&p3));
+            }
+        }
+        if (ci & 1) {
+            fence_async_shared();
+            __syncwarp();
+            if (lane == 0) {
+                const int f0 = f_base + 64 * (ci >> 1);
+                tma_store_2d(map_out, smem_u32(slabs), f0, first_token);
+                tma_store_2d(map_out, smem_u32(slabs + 4096), args.features + f0, first_token);
+                bulk_commit_group();
+            }
+        }
+    }
+}
+
 // A warp's 32 rows of an accumulator that holds only a share of the tile's k: four columns at a time into the warp's own
 // 32 KB of scratch memory, the 32 lanes' 16-byte pieces side by side (whole lines a store; the layout is nobody
 // else's business).  The pair that holds the tile's first k-blocks adds it to its own share (store_accumulator_bulk).
@@ -893,7 +961,10 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const 
                 // stored by qkv_row_epilogue
             } else if (bulk_out) {
                 if constexpr (FORM == TOKENS_ON_M) store_accumulator_bulk<WIDE>(lane_addr, token - lane, f_base, slice, args, &map_out, slabs, lane, round);
-                else if constexpr (dual) store_swiglu_bulk(lane_addr, token - lane, f_base, args, &map_out, slabs, lane, round);
+                else if constexpr (dual) {
+                    if (args.activation == 4) store_unary_bulk(lane_addr, token - lane, f_base, args, &map_out, slabs, lane);
+                    else store_swiglu_bulk(lane_addr, token - lane, f_base, args, &map_out, slabs, lane, round);
+                }
             } else if (dual || slice == 0) {
                 store_accumulator<dual, WIDE>(lane_addr, token, f_base, args);
             } else {                                            // a later k-slice: its own plane of the output, no bias
@@ -1102,7 +1173,8 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid
                     store_accumulator<dual>(lane_addr, token, f_base, args);
                 }
             } else if constexpr (dual) {
-                if (bulk_out) store_swiglu_bulk(lane_addr, token - lane, f_base, args, &map_out, slabs, lane, round);
+                if (bulk_out && args.activation == 4) store_unary_bulk(lane_addr, token - lane, f_base, args, &map_out, slabs, lane);
+                else if (bulk_out) store_swiglu_bulk(lane_addr, token - lane, f_base, args, &map_out, slabs, lane, round);
                 else store_accumulator<dual>(lane_addr, token, f_base, args);
             }                                                                // the qkv form has stored its row
             // this warp is done with the accumulator: tell the issuer, who sits in the even CTA
@@ -1317,11 +1389,12 @@ static bool deals_k_out(int tiles, int pairs, int k_blocks) {
 }
 
 struct GateClamp { float low, high, alpha; int split; };
+struct Unary { int activation; const float* scales; int row, width; };
 
 static int gemm_dispatch(const void* x, long long ldx, const void* w, long long ldw, const float* bias, void* out,
                          long long ld_out, long long split_stride, int tokens, int features, int k, int splits,
                          int form, unsigned* status, cudaStream_t stream, void* shares, long long shares_bytes, const GateClamp clamp,
-                         int group_features = 0) {
+                         int group_features = 0, const Unary unary = Unary{}) {
     if (tokens <= 0 || features <= 0) return 0;
     if (k <= 0 || (k % 8) || (ldx % 8) || (ldw % 8) || ((uintptr_t)x & 15) || ((uintptr_t)w & 15) || splits < 1)
         return (int)cudaErrorInvalidValue;
@@ -1329,7 +1402,7 @@ static int gemm_dispatch(const void* x, long long ldx, const void* w, long long 
     if (splits > k_blocks) splits = k_blocks;
     const int activation = form >> 4;       // the gated form carries its gate's activation in the bits above the form
     form &= 15;
-    if (activation < 0 || activation > 3 || (activation && form != 1)) return (int)cudaErrorInvalidValue;
+    if (activation < 0 || activation > 4 || (activation && form != 1)) return (int)cudaErrorInvalidValue;
     Args args;
     args.activation = activation;
     args.clamp_low = clamp.low; args.clamp_high = clamp.high; args.clamp_alpha = clamp.alpha; args.clamp_split = clamp.split;
@@ -1342,6 +1415,7 @@ static int gemm_dispatch(const void* x, long long ldx, const void* w, long long 
     args.bulk_out = 0;
     args.shares = nullptr;
     args.group_features = group_features;
+    args.unary = unary.activation; args.scales = unary.scales; args.scale_row = unary.row; args.scale_width = unary.width;
     const long long x_rows = group_features > 0 ? (long long)tokens * ((features + group_features - 1) / group_features) : tokens;
     if (x_rows > 2147483647LL) return (int)cudaErrorInvalidValue;
     CUtensorMap map_a, map_b;
@@ -1350,6 +1424,7 @@ static int gemm_dispatch(const void* x, long long ldx, const void* w, long long 
     if (form == 1) {
         if (splits != 1 || bias) return (int)cudaErrorInvalidValue;
         if (!make_map(&map_a, x, tokens, k, ldx, BM) || !make_map(&map_b, w, 2LL * features, k, ldw, 128)) return -1;
+        if (activation == 4 && tokens <= 128) return (int)cudaErrorInvalidValue;
         if (tokens <= 128) {
             // few tokens: features on the 128-row side, 64 gate rows paired with their 64 up rows
             const int bn = tokens <= 16 ? 16 : tokens <= 32 ? 32 : tokens <= 64 ? 64 : 128;
@@ -1367,11 +1442,12 @@ static int gemm_dispatch(const void* x, long long ldx, const void* w, long long 
         // a multiple of 16 bytes apart): boxes of 64 features x 32 tokens
         CUtensorMap map_out = map_a;
         if (tiles >= 8 && (ld_out % 8) == 0 && (((uintptr_t)out) & 15) == 0) {
-            const cuuint64_t dims[2] = {(cuuint64_t)features, (cuuint64_t)tokens};
+            const cuuint64_t dims[2] = {(cuuint64_t)(activation == 4 ? 2LL * features : features), (cuuint64_t)tokens};
             const cuuint64_t strides[1] = {(cuuint64_t)ld_out * 2};
             const cuuint32_t box[2] = {64, 32};
             args.bulk_out = tc::make_map(&map_out, out, 2, dims, strides, box) ? 1 : 0;
         }
+        if (activation == 4 && (!args.bulk_out || features % 128)) return (int)cudaErrorInvalidValue;
         if (tiles >= 8 && tokens < PAIR_MIN_TOKENS_SWIGLU) return launch_persistent<TOKENS_ON_M_SWIGLU>(map_a, map_b, map_out, args, tiles_m, tiles, 1, stream);
         if (tiles >= 8) {
             const int pair_tiles_m = (tokens + 2 * BM - 1) / (2 * BM);
@@ -1456,4 +1532,17 @@ extern "C" int tt_gemm_tcgen05_groups(const void* x, long long ldx, const void* 
     if (group_features <= 0 || group_features % (tokens > 128 ? 256 : 128)) return (int)cudaErrorInvalidValue;
     return gemm_dispatch(x, ldx, w, ldw, nullptr, out, ld_out, split_stride, tokens, features, k, splits, 0, status, stream, shares, shares_bytes,
                          GateClamp{0.0f, 0.0f, 1.0f, 0}, group_features);
+}
+
+// A product with an ungated activation and a factor per token and column range as its epilogue: act[t][f] = f(x[t] . w[f]) *
+// scales[t][f / scale_width] in bfloat16 (scales null: no factor).  Prompts whose tiles leave by tiled copies only: more than 128
+// tokens, features a multiple of 256, scale_width a multiple of 128, at least 8 tiles of 128 tokens x 256 features.
+extern "C" int tt_gemm_tcgen05_unary(const void* x, long long ldx, const void* w, long long ldw, void* out, long long ld_out, int tokens,
+                                     int features, int k, int activation, const float* scales, int scale_row, int scale_width,
+                                     unsigned* status, cudaStream_t stream) {
+    if (features % 256 || scale_width <= 0 || scale_width % 128 || (activation != 5 && (activation < 0 || activation > 2)) || (ld_out % 8) ||
+        ((uintptr_t)out & 15) || tokens <= 128 || ((tokens + BM - 1) / BM) * (features / 256) < 8)
+        return (int)cudaErrorInvalidValue;
+    return gemm_dispatch(x, ldx, w, ldw, nullptr, out, ld_out, 0, tokens, features / 2, k, 1, 1 + 16 * 4, status, stream, nullptr, 0,
+                         GateClamp{0.0f, 0.0f, 1.0f, 0}, 0, Unary{activation, scales, scale_row, scale_width});
 }

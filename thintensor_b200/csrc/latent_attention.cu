@@ -18,8 +18,10 @@
 // sigmoid of its gate number, or every output number by its own, where the layer has gates.
 //
 // Prompts may instead EXPAND the latents they can see into per-head keys and values for the step, laid out like blocks
-// of the ordinary cache (keys [block][head][64][dim + rot], values transposed [block][head][vdim][64]) with a table of
-// their own, so that the tensor-core attention kernels for ordinary heads run on them:
+// of the ordinary cache (keys [block][head][64][size], values transposed [block][head][size][64]) with a table of
+// their own, so that the tensor-core attention kernels for ordinary heads run on them.  size is the head size of those kernels, at
+// least dim + rot and vdim; queries and keys are zero beyond their dim + rot numbers, value rows beyond vdim are whatever they are
+// (they only reach output numbers that nobody writes):
 // tt_latent_expand_plan (which blocks of which sequence the step can see, and where they go), tt_latent_gather (their
 // latents into one matrix for the product with [Wk; Wv], their shared rotated parts into every head's keys),
 // tt_latent_scatter (the product's rows into keys and transposed values) and tt_latent_queries (rotated queries).
@@ -696,11 +698,11 @@ __global__ void latent_expand_plan_kernel(const int* __restrict__ cu, const int*
     }
 }
 
-// One block per row of the temporary blocks (block * 64 + token).  x: [rows][rank]; keys: [block][heads][64][dim + rot].
+// One block per row of the temporary blocks (block * 64 + token).  x: [rows][rank]; keys: [block][heads][64][size].
 template <typename T>
 __global__ void latent_gather_kernel(const T* __restrict__ pool, const int* __restrict__ table, int table_width, int pool_blocks,
                                      const int* __restrict__ cu, const int* __restrict__ len_before, int sequences,
-                                     const int* __restrict__ plan, int heads, int dim, int rot, int rank, T* __restrict__ x,
+                                     const int* __restrict__ plan, int heads, int dim, int rot, int rank, int size, T* __restrict__ x,
                                      T* __restrict__ keys) {
     tt_pdl_launch_dependents();
     tt_pdl_wait();
@@ -714,10 +716,10 @@ __global__ void latent_gather_kernel(const T* __restrict__ pool, const int* __re
     }
     const T zero = tt_from_float<T>(0.0f);
     for (int j = threadIdx.x; j < rank; j += blockDim.x) x[(size_t)row * rank + j] = off >= 0 ? pool[off + j] : zero;
-    const int hd = dim + rot;
-    for (int e = threadIdx.x; e < heads * rot; e += blockDim.x) {
-        const int h = e / rot, j = e - h * rot;
-        keys[(((size_t)tb * heads + h) * TT_BLOCK_TOKENS + r) * hd + dim + j] = off >= 0 ? pool[off + rank + j] : zero;
+    const int tail = size - dim;                                // the rotated part and the padding behind it
+    for (int e = threadIdx.x; e < heads * tail; e += blockDim.x) {
+        const int h = e / tail, j = e - h * tail;
+        keys[(((size_t)tb * heads + h) * TT_BLOCK_TOKENS + r) * size + dim + j] = off >= 0 && j < rot ? pool[off + rank + j] : zero;
     }
 }
 
@@ -725,19 +727,19 @@ __global__ void latent_gather_kernel(const T* __restrict__ pool, const int* __re
 // head: the unrotated key parts go out row by row, the values through shared memory so that a value number's 64 tokens
 // are written side by side.
 template <typename T>
-__global__ void latent_scatter_kernel(const float* __restrict__ y, int splits, size_t split_stride, int heads, int dim, int rot,
+__global__ void latent_scatter_kernel(const float* __restrict__ y, int splits, size_t split_stride, int heads, int dim, int size,
                                       int vdim, T* __restrict__ keys, T* __restrict__ values) {
     tt_pdl_launch_dependents();
     tt_pdl_wait();
     extern __shared__ float lat_shared[];                       // [64][vdim + 1]
     const int tb = blockIdx.x / heads, h = blockIdx.x - tb * heads;
-    const int cols = heads * (dim + vdim), hd = dim + rot;
+    const int cols = heads * (dim + vdim);
     const float* base = y + (size_t)tb * TT_BLOCK_TOKENS * cols;
     for (int e = threadIdx.x; e < TT_BLOCK_TOKENS * dim; e += blockDim.x) {
         const int r = e / dim, d = e - r * dim;
         float v = 0.0f;
         for (int s = 0; s < splits; ++s) v += base[(size_t)s * split_stride + (size_t)r * cols + h * dim + d];
-        keys[(((size_t)tb * heads + h) * TT_BLOCK_TOKENS + r) * hd + d] = tt_from_float<T>(v);
+        keys[(((size_t)tb * heads + h) * TT_BLOCK_TOKENS + r) * size + d] = tt_from_float<T>(v);
     }
     for (int e = threadIdx.x; e < TT_BLOCK_TOKENS * vdim; e += blockDim.x) {
         const int r = e / vdim, d = e - r * vdim;
@@ -748,16 +750,16 @@ __global__ void latent_scatter_kernel(const float* __restrict__ y, int splits, s
     __syncthreads();
     for (int e = threadIdx.x; e < TT_BLOCK_TOKENS * vdim; e += blockDim.x) {
         const int d = e / TT_BLOCK_TOKENS, r = e - d * TT_BLOCK_TOKENS;
-        values[(((size_t)tb * heads + h) * vdim + d) * TT_BLOCK_TOKENS + r] = tt_from_float<T>(lat_shared[r * (vdim + 1) + d]);
+        values[(((size_t)tb * heads + h) * size + d) * TT_BLOCK_TOKENS + r] = tt_from_float<T>(lat_shared[r * (vdim + 1) + d]);
     }
 }
 
 // q: float32 partial sums [splits][tokens][heads * (dim + rot)]; out: the same numbers in T with each head's last rot
-// numbers rotated by the token's position (the first rotary_dim of them, halves or neighbours paired); a token's row of q
-// is q_row numbers long.
+// numbers rotated by the token's position (the first rotary_dim of them, halves or neighbours paired) and padded with zeros to
+// `size` numbers a head; a token's row of q is q_row numbers long.
 template <typename T>
 __global__ void latent_queries_kernel(const float* __restrict__ q, int splits, size_t split_stride, int q_row, int heads, int dim, int rot,
-                                      const float* __restrict__ inv_freq, int rotary_dim, int interleaved, float rot_scale,
+                                      int size, const float* __restrict__ inv_freq, int rotary_dim, int interleaved, float rot_scale,
                                       const int* __restrict__ cu,
                                       const int* __restrict__ len_before, int sequences, T* __restrict__ out) {
     tt_pdl_launch_dependents();
@@ -767,8 +769,10 @@ __global__ void latent_queries_kernel(const float* __restrict__ q, int splits, s
     tt_pdl_wait();
     const int hd = dim + rot, half = rotary_dim >> 1;
     const float* row = q + (size_t)t * q_row;
-    for (int e = threadIdx.x; e < heads * hd; e += blockDim.x) {
-        const int i = e % hd - dim;                             // index inside the rotated part, negative in front of it
+    for (int o = threadIdx.x; o < heads * size; o += blockDim.x) {
+        const int h = o / size, d = o - h * size;
+        if (d >= hd) { out[(size_t)t * heads * size + o] = tt_from_float<T>(0.0f); continue; }
+        const int e = h * hd + d, i = d - dim;                  // i: index inside the rotated part, negative in front of it
         float x = 0.0f;
         for (int s = 0; s < splits; ++s) x += row[(size_t)s * split_stride + e];
         if (i >= 0 && i < rotary_dim) {
@@ -781,7 +785,7 @@ __global__ void latent_queries_kernel(const float* __restrict__ q, int splits, s
             sn *= rot_scale; cs *= rot_scale;
             x = first ? x * cs - other * sn : x * cs + other * sn;
         }
-        out[(size_t)t * heads * hd + e] = tt_from_float<T>(x);
+        out[(size_t)t * heads * size + o] = tt_from_float<T>(x);
     }
 }
 
@@ -795,38 +799,39 @@ extern "C" int tt_latent_expand_plan(const int* cu, const int* len_before, int s
 
 extern "C" int tt_latent_gather(const void* pool, int dtype, const int* table, int table_width, int pool_blocks, const int* cu,
                                 const int* len_before, int sequences, const int* plan, int bound_blocks, int heads, int dim, int rot,
-                                int rank, void* x, void* keys, cudaStream_t stream) {
+                                int rank, int size, void* x, void* keys, cudaStream_t stream) {
     if (bound_blocks <= 0) return 0;
+    if (size < dim + rot) return (int)cudaErrorInvalidValue;
     const dim3 grid((unsigned)bound_blocks * TT_BLOCK_TOKENS), block(128);
     if (dtype == TT_F32)
-        tt_launch_pdl(latent_gather_kernel<float>, grid, block, 0, stream, (const float*)pool, table, table_width, pool_blocks, cu, len_before, sequences, plan, heads, dim, rot, rank, (float*)x, (float*)keys);
+        tt_launch_pdl(latent_gather_kernel<float>, grid, block, 0, stream, (const float*)pool, table, table_width, pool_blocks, cu, len_before, sequences, plan, heads, dim, rot, rank, size, (float*)x, (float*)keys);
     else
-        tt_launch_pdl(latent_gather_kernel<__nv_bfloat16>, grid, block, 0, stream, (const __nv_bfloat16*)pool, table, table_width, pool_blocks, cu, len_before, sequences, plan, heads, dim, rot, rank, (__nv_bfloat16*)x, (__nv_bfloat16*)keys);
+        tt_launch_pdl(latent_gather_kernel<__nv_bfloat16>, grid, block, 0, stream, (const __nv_bfloat16*)pool, table, table_width, pool_blocks, cu, len_before, sequences, plan, heads, dim, rot, rank, size, (__nv_bfloat16*)x, (__nv_bfloat16*)keys);
     TT_LAUNCH_CHECK();
 }
 
-extern "C" int tt_latent_scatter(const float* y, int splits, long long split_stride, int bound_blocks, int heads, int dim, int rot, int vdim,
+extern "C" int tt_latent_scatter(const float* y, int splits, long long split_stride, int bound_blocks, int heads, int dim, int size, int vdim,
                                  void* keys, void* values, int dtype, cudaStream_t stream) {
     if (bound_blocks <= 0) return 0;
     const size_t shared = (size_t)TT_BLOCK_TOKENS * (vdim + 1) * sizeof(float);
-    if (shared > 48 * 1024) return (int)cudaErrorInvalidValue;
+    if (size < dim || size < vdim || shared > 48 * 1024) return (int)cudaErrorInvalidValue;
     const dim3 grid((unsigned)bound_blocks * heads), block(256);
     if (dtype == TT_F32)
-        tt_launch_pdl(latent_scatter_kernel<float>, grid, block, shared, stream, y, splits, (size_t)split_stride, heads, dim, rot, vdim, (float*)keys, (float*)values);
+        tt_launch_pdl(latent_scatter_kernel<float>, grid, block, shared, stream, y, splits, (size_t)split_stride, heads, dim, size, vdim, (float*)keys, (float*)values);
     else
-        tt_launch_pdl(latent_scatter_kernel<__nv_bfloat16>, grid, block, shared, stream, y, splits, (size_t)split_stride, heads, dim, rot, vdim, (__nv_bfloat16*)keys, (__nv_bfloat16*)values);
+        tt_launch_pdl(latent_scatter_kernel<__nv_bfloat16>, grid, block, shared, stream, y, splits, (size_t)split_stride, heads, dim, size, vdim, (__nv_bfloat16*)keys, (__nv_bfloat16*)values);
     TT_LAUNCH_CHECK();
 }
 
-extern "C" int tt_latent_queries(const float* q, int splits, long long split_stride, int q_row, int heads, int dim, int rot,
+extern "C" int tt_latent_queries(const float* q, int splits, long long split_stride, int q_row, int heads, int dim, int rot, int size,
                                  const float* inv_freq, int rotary_dim, int interleaved, float rot_scale, const int* cu, const int* len_before, int sequences, int n_tokens, void* out, int dtype,
                                  cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (rotary_dim > rot || (rotary_dim & 1)) return (int)cudaErrorInvalidValue;
+    if (rotary_dim > rot || (rotary_dim & 1) || size < dim + rot) return (int)cudaErrorInvalidValue;
     if (dtype == TT_F32)
-        tt_launch_pdl(latent_queries_kernel<float>, dim3(n_tokens), dim3(256), 0, stream, q, splits, (size_t)split_stride, q_row, heads, dim, rot, inv_freq, rotary_dim, interleaved, rot_scale, cu, len_before, sequences, (float*)out);
+        tt_launch_pdl(latent_queries_kernel<float>, dim3(n_tokens), dim3(256), 0, stream, q, splits, (size_t)split_stride, q_row, heads, dim, rot, size, inv_freq, rotary_dim, interleaved, rot_scale, cu, len_before, sequences, (float*)out);
     else
-        tt_launch_pdl(latent_queries_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(256), 0, stream, q, splits, (size_t)split_stride, q_row, heads, dim, rot, inv_freq, rotary_dim, interleaved, rot_scale, cu, len_before, sequences, (__nv_bfloat16*)out);
+        tt_launch_pdl(latent_queries_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(256), 0, stream, q, splits, (size_t)split_stride, q_row, heads, dim, rot, size, inv_freq, rotary_dim, interleaved, rot_scale, cu, len_before, sequences, (__nv_bfloat16*)out);
     TT_LAUNCH_CHECK();
 }
 

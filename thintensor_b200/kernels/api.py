@@ -811,10 +811,14 @@ def attention_tcgen05(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tenso
                       len_before: torch.Tensor, sequences: int, n_tokens: int, heads: int, kv_heads: int, head_dim: int,
                       scale: float, window: int, out: torch.Tensor, status: torch.Tensor, sinks: torch.Tensor | None = None,
                       softcap: float = 0.0, slopes: torch.Tensor | None = None, gate: torch.Tensor | None = None,
-                      gate_per_head: bool = False) -> None:
+                      gate_per_head: bool = False, out_dim: int | None = None) -> None:
     """Causal attention of packed bfloat16 prompts over the block cache with both products on
-    the tcgen05 tensor cores.  ``sinks``, ``softcap``, ``slopes``, ``gate``: see :func:`attention`."""
+    the tcgen05 tensor cores.  ``sinks``, ``softcap``, ``slopes``, ``gate``: see :func:`attention`.  ``out_dim``: only the first so many
+    numbers of a head's output are written, ``out`` ``[tokens, heads * out_dim]`` (heads padded to a size the kernel takes; no gate)."""
     _check_sinks(sinks, heads)
+    out_dim = head_dim if out_dim is None else int(out_dim)
+    if out.numel() != n_tokens * heads * out_dim or not 1 <= out_dim <= head_dim or (gate is not None and out_dim != head_dim):
+        raise KernelError("attention_tcgen05: the output does not fit the heads")
     if slopes is not None:
         _need(slopes, torch.float32, "slopes")
         if slopes.numel() != heads:
@@ -830,10 +834,10 @@ def attention_tcgen05(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tenso
         raise KernelError("queries, cache and output must all be contiguous bfloat16")
     fn = _fn("attention_tcgen05", "tt_attention_tcgen05", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int,
                                                            c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_void_p, c_float,
-                                                           c_void_p, c_void_p, c_int, c_longlong, c_int, c_int, c_void_p])
+                                                           c_void_p, c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_void_p])
     _check(fn(_ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(table), table.shape[1], k_pool.shape[0], _ptr(cu), _ptr(len_before), sequences,
               n_tokens, heads, kv_heads, head_dim, scale, _ptr(sinks), window, _ptr(out), _ptr(status), float(softcap or 0.0), _ptr(slopes),
-              g_ptr, g_splits, g_stride, g_row, 1 if gate_per_head else 0, _stream()), "attention_tcgen05")
+              g_ptr, g_splits, g_stride, g_row, 1 if gate_per_head else 0, out_dim, _stream()), "attention_tcgen05")
 
 
 # --------------------------------------------------------------------------- recurrent
@@ -1245,37 +1249,38 @@ def latent_expand(pool: torch.Tensor, table: torch.Tensor, cu: torch.Tensor, len
     """First half of expanding the latents a step of prompts can see into per-head keys and values laid out like cache blocks:
     ``table_tmp`` (int32 ``[sequences, table width]``) names, for every sequence, the temporary block that stands for each
     cache block the step reads (-1 elsewhere); ``x`` ``[bound_blocks * 64, rank]`` receives those blocks' latents (zero rows where
-    there is no token) for the product with ``[w_key; w_value]``, and ``keys`` ``[bound_blocks, heads, 64, dim + rot]`` the
-    shared rotated part behind every head's ``dim`` numbers.  ``plan``: int32 scratch ``[2 * sequences + 1]``.
+    there is no token) for the product with ``[w_key; w_value]``, and ``keys`` ``[bound_blocks, heads, 64, size]`` the
+    shared rotated part behind every head's ``dim`` numbers, zeros behind that (``size`` >= ``dim + rot``).  ``plan``: int32 scratch ``[2 * sequences + 1]``.
     ``bound_blocks`` must be at least the blocks the step can see (the kernel flags a bad shape otherwise)."""
     _need(plan, torch.int32, "expansion plan")
     _need(table_tmp, torch.int32, "temporary table")
     if (plan.numel() < 2 * sequences + 1 or tuple(table_tmp.shape) != tuple(table.shape) or tuple(x.shape) != (bound_blocks * BLOCK_TOKENS, rank)
-            or tuple(keys.shape) != (bound_blocks, heads, BLOCK_TOKENS, dim + rot) or not (pool.dtype == x.dtype == keys.dtype)
+            or tuple(keys.shape[:3]) != (bound_blocks, heads, BLOCK_TOKENS) or keys.shape[3] < dim + rot or not (pool.dtype == x.dtype == keys.dtype)
             or tuple(pool.shape[1:]) != (1, BLOCK_TOKENS, rank + rot) or not x.is_contiguous() or not keys.is_contiguous()):
         raise KernelError("latent_expand: shapes do not fit the sizes")
     fn = _fn("latent_attention", "tt_latent_expand_plan", [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p])
     _check(fn(_ptr(cu), _ptr(len_before), sequences, window, table.shape[1], bound_blocks, _ptr(plan), _ptr(table_tmp), _ptr(status), _stream()),
            "latent_expand_plan")
     fn = _fn("latent_attention", "tt_latent_gather", [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int,
-                                                      c_int, c_int, c_int, c_void_p, c_void_p, c_void_p])
+                                                      c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p])
     _check(fn(_ptr(pool), dtype_code(pool.dtype), _ptr(table), table.shape[1], pool.shape[0], _ptr(cu), _ptr(len_before), sequences, _ptr(plan),
-              bound_blocks, heads, dim, rot, rank, _ptr(x), _ptr(keys), _stream()), "latent_gather")
+              bound_blocks, heads, dim, rot, rank, keys.shape[3], _ptr(x), _ptr(keys), _stream()), "latent_gather")
 
 
 def latent_scatter(y: torch.Tensor, heads: int, dim: int, rot: int, vdim: int, keys: torch.Tensor, values: torch.Tensor) -> None:
     """Second half: ``y``, the float32 partial sums ``[slices, bound_blocks * 64, heads * dim + heads * vdim]`` of the gathered
     latents times ``[w_key; w_value]``, into the first ``dim`` numbers of every head's keys and into ``values``
-    ``[bound_blocks, heads, vdim, 64]`` (transposed inside a block, like the cache's)."""
+    ``[bound_blocks, heads, size, 64]`` (transposed inside a block, like the cache's; ``size`` is the keys', rows from ``vdim`` on are
+    not written)."""
     p, splits, stride, cols = _projection(y)
     blocks = keys.shape[0]
-    if (cols != heads * (dim + vdim) or y.shape[1] != blocks * BLOCK_TOKENS or tuple(keys.shape) != (blocks, heads, BLOCK_TOKENS, dim + rot)
-            or tuple(values.shape) != (blocks, heads, vdim, BLOCK_TOKENS) or keys.dtype != values.dtype
+    if (cols != heads * (dim + vdim) or y.shape[1] != blocks * BLOCK_TOKENS or tuple(keys.shape[:3]) != (blocks, heads, BLOCK_TOKENS)
+            or keys.shape[3] < max(dim + rot, vdim) or tuple(values.shape) != (blocks, heads, keys.shape[3], BLOCK_TOKENS) or keys.dtype != values.dtype
             or not keys.is_contiguous() or not values.is_contiguous()):
         raise KernelError("latent_scatter: shapes do not fit the sizes")
     fn = _fn("latent_attention", "tt_latent_scatter", [c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
                                                        c_void_p])
-    _check(fn(p, splits, stride, blocks, heads, dim, rot, vdim, _ptr(keys), _ptr(values), dtype_code(keys.dtype), _stream()), "latent_scatter")
+    _check(fn(p, splits, stride, blocks, heads, dim, keys.shape[3], vdim, _ptr(keys), _ptr(values), dtype_code(keys.dtype), _stream()), "latent_scatter")
 
 
 def latent_queries(q: torch.Tensor, heads: int, dim: int, rot: int, inv_freq: torch.Tensor, rotary_dim: int, cu: torch.Tensor,
@@ -1283,14 +1288,16 @@ def latent_queries(q: torch.Tensor, heads: int, dim: int, rot: int, inv_freq: to
                    rot_scale: float = 1.0) -> None:
     """The queries of the expanded form: the partial sums ``q`` ``[slices, tokens, heads * (dim + rot)]`` (possibly a range of a
     wider projection's columns) summed, every head's last ``rot`` numbers rotated by the position (the first ``rotary_dim`` of
-    them, halves or neighbours paired, cosines and sines times ``rot_scale``), narrowed to ``out``."""
+    them, halves or neighbours paired, cosines and sines times ``rot_scale``), narrowed to ``out`` ``[tokens, heads * size]`` with zeros
+    behind a head's ``dim + rot`` numbers."""
     _need(inv_freq, torch.float32, "inverse frequencies")
     p, splits, stride, q_row, cols = _projection_view(q)
-    if cols != heads * (dim + rot) or tuple(out.shape) != (n_tokens, cols) or not out.is_contiguous():
+    size = out.shape[1] // heads
+    if cols != heads * (dim + rot) or tuple(out.shape) != (n_tokens, heads * size) or size < dim + rot or not out.is_contiguous():
         raise KernelError("latent_queries: shapes do not fit the sizes")
-    fn = _fn("latent_attention", "tt_latent_queries", [c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_float,
+    fn = _fn("latent_attention", "tt_latent_queries", [c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_float,
                                                        c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p])
-    _check(fn(p, splits, stride, q_row, heads, dim, rot, _ptr(inv_freq), rotary_dim, 1 if interleaved else 0, float(rot_scale), _ptr(cu),
+    _check(fn(p, splits, stride, q_row, heads, dim, rot, size, _ptr(inv_freq), rotary_dim, 1 if interleaved else 0, float(rot_scale), _ptr(cu),
               _ptr(len_before), sequences, n_tokens, _ptr(out), dtype_code(out.dtype), _stream()), "latent_queries")
 
 
@@ -1756,6 +1763,32 @@ def gemm_tcgen05_swiglu(x: torch.Tensor, w: torch.Tensor, act: torch.Tensor, sta
                                                  c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_longlong])
     _check(fn(_ptr(x), x.stride(0), _ptr(w), w.stride(0), _ptr(None), _ptr(act), act.stride(0), 0, tokens, inter, k, 1,
               1 + 16 * GATE_ACTIVATIONS[activation], _ptr(status), _stream(), _ptr(None), 0), "gemm_tcgen05_swiglu")
+
+
+def gemm_tcgen05_unary_takes(x: torch.Tensor, w: torch.Tensor, width: int, activation: str) -> bool:
+    """Whether :func:`gemm_tcgen05_unary` takes these operands: a prompt of enough tiles, whole tiles of features, factors for whole tiles."""
+    tokens, features = x.shape[0], w.shape[0]
+    return (gemm_tcgen05_usable(x, w) and tokens > SKINNY_TOKENS and features % 256 == 0 and width % 128 == 0
+            and activation in ("silu", "relu", "gelu_tanh", "relu2") and -(-tokens // 128) * (features // 256) >= PERSISTENT_TILES)
+
+
+def gemm_tcgen05_unary(x: torch.Tensor, w: torch.Tensor, act: torch.Tensor, status: torch.Tensor, activation: str,
+                       scales: torch.Tensor | None = None, width: int = 128) -> None:
+    """act[t, f] = f(x[t] . w[f]) * scales[t, f // width] in bfloat16 with an ungated activation as the product's epilogue (``scales``
+    float32 ``[tokens, columns]``, None: no factor).  Only where :func:`gemm_tcgen05_unary_takes`."""
+    _need(act, torch.bfloat16, "activation output")
+    tokens, k = x.shape
+    features = w.shape[0]
+    if not gemm_tcgen05_unary_takes(x, w, width, activation) or w.shape[1] != k or tuple(act.shape) != (tokens, features):
+        raise KernelError(f"tcgen05 unary gemm cannot take x {tuple(x.shape)} / w {tuple(w.shape)} / act {tuple(act.shape)}")
+    if scales is not None:
+        _need(scales, torch.float32, "factors")
+        if scales.shape[0] != tokens or scales.shape[1] * width < features:
+            raise KernelError("gemm_tcgen05_unary: the factors do not fit the product")
+    fn = _fn("gemm_tcgen05", "tt_gemm_tcgen05_unary", [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_int, c_int,
+                                                       c_void_p, c_int, c_int, c_void_p, c_void_p])
+    _check(fn(_ptr(x), x.stride(0), _ptr(w), w.stride(0), _ptr(act), act.stride(0), tokens, features, k, UNARY_ACTIVATIONS[activation],
+              _ptr(scales), 0 if scales is None else scales.shape[1], width, _ptr(status), _stream()), "gemm_tcgen05_unary")
 
 
 def gemm_tcgen05_clamped(x: torch.Tensor, w: torch.Tensor, act: torch.Tensor, status: torch.Tensor, limit: float, shared_limit: float,

@@ -16,10 +16,10 @@ the queries are projected directly, ONE product makes ``[kv latent | shared key 
 Only ``[c | k_rot]`` is cached: one row per token, one key/value head, no value pool.  Decoding (and every step
 the tensor-core kernels do not take) never forms keys or values: the kernel folds ``W_uk`` into the query
 (``a = W_uk_h^T q_h``, so that ``q_h . W_uk_h c = a . c``) and applies ``W_uv_h`` once to the softmax-weighted sum of
-latents.  Prompts in bfloat16 whose heads have a size the tcgen05 attention kernel takes (``dim + rot_dim ==
-value_dim`` of 64 or 128) expand the latents the step can see into per-head keys and values for the length of the
-step, in scratch memory laid out like blocks of the ordinary cache, with one product over ``[W_uk; W_uv]``, and run
-that kernel on them: a prompt's arithmetic is then that of ordinary heads (``dim + rot_dim + value_dim`` numbers a
+latents.  Prompts in bfloat16 whose heads fit a size the tcgen05 attention kernel takes (``dim + rot_dim`` and
+``value_dim`` of at most 64 or 128) expand the latents the step can see into per-head keys and values for the length of the
+step, in scratch memory laid out like blocks of the ordinary cache (padded to the kernel's size), with one product over ``[W_uk; W_uv]``,
+and run that kernel on them: a prompt's arithmetic is then that of ordinary heads (``dim + rot_dim + value_dim`` numbers a
 pair instead of ``2 kv_rank + rot_dim``) and runs on the tensor cores.  Norms, positions, angles, scores and softmax
 weights are float32 in both dtypes.
 """
@@ -167,9 +167,13 @@ class LatentAttention(Mixer):
     EXPAND_FROM = 128           # packed tokens from which a step of prompts is expanded
 
     def expands(self, ctx, x) -> bool:
-        head = self.dim + self.rot_dim
-        return (not ctx.decode and ctx.n_tokens >= self.EXPAND_FROM and x.dtype == torch.bfloat16 and head == self.value_dim
-                and self.w_key.dtype == torch.bfloat16 and api.attention_tcgen05_supports(x.dtype, self.heads, self.heads, head))
+        return (not ctx.decode and ctx.n_tokens >= self.EXPAND_FROM and x.dtype == torch.bfloat16 and self.expanded_size is not None
+                and self.w_key.dtype == torch.bfloat16 and api.attention_tcgen05_supports(x.dtype, self.heads, self.heads, self.expanded_size))
+
+    @property
+    def expanded_size(self) -> int | None:
+        """The head size of the tcgen05 attention kernel that holds a head's keys and values."""
+        return next((size for size in (64, 128) if max(self.dim + self.rot_dim, self.value_dim) <= size), None)
 
     def expansion_bound(self, ctx, width: int) -> int:
         """Temporary blocks the step can need, from the step's shape alone (a replayed step has other lengths): every
@@ -179,13 +183,13 @@ class LatentAttention(Mixer):
         return min(ctx.sequences * width, (ctx.n_tokens + ctx.sequences * (self.window - 1)) // 64 + 2 * ctx.sequences)
 
     def attend_expanded(self, ctx, q, cache, table, mixed) -> None:
-        head = self.dim + self.rot_dim
+        head = self.expanded_size
         blocks = self.expansion_bound(ctx, table.shape[1])
         plan = ctx.scratch("latent.plan", (2 * ctx.sequences + 1,), torch.int32)
         table_tmp = ctx.scratch("latent.table", tuple(table.shape), torch.int32)
         latents = ctx.scratch("latent.visible", (blocks * 64, self.kv_rank))
         keys = ctx.scratch("latent.keys", (blocks, self.heads, 64, head))
-        values = ctx.scratch("latent.values", (blocks, self.heads, self.value_dim, 64))
+        values = ctx.scratch("latent.values", (blocks, self.heads, head, 64))
         api.latent_expand(cache.k_pool, table, ctx.cu, ctx.len_before, ctx.sequences, self.window or 0, blocks, self.heads, self.dim,
                           self.rot_dim, self.kv_rank, plan, table_tmp, latents, keys, ctx.status)
         expanded = self.expander(ctx, latents, "latent.expand")
@@ -194,4 +198,4 @@ class LatentAttention(Mixer):
         api.latent_queries(q, self.heads, self.dim, self.rot_dim, self.rot.inv_freq, self.rot.rotary_dim, ctx.cu, ctx.len_before,
                            ctx.sequences, ctx.n_tokens, queries, interleaved=self.rot.interleaved, rot_scale=self.rot.attention_scaling)
         api.attention_tcgen05(queries, keys, values, table_tmp, ctx.cu, ctx.len_before, ctx.sequences, ctx.n_tokens, self.heads, self.heads,
-                              head, self.scale, self.window or 0, mixed, ctx.status)
+                              head, self.scale, self.window or 0, mixed, ctx.status, out_dim=self.value_dim)

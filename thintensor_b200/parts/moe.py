@@ -151,5 +151,9 @@ class MixtureOfExperts(FeedForward):
     def ungated(self, ctx, x, gates) -> torch.Tensor:
         """``f(up x)`` of every expert's columns times the token's weight for the expert."""
         act = ctx.scratch("moe.up.act", (ctx.n_tokens, self.experts * self.inter))
+        if api.gemm_tcgen05_unary_takes(x, self.up.weight, self.inter, self.activation):      # all in the product's epilogue
+            api.set_label("moe.up")
+            api.gemm_tcgen05_unary(x, self.up.weight, act, ctx.status, self.activation, gates, self.inter)
+            return act
         api.expert_unary_activation(self.up(ctx, x, "moe.up"), act, self.inter, self.activation, gates)
         return act
