@@ -1073,7 +1073,8 @@ constexpr int SHIFT_BLENDS = 8;
 
 template <typename T, int VEC> struct alignas(VEC * sizeof(T)) ShiftPack { T v[VEC]; };
 
-template <typename T, int VEC>
+// BLENDS > 0: so many blends, whose weights stay in registers for the tile; 0: `blends` of them, fetched for every token
+template <typename T, int VEC, int BLENDS>
 __global__ void token_shifts_kernel(const T* __restrict__ x, const float* __restrict__ mix, int blends, float* __restrict__ state,
                                     T* __restrict__ out, size_t out_stride, const int* __restrict__ cu, const int* __restrict__ slots,
                                     int sequences, int n_tokens, int hidden, int tile) {
@@ -1083,10 +1084,22 @@ __global__ void token_shifts_kernel(const T* __restrict__ x, const float* __rest
     const int t0 = blockIdx.x * tile, t1 = min(t0 + tile, n_tokens);
     int b = tt_find_sequence(cu, sequences, t0);
     int first = cu[b], next = cu[b + 1];
-    float before[VEC];
+    float before[VEC], w[BLENDS > 0 ? BLENDS : 1][VEC];
+    auto weights = [&](int m, float (&to)[VEC]) {
+        const ShiftPack<float, VEC> p = *reinterpret_cast<const ShiftPack<float, VEC>*>(mix + (size_t)m * hidden + j);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) to[e] = p.v[e];
+    };
+    if constexpr (BLENDS > 0) {                                 // written by no kernel: fetched before the wait
+#pragma unroll
+        for (int m = 0; m < BLENDS; ++m) weights(m, w[m]);
+    }
     tt_pdl_wait();
     using Pack = ShiftPack<T, VEC>;
+    Pack ahead = *reinterpret_cast<const Pack*>(x + (size_t)t0 * hidden + j);
     for (int t = t0; t < t1; ++t) {
+        const Pack row = ahead;
+        if (t + 1 < t1) ahead = *reinterpret_cast<const Pack*>(x + (size_t)(t + 1) * hidden + j);
         while (t >= next) {                                     // the next sequence starts here
             ++b;
             first = next;
@@ -1101,19 +1114,24 @@ __global__ void token_shifts_kernel(const T* __restrict__ x, const float* __rest
                 st[e] = tt_to_float(tail.v[e]);
             }
         } else if (t == t0) {
-            const Pack row = *reinterpret_cast<const Pack*>(x + (size_t)(t - 1) * hidden + j);
+            const Pack last = *reinterpret_cast<const Pack*>(x + (size_t)(t - 1) * hidden + j);
 #pragma unroll
-            for (int e = 0; e < VEC; ++e) before[e] = tt_to_float(row.v[e]);
+            for (int e = 0; e < VEC; ++e) before[e] = tt_to_float(last.v[e]);
         }
-        const Pack row = *reinterpret_cast<const Pack*>(x + (size_t)t * hidden + j);
         float now[VEC];
 #pragma unroll
         for (int e = 0; e < VEC; ++e) now[e] = tt_to_float(row.v[e]);
-        for (int m = 0; m < blends; ++m) {
+        auto put = [&](int m, const float (&by)[VEC]) {
             Pack o;
 #pragma unroll
-            for (int e = 0; e < VEC; ++e) o.v[e] = tt_from_float<T>(fmaf(before[e] - now[e], __ldg(mix + (size_t)m * hidden + j + e), now[e]));
+            for (int e = 0; e < VEC; ++e) o.v[e] = tt_from_float<T>(fmaf(before[e] - now[e], by[e], now[e]));
             *reinterpret_cast<Pack*>(out + (size_t)m * out_stride + (size_t)t * hidden + j) = o;
+        };
+        if constexpr (BLENDS > 0) {
+#pragma unroll
+            for (int m = 0; m < BLENDS; ++m) put(m, w[m]);
+        } else {
+            for (int m = 0; m < blends; ++m) { weights(m, w[0]); put(m, w[0]); }
         }
 #pragma unroll
         for (int e = 0; e < VEC; ++e) before[e] = now[e];
@@ -1126,14 +1144,16 @@ extern "C" int tt_token_shifts(const void* x, int dtype, const float* mix, int b
     if (n_tokens <= 0) return 0;
     if (blends < 1 || blends > SHIFT_BLENDS || hidden <= 0) return (int)cudaErrorInvalidValue;
     const int vec = dtype == TT_F32 ? 4 : 8, threads = 128;
-    const bool wide = hidden % vec == 0 && out_stride % vec == 0 && (((uintptr_t)x | (uintptr_t)out) & 15) == 0;
-    const int per_block = threads * (wide ? vec : 1), tile = n_tokens >= 1024 ? 8 : 1;
+    const bool wide = hidden % vec == 0 && out_stride % vec == 0 && (((uintptr_t)x | (uintptr_t)out | (uintptr_t)mix) & (dtype == TT_F32 ? 15 : 31)) == 0;
+    const int per_block = threads * (wide ? vec : 1), tile = n_tokens >= 1024 ? 4 : 1;
     const dim3 grid((n_tokens + tile - 1) / tile, (hidden + per_block - 1) / per_block), block(threads);
     if (grid.y > 65535) return (int)cudaErrorInvalidValue;
-#define TT_SHIFTS(T, V) tt_launch_pdl(token_shifts_kernel<T, V>, grid, block, 0, stream, (const T*)x, mix, blends, state, (T*)out, (size_t)out_stride, cu, slots, sequences, n_tokens, hidden, tile)
+#define TT_SHIFTS_FORM(T, V, B) tt_launch_pdl(token_shifts_kernel<T, V, B>, grid, block, 0, stream, (const T*)x, mix, blends, state, (T*)out, (size_t)out_stride, cu, slots, sequences, n_tokens, hidden, tile)
+#define TT_SHIFTS(T, V) do { if (blends == 5) TT_SHIFTS_FORM(T, V, 5); else TT_SHIFTS_FORM(T, V, 0); } while (0)
     if (dtype == TT_F32) { if (wide) TT_SHIFTS(float, 4); else TT_SHIFTS(float, 1); }
     else { if (wide) TT_SHIFTS(__nv_bfloat16, 8); else TT_SHIFTS(__nv_bfloat16, 1); }
 #undef TT_SHIFTS
+#undef TT_SHIFTS_FORM
     TT_LAUNCH_CHECK();
 }
 
