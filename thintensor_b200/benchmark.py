@@ -201,7 +201,7 @@ def class_fractions(model, classes: dict, pk: dict, prefill_prompts: list[list[i
     one after another (see :func:`measure_classes`)."""
     attention_kernels = ("tt_attention", "tt_latent_attention", "tt_differential_attention", "tt_pooled_window_attention")
     recurrent = ("tt_mamba2_scan", "tt_delta_scan", "tt_causal_conv", "tt_gated_group_norm", "tt_decay_scan", "tt_row_decay_scan", "tt_row_decay_blocks",
-                 "tt_low_rank", "tt_low_rank_inputs", "tt_low_rank_finish", "tt_linear_attention_prepare", "tt_token_shifts")
+                 "tt_low_rank", "tt_low_rank_inputs", "tt_low_rank_finish", "tt_linear_attention_prepare")
 
     def split(spans: dict) -> dict:
         out = {"products": 0.0, "attention": 0.0, "recurrence": 0.0, "rest": 0.0}
