@@ -52,7 +52,7 @@ CONFIGS = {
         "layers": [
             {"type": "latent_attention_2", "mlp": _dense(160, 1.5), "mixer": {
                 "heads": 3, "dim": 72, "rot_dim": 32, "vdim": 100, "kv_rank": 64, "scale": 0.11, "rot": {"dims": 32, "base": 100000.0}}},
-            {"type": "wkv", "mlp": _moe(8, 3, 128, 1.3), "mixer": {"heads": 2, "dim": 128}},
+            {"type": "wkv", "mlp": _moe(8, 4, 128, 1.3), "mixer": {"heads": 2, "dim": 128}},
             {"type": "latent_attention", "mlp": _moe(6, 2, 64, 0.9), "mixer": {
                 "heads": 4, "dim": 32, "rot_dim": 16, "vdim": 56, "kv_rank": 48, "q_rank": 72, "scale": 0.16, "rot": {"dims": 16, "base": 10000.0}}},
             {"type": "wkv", "mlp": _dense(96, 1.0), "mixer": {"heads": 4, "dim": 32}},
